@@ -12,6 +12,7 @@ from dataclasses import dataclass
 from pathlib import Path
 from typing import Any, Callable
 
+from .gedunex import GedunexConfig, gedunex_model_spec
 from .llama import LlamaConfig, UnsupportedModelError, llama_model_spec
 from .lokolorn import LokolornConfig, lokolorn_model_spec
 from .pazenex import PazenexConfig, pazenex_model_spec
@@ -66,3 +67,4 @@ register_architecture(Architecture("Pazenex", PazenexConfig.from_dict, pazenex_m
 register_architecture(Architecture("Sugonex", SugonexConfig.from_dict, sugonex_model_spec))
 register_architecture(Architecture("Pokadra", PokadraConfig.from_dict, pokadra_model_spec))
 register_architecture(Architecture("Lokolorn", LokolornConfig.from_dict, lokolorn_model_spec))
+register_architecture(Architecture("Gedunex", GedunexConfig.from_dict, gedunex_model_spec))

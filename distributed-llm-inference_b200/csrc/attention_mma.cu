@@ -19,6 +19,7 @@
 // Shared-memory rows are padded by 16 bytes: for every head size that is a multiple of 16 the
 // eight rows an ldmatrix reads then fall into eight different 16-byte bank groups.
 #include "common.cuh"
+#include "score_bend.cuh"
 #include <math_constants.h>
 
 #ifndef HEAD_DIM
@@ -55,7 +56,8 @@ struct Params {
   const int* kv_len;         // [seqs]
   int seq0;                  // first sequence of this launch
   int nh, nkv, page_size, window;
-  float scale_log2;          // softmax scale times log2(e)
+  float scale_log2;          // softmax scale times log2(e); 1 with BENT_SCORES (the scores then come in log2 units)
+  ScoreBend bend;            // what happens to the scores (BENT_SCORES only)
   float sink_log2;           // score of a sink (a term of the denominator without a value) times log2(e); -inf: none
   const float* sink_heads;   // if not null: a sink score per query head (natural units), instead of sink_log2
   int tokens_per_tile, heads_per_chunk, head_chunks, splits;
@@ -147,7 +149,8 @@ __device__ __forceinline__ void load_kv_tile(unsigned char* dK, unsigned char* d
 template <int NK>
 __device__ __forceinline__ void tile_update(const unsigned char* sQ, const unsigned char* tK, const unsigned char* tV, int base,
                                             const bool (&rvalid)[2], const int (&rpos)[2], int window, float scale_log2,
-                                            float (&m)[2], float (&l)[2], float (&o)[D / 8][4], int lane) {
+                                            const ScoreBend& bend, const float (&slope)[2], float (&m)[2], float (&l)[2],
+                                            float (&o)[D / 8][4], int lane) {
   // ---- S = Q K^T
   float sc[NK / 8][4];
 #pragma unroll
@@ -177,7 +180,11 @@ __device__ __forceinline__ void tile_update(const unsigned char* sQ, const unsig
       const int key = base + j * 8 + (lane & 3) * 2 + (e & 1);
       bool ok = rvalid[rr] && key <= rpos[rr];
       if (window > 0) ok = ok && key > rpos[rr] - window;
+#if BENT_SCORES
+      const float t = ok ? bent_score(sc[j][e], bend, slope[rr] * (float)(key - rpos[rr])) : -CUDART_INF_F;
+#else
       const float t = ok ? sc[j][e] * scale_log2 : -CUDART_INF_F;
+#endif
       sc[j][e] = t;
       tmax[rr] = fmaxf(tmax[rr], t);
     }
@@ -292,6 +299,11 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
     rpos[0] = pos0 + t0;
     rpos[1] = pos0 + t1;
   }
+  float slope[2] = {0.f, 0.f};
+#if BENT_SCORES
+  if (rvalid[0]) slope[0] = bend_slope(p.bend, head0 + r0 % Gc);
+  if (rvalid[1]) slope[1] = bend_slope(p.bend, head0 + r1 % Gc);
+#endif
 
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F};
   float l[2] = {0.f, 0.f};
@@ -311,7 +323,7 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
 
     if (warp_active)
       tile_update<BLOCK_N>(sQ + warp * 16 * ROW_BYTES, sK + stage * TILE_BYTES, sV + stage * TILE_BYTES, (t_begin + it) * BLOCK_N,
-                           rvalid, rpos, p.window, p.scale_log2, m, l, o, lane);
+                           rvalid, rpos, p.window, p.scale_log2, p.bend, slope, m, l, o, lane);
     __syncthreads();  // the stage is overwritten by the load issued next iteration
   }
   cp_async_wait<0>();
@@ -422,6 +434,11 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
   const int rows[2] = {lane >> 2, (lane >> 2) + 8};
   const bool rvalid[2] = {rows[0] < nheads, rows[1] < nheads};
   const int rpos[2] = {pos, pos};
+  float slope[2] = {0.f, 0.f};
+#if BENT_SCORES
+  if (rvalid[0]) slope[0] = bend_slope(p.bend, head0 + rows[0]);
+  if (rvalid[1]) slope[1] = bend_slope(p.bend, head0 + rows[1]);
+#endif
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F};
   float l[2] = {0.f, 0.f};
   float o[D / 8][4];
@@ -442,7 +459,7 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
     cp_async_wait<DEC_STAGES - 1>();
     __syncwarp();
     tile_update<DEC_N>(sQ, wK + stage * DEC_TILE_BYTES, wV + stage * DEC_TILE_BYTES, (t_begin + warp + it * NWARPS) * DEC_N, rvalid,
-                       rpos, p.window, p.scale_log2, m, l, o, lane);
+                       rpos, p.window, p.scale_log2, p.bend, slope, m, l, o, lane);
     __syncwarp();  // the stage is overwritten by the load issued next iteration
   }
   cp_async_wait<0>();
@@ -531,9 +548,10 @@ __global__ void merge_splits_kernel(bf16* __restrict__ out, const float* __restr
 DLI_EXPORT int dli_paged_attention_mma(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                        const int* block_tables, int max_blocks, const int* q_start, const int* kv_len,
                                        int seq0, int num_seqs, int max_q_len, int first_row, int nh, int nkv, int page_size,
-                                       int window, float scale, float sink, const float* sink_heads, int splits, float* part_acc,
-                                       float* part_ml, cudaStream_t stream) {
+                                       int window, float scale, float sink, const float* sink_heads, float softcap, const float* slopes,
+                                       int splits, float* part_acc, float* part_ml, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
+  if (!BENT_SCORES && (softcap != 0.f || slopes)) return DLI_ERR_UNSUPPORTED;
   if (nkv < 1 || nh % nkv || splits < 1 || (splits > 1 && (max_q_len != 1 || !part_acc || !part_ml))) return DLI_ERR_UNSUPPORTED;
   static OncePerDevice configured;
   if (!configured.here()) {
@@ -556,7 +574,8 @@ DLI_EXPORT int dli_paged_attention_mma(void* out, const void* q, long long q_str
   p.k_pool = (const bf16*)k_pool; p.v_pool = (const bf16*)v_pool;
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.q_start = q_start; p.kv_len = kv_len; p.seq0 = seq0;
   p.nh = nh; p.nkv = nkv; p.page_size = page_size; p.window = window;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = BENT_SCORES ? 1.f : scale * 1.4426950408889634f;
+  p.bend = make_score_bend(scale, softcap, slopes);
   p.sink_log2 = sink * 1.4426950408889634f;  // -inf (no sink) stays -inf
   p.sink_heads = sink_heads;
   const int G = nh / nkv;
@@ -633,5 +652,5 @@ DLI_EXPORT int dli_paged_decode_attention_noalloc(void* out, const void* q, long
   float* part_ml = part_acc + rows * (unsigned long long)splits * (unsigned long long)D;
   if (splits == 1) part_acc = part_ml = nullptr;  // no partial results: the kernel writes the output itself
   return dli_paged_attention_mma(out, q, q_stride, k_pool, v_pool, block_tables, max_blocks, q_start, kv_len, seq0, num_seqs, 1,
-                                 first_row, nh, nkv, page_size, window, scale, -INFINITY, nullptr, splits, part_acc, part_ml, stream);
+                                 first_row, nh, nkv, page_size, window, scale, -INFINITY, nullptr, 0.f, nullptr, splits, part_acc, part_ml, stream);
 }

@@ -415,6 +415,140 @@ DLI_EXPORT int dli_rotary_unit_store(void* q_out, const void* x, long long x_str
   return (int)e;
 }
 
+// ---------------------------------------------------------------- whole-projection norm, temperature, mixed values, then the pages
+// One block per token.  x row: q (nh heads of d) | k (nkv heads of d) | v (nkv heads of dv), plus a float32 bias (or none).
+//   q <- q / rms(q over all heads) * wq * temp,  k <- k / rms(k over all heads) * wk                        (normed != 0)
+//   temp = 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) at position p                                 (temp_coef != 0)
+//   mix 1: v -> source [n][nkv dv] (float32, for the layers behind this one);  mix 2: v <- (1 - lam) v + lam source
+// Rows of D >= max(d, dv) numbers leave, padded with zeros: q -> q_out [n][nh][D]; k, v -> pools [pages][nkv][page_size][D]
+// at the token's slot (if slots).  VEC columns a thread at a time (8: d, dv, D multiples of 8 and aligned rows; else 1).
+template <typename TI, int VEC>
+__device__ __forceinline__ void load_run(const TI* __restrict__ x, const float* __restrict__ bias, int c, float (&v)[VEC]) {
+  if constexpr (VEC == 8) {
+    load8(x + c, v);
+    if (bias) {
+      float b[8];
+      load8(bias + c, b);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[k] += b[k];
+    }
+  } else {
+    v[0] = to_float(x[c]) + (bias ? bias[c] : 0.f);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_run(T* __restrict__ dst, const float (&v)[VEC]) {
+  if constexpr (VEC == 8) store8(dst, v);
+  else dst[0] = from_float<T>(v[0]);
+}
+
+template <typename TI, typename T, int VEC>
+__global__ void qk_norm_mix_store_kernel(T* __restrict__ q_out, const TI* __restrict__ x, const float* __restrict__ bias, const float* __restrict__ wq,
+                                         const float* __restrict__ wk, float eps, const int* __restrict__ positions, float temp_coef, float temp_every,
+                                         float* __restrict__ source, float lam, const int* __restrict__ slots, T* __restrict__ k_pool,
+                                         T* __restrict__ v_pool, int nh, int nkv, int d, int dv, int D, int page_size, int mix, int normed) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[33];
+  const int t = blockIdx.x;
+  const int nq = nh * d, nk = nkv * d, nv = nkv * dv;
+  const TI* src = x + (size_t)t * (nq + nk + nv);
+  float rq = 1.f, rk = 1.f;
+  if (normed) {
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * VEC; c < nq + nk; c += blockDim.x * VEC) {
+      float v[VEC];
+      load_run<TI, VEC>(src, bias, c, v);
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) ss = fmaf(v[k], v[k], ss);
+      if (c < nq) sq += ss; else sk += ss;
+    }
+    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
+    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+  }
+  if (temp_coef != 0.f) rq *= 1.f + temp_coef * logf(floorf((float)(positions[t] + 1) / temp_every) + 1.f);
+  const int slot = slots ? slots[t] : -1;
+  const long long page = slot >= 0 ? slot / page_size : 0;
+  const int off = slot >= 0 ? slot - (int)page * page_size : 0;
+  const int per = D / VEC;  // runs of a head's row as it leaves
+  const int heads = nh + (slot >= 0 ? 2 * nkv : (mix == 1 ? 2 * nkv : 0));
+  for (int item = threadIdx.x; item < heads * per; item += blockDim.x) {
+    const int head = item / per, i = (item - head * per) * VEC;
+    float v[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = 0.f;
+    if (head < nh + nkv) {
+      const bool is_q = head < nh;
+      if (!is_q && slot < 0) continue;
+      if (i < d) {
+        const int c = head * d + i;  // q heads, then k heads, lie back to back
+        load_run<TI, VEC>(src, bias, c, v);
+        const float r = is_q ? rq : rk;
+        if (normed) {
+          float w[VEC];
+          load_run<float, VEC>(is_q ? wq : wk, nullptr, is_q ? c : c - nq, w);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) v[k] = v[k] * r * w[k];
+        } else {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) v[k] *= r;
+        }
+      }
+      T* dst = is_q ? q_out + ((size_t)t * nh + head) * D : k_pool + ((page * nkv + (head - nh)) * page_size + off) * D;
+      store_run<T, VEC>(dst + i, v);
+    } else {
+      const int g = head - nh - nkv;
+      if (i < dv) {
+        const int c = g * dv + i;
+        load_run<TI, VEC>(src + nq + nk, bias ? bias + nq + nk : nullptr, c, v);
+        float* s = mix ? source + (size_t)t * nv + c : nullptr;
+        if (mix == 1) {
+          store_run<float, VEC>(s, v);
+        } else if (mix == 2) {
+          float first[VEC];
+          load_run<float, VEC>(s, nullptr, 0, first);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) v[k] = (1.f - lam) * v[k] + lam * first[k];
+        }
+      }
+      if (slot >= 0) store_run<T, VEC>(v_pool + ((page * nkv + g) * page_size + off) * D + i, v);
+    }
+  }
+}
+
+template <typename TI, typename T>
+static int launch_qk_norm_mix_store(void* q_out, const void* x, const float* bias, const float* wq, const float* wk, float eps, const int* positions,
+                                    float temp_coef, float temp_every, float* source, float lam, const int* slots, void* k_pool, void* v_pool, int n,
+                                    int nh, int nkv, int d, int dv, int D, int page_size, int mix, int normed, cudaStream_t stream) {
+  const bool vec = (d % 8) == 0 && (dv % 8) == 0 && (D % 8) == 0 &&
+                   (((uintptr_t)q_out | (uintptr_t)x | (uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk | (uintptr_t)source | (uintptr_t)k_pool |
+                     (uintptr_t)v_pool) & 15) == 0;
+  const int items = (nh + 2 * nkv) * (vec ? D / 8 : D);
+  const int threads = items >= 512 ? 512 : (items >= 256 ? 256 : (items >= 128 ? 128 : 64));
+#define DLI_QKM(V)                                                                                                                            \
+  launch_pdl((qk_norm_mix_store_kernel<TI, T, V>), dim3(n), dim3(threads), 0, stream, 1, (T*)q_out, (const TI*)x, bias, wq, wk, eps, positions, \
+             temp_coef, temp_every, source, lam, slots, (T*)k_pool, (T*)v_pool, nh, nkv, d, dv, D, page_size, mix, normed)
+  return (int)(vec ? DLI_QKM(8) : DLI_QKM(1));
+#undef DLI_QKM
+}
+
+DLI_EXPORT int dli_qk_norm_mix_store(void* q_out, const void* x, const float* bias, const float* wq, const float* wk, float eps, const int* positions,
+                                     float temp_coef, float temp_every, float* source, float lam, const int* slots, void* k_pool, void* v_pool, int n,
+                                     int nh, int nkv, int d, int dv, int D, int page_size, int mix, int normed, int in_dtype, int dtype,
+                                     cudaStream_t stream) {
+  if (n == 0) return 0;
+  if (nh < 1 || nkv < 1 || nh % nkv || d < 1 || dv < 1 || D < d || D < dv || page_size < 1 || (slots && (!k_pool || !v_pool)) || (mix && !source) ||
+      mix < 0 || mix > 2 || (normed && (!wq || !wk)) || (temp_coef != 0.f && !(temp_every > 0.f)))
+    return DLI_ERR_UNSUPPORTED;
+#define DLI_QKM(TI, T)                                                                                                                        \
+  launch_qk_norm_mix_store<TI, T>(q_out, x, bias, wq, wk, eps, positions, temp_coef, temp_every, source, lam, slots, k_pool, v_pool, n, nh, nkv, \
+                                  d, dv, D, page_size, mix, normed, stream)
+  if (dtype == DLI_F32) return in_dtype == DLI_F32 ? DLI_QKM(float, float) : DLI_ERR_UNSUPPORTED;
+  return in_dtype == DLI_F32 ? DLI_QKM(float, __nv_bfloat16) : DLI_QKM(__nv_bfloat16, __nv_bfloat16);
+#undef DLI_QKM
+}
+
 // ---------------------------------------------------------------- a product per head, for a decode step's few tokens
 // out[t, h, f] = sum_i x[t, h, i] * w[h, i, f]  (float32 sums), times sigmoid(gate[t, h, f]) if a gate is given.
 // x, out and gate are column slices of wider rows (row and head strides in elements); w [heads][in][features] is

@@ -14,7 +14,7 @@ __global__ void paged_attention_simt_kernel(T* __restrict__ out, const T* __rest
                                             const int* __restrict__ block_tables, int max_blocks,
                                             const int* __restrict__ seq_of_token, const int* __restrict__ positions, int n,
                                             int nh, int nkv, int d, int page_size, int window, float scale, float sink,
-                                            const float* __restrict__ sink_heads) {
+                                            const float* __restrict__ sink_heads, float softcap, const float* __restrict__ slopes) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float smem[];
@@ -31,6 +31,7 @@ __global__ void paged_attention_simt_kernel(T* __restrict__ out, const T* __rest
   __syncwarp();
 
   const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
+  const float slope = slopes ? slopes[h] : 0.f;
   float m = -CUDART_INF_F, l = 0.f;
   float acc[R];
 #pragma unroll
@@ -48,6 +49,8 @@ __global__ void paged_attention_simt_kernel(T* __restrict__ out, const T* __rest
       float dot = 0.f;
       for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_float(kr[i]), dot);
       sc = dot * scale;
+      if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+      sc -= slope * (float)(p - key);
     }
     const float m_new = fmaxf(m, warp_max(sc));
     const float pj = valid ? expf(sc - m_new) : 0.f;
@@ -83,7 +86,8 @@ __global__ void paged_attention_simt_kernel(T* __restrict__ out, const T* __rest
 DLI_EXPORT int dli_paged_attention_simt(void* out, const void* q, int q_stride, const void* k_pool, const void* v_pool,
                                         const int* block_tables, int max_blocks, const int* seq_of_token,
                                         const int* positions, int n, int nh, int nkv, int d, int page_size, int window,
-                                        float scale, float sink, const float* sink_heads, int dtype, cudaStream_t stream) {
+                                        float scale, float sink, const float* sink_heads, float softcap, const float* slopes, int dtype,
+                                        cudaStream_t stream) {
   if (n == 0) return 0;
   if (d < 1 || d > 1024 || nkv < 1 || nh % nkv) return DLI_ERR_UNSUPPORTED;
   const int warps = 4;
@@ -93,7 +97,7 @@ DLI_EXPORT int dli_paged_attention_simt(void* out, const void* q, int q_stride, 
 #define DLI_SIMT(T, R)                                                                                                                  \
   launch_pdl((paged_attention_simt_kernel<T, R>), dim3(blocks), dim3(warps * 32), smem, stream, 1, (T*)out, (const T*)q, q_stride,       \
              (const T*)k_pool, (const T*)v_pool, block_tables, max_blocks, seq_of_token, positions, n, nh, nkv, d, page_size, window, \
-             scale, sink, sink_heads)
+             scale, sink, sink_heads, softcap, slopes)
   if (dtype == DLI_F32) {
     if (d <= 256) DLI_SIMT(float, 8);
     else DLI_SIMT(float, 32);

@@ -22,6 +22,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "score_bend.cuh"
 #include <math_constants.h>
 
 using namespace dli;
@@ -48,7 +49,8 @@ struct Params {
   const int* q_start;
   const int* kv_len;
   int seq0, nh, nkv, page_size, window;
-  float scale_log2;
+  float scale_log2;  // 1 with BENT_SCORES: the scores then come in log2 units
+  ScoreBend bend;    // what happens to the scores (BENT_SCORES only)
   float sink_log2;  // score of a sink (a term of the denominator without a value) times log2(e); -inf: none
   const float* sink_heads;  // if not null: a sink score per query head (natural units), instead of sink_log2
   int tokens_per_tile, heads_per_chunk, head_chunks;
@@ -117,6 +119,21 @@ __device__ __forceinline__ float sink_term(float sink_log2, float m) {
 __device__ __forceinline__ float sink_of(const float* sink_heads, float sink_log2, int head) {
   return sink_heads ? sink_heads[head] * 1.4426950408889634f : sink_log2;
 }
+#if BENT_SCORES
+// N consecutive raw scores of a row, bent in place; the first belongs to the key `offset` places behind the query (negative: ahead,
+// masked later).
+template <int N>
+__device__ __forceinline__ void bend_row(float (&sc)[N], const ScoreBend& b, float slope, int offset) {
+  const float first = -slope * (float)offset;
+  if (b.cap_log2 != 0.f) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) sc[j] = capped_score(sc[j], b, fmaf(slope, (float)j, first));
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) sc[j] = fmaf(sc[j], b.scale_log2, fmaf(slope, (float)j, first));
+  }
+}
+#endif
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
 }
@@ -312,6 +329,9 @@ __global__ void __launch_bounds__(THREADS, 1) paged_prefill_tc_kernel(const __gr
     constexpr float RESCALE_STEP = 8.f;
     float m = -CUDART_INF_F, m_ref = -CUDART_INF_F, l = 0.f;
     bool ok = true;
+#if BENT_SCORES
+    const float slope = rvalid ? bend_slope(p.bend, head0 + (r - rtok * Gc)) : 0.f;
+#endif
     const int group = r >> 6;  // rows 0..63 (warps 0, 1, 4, 5) and rows 64..127 (warps 2, 3, 6, 7)
     const uint32_t my_o = tmem_o + lane_bits + half * 32;  // output columns 32 * half .. 32 * half + 31 of the row
 
@@ -335,6 +355,9 @@ __global__ void __launch_bounds__(THREADS, 1) paged_prefill_tc_kernel(const __gr
 #pragma unroll
         for (int j = 0; j < 32; ++j) { sc[j] = __uint_as_float(v0[j]); sc[32 + j] = __uint_as_float(v1[j]); }
       }
+#if BENT_SCORES
+      bend_row(sc, p.bend, slope, rpos - base - col0);
+#endif
       if (!full) {
         const int first = base + col0;  // visible: first + j in (rpos - window, rpos]
         const int hi_j = rpos - first, lo_j = p.window > 0 ? rpos - p.window - first : -1;
@@ -675,6 +698,9 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     float m = -CUDART_INF_F, m_ref = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     const int first_pos = pos0 + q * tpt;  // position of the tile's first row
+#if BENT_SCORES
+    const float slope = rvalid ? bend_slope(p.bend, head0 + (r % Gc)) : 0.f;
+#endif
     // where this row's eight 16-byte chunks of a 128-byte slab of P lie (the swizzle), as shared-memory addresses: a
     // store then needs no address arithmetic of its own (through a generic pointer each cost five instructions more;
     // 8,192 tokens: 455 -> 436 us)
@@ -702,6 +728,9 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       mbar_arrive(my_s_read);  // S is in registers: the next product of this tile may overwrite it
+#if BENT_SCORES
+      bend_row(sc, p.bend, slope, rpos - base);
+#endif
       // a tile that lies wholly at or before the first row's position, inside every row's window, needs no mask
       const bool full = base + KEYS - 1 <= first_pos && base >= lo && p.window <= 0;
       if (!full) {
@@ -852,8 +881,10 @@ int* error_flag_host = nullptr;
 DLI_EXPORT int dli_paged_prefill_tc(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long num_pages, const int* block_tables, int max_blocks, const int* q_start,
                                     const int* kv_len, int seq0, int num_seqs, int max_q_len, int nh, int nkv, int head_dim,
-                                    int page_size, int window, float scale, float sink, const float* sink_heads, int query_tiles, cudaStream_t stream) {
+                                    int page_size, int window, float scale, float sink, const float* sink_heads, float softcap, const float* slopes,
+                                    int query_tiles, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
+  if (!BENT_SCORES && (softcap != 0.f || slopes)) return DLI_ERR_UNSUPPORTED;
   if (head_dim != 64 && head_dim != 128) return DLI_ERR_UNSUPPORTED;
   if (nkv < 1 || nh % nkv || page_size < 8 || page_size > 128 || (KEYS % page_size) != 0) return DLI_ERR_UNSUPPORTED;
   if (((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)q) & 15) return DLI_ERR_UNSUPPORTED;
@@ -875,7 +906,8 @@ DLI_EXPORT int dli_paged_prefill_tc(void* out, const void* q, long long q_stride
   p.out = (bf16*)out; p.q = (const bf16*)q; p.q_stride = q_stride;
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.q_start = q_start; p.kv_len = kv_len; p.seq0 = seq0;
   p.nh = nh; p.nkv = nkv; p.page_size = page_size; p.window = window;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = BENT_SCORES ? 1.f : scale * 1.4426950408889634f;
+  p.bend = make_score_bend(scale, softcap, slopes);
   p.sink_log2 = sink * 1.4426950408889634f;  // -inf (no sink) stays -inf
   p.sink_heads = sink_heads;
   const int G = nh / nkv;
@@ -961,7 +993,8 @@ struct DecodeParams {
   const int* kv_len;
   int seq0, nh, nkv, page_size, window, splits;
   int cluster_merge;  // the splits of a (sequence, head group) are one cluster and merge through shared memory
-  float scale_log2;
+  float scale_log2;   // as in Params
+  ScoreBend bend;     // as in Params
   float sink_log2;  // as in Params
   const float* sink_heads;  // as in Params
   float* part_acc;
@@ -1138,6 +1171,9 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   // Scores stay raw; the scale goes into the exponent's multiply-add.  Tiles that lie wholly inside the visible
   // range, all but the last and a window's first, skip the mask.
   constexpr float RESCALE_STEP = 8.f;
+#if BENT_SCORES
+  const float slope0 = r0 < nheads ? bend_slope(p.bend, head0 + r0) : 0.f, slope1 = r1 < nheads ? bend_slope(p.bend, head0 + r1) : 0.f;
+#endif
   bool ok = true;
   int st = 0, phase = 0;
   for (int i = 0; i < my_tiles; ++i) {
@@ -1158,6 +1194,13 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
         mma16816(sc[0], qf[kk], b[0], b[1]);
         mma16816(sc[1], qf[kk], b[2], b[3]);
       }
+#if BENT_SCORES
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          sc[j][e] = bent_score(sc[j][e], p.bend, ((e >> 1) ? slope1 : slope0) * (float)(base + j * 8 + (lane & 3) * 2 + (e & 1) - pos));
+#endif
       // ---- mask (only a tile that reaches beyond the visible keys) and online softmax
       if (base < lo || base + DN - 1 > pos) {
 #pragma unroll
@@ -1382,9 +1425,10 @@ int launch_decode(const CUtensorMap& map_k, const CUtensorMap& map_v, const Deco
 DLI_EXPORT int dli_paged_decode_tma(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long num_pages, const int* block_tables, int max_blocks, const int* q_start,
                                     const int* kv_len, int seq0, int num_seqs, int first_row, int nh, int nkv, int head_dim,
-                                    int page_size, int window, float scale, float sink, const float* sink_heads, int splits, float* part_acc, float* part_ml,
-                                    int max_kv_len, cudaStream_t stream) {
+                                    int page_size, int window, float scale, float sink, const float* sink_heads, float softcap, const float* slopes,
+                                    int splits, float* part_acc, float* part_ml, int max_kv_len, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
+  if (!BENT_SCORES && (softcap != 0.f || slopes)) return DLI_ERR_UNSUPPORTED;
   if (head_dim != 64 && head_dim != 128) return DLI_ERR_UNSUPPORTED;
   if (nkv < 1 || nh % nkv || splits < 1 || (splits > 1 && (!part_acc || !part_ml))) return DLI_ERR_UNSUPPORTED;
   if (page_size < 8 || (page_size % 8) || (page_size > 8 && (page_size % 16)) || page_size > 256) return DLI_ERR_UNSUPPORTED;
@@ -1403,7 +1447,8 @@ DLI_EXPORT int dli_paged_decode_tma(void* out, const void* q, long long q_stride
   p.out = (bf16*)out; p.q = (const bf16*)q; p.q_stride = q_stride;
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.q_start = q_start; p.kv_len = kv_len; p.seq0 = seq0;
   p.nh = nh; p.nkv = nkv; p.page_size = page_size; p.window = window; p.splits = splits;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = BENT_SCORES ? 1.f : scale * 1.4426950408889634f;
+  p.bend = make_score_bend(scale, softcap, slopes);
   p.sink_log2 = sink * 1.4426950408889634f;  // -inf (no sink) stays -inf
   p.sink_heads = sink_heads;
   p.part_acc = part_acc; p.part_ml = part_ml; p.error_flag = error_flag_device;

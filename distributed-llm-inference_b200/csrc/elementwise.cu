@@ -48,6 +48,60 @@ DLI_EXPORT int dli_embedding(float* h, const void* table, const int* ids, int n,
   return (int)cudaGetLastError();
 }
 
+// h[t] = table[ids[t]] * scale + the position's vector of sines (even places) and cosines (odd places).  A thread makes a pair of
+// places with one sincosf: the angle a is the rounded product position * frequency, e what that rounding and the frequency's
+// own left out, and sin(a + e) = sin a + e cos a, cos(a + e) = cos a - e sin a to float32.
+template <typename T, bool PAIRS>
+__global__ void sinusoid_embedding_kernel(float* __restrict__ h, const T* __restrict__ table, float scale, const float* __restrict__ freq,
+                                          const int* __restrict__ ids, const int* __restrict__ positions, int H) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, pairs = (H + 1) >> 1;
+  const T* src = table + (size_t)ids[t] * H;
+  float* dst = h + (size_t)t * H;
+  const float pos = (float)positions[t];
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < pairs; i += gridDim.y * blockDim.x) {
+    const float f = freq[i], a = pos * f;
+    const float e = fmaf(pos, f, -a) + pos * freq[pairs + i];
+    float sn, cs;
+    sincosf(a, &sn, &cs);
+    const float s0 = fmaf(e, cs, sn), c0 = fmaf(-e, sn, cs);
+    if (PAIRS) {
+      float x0, x1;
+      if constexpr (sizeof(T) == 2) {
+        const float2 x = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(src)[i]);
+        x0 = x.x; x1 = x.y;
+      } else {
+        const float2 x = reinterpret_cast<const float2*>(src)[i];
+        x0 = x.x; x1 = x.y;
+      }
+      reinterpret_cast<float2*>(dst)[i] = make_float2(fmaf(x0, scale, s0), fmaf(x1, scale, c0));
+    } else {
+      dst[2 * i] = fmaf(to_float(src[2 * i]), scale, s0);
+      if (2 * i + 1 < H) dst[2 * i + 1] = fmaf(to_float(src[2 * i + 1]), scale, c0);
+    }
+  }
+}
+
+DLI_EXPORT int dli_sinusoid_embedding(float* h, const void* table, float scale, const float* freq, const int* ids, const int* positions, int n, int H,
+                                      int dtype, cudaStream_t stream) {
+  if (n == 0) return 0;
+  const int pairs = (H + 1) / 2, threads = pairs >= 256 ? 256 : (pairs >= 128 ? 128 : 64);
+  // a decode step's few tokens are spread over several blocks each
+  const dim3 grid(n, n <= 64 ? (pairs + threads - 1) / threads : (pairs + 4 * threads - 1) / (4 * threads));
+  const bool even = (H % 2) == 0;
+#define DLI_SIN(T, P) launch_pdl((sinusoid_embedding_kernel<T, P>), grid, dim3(threads), 0, stream, 1, h, (const T*)table, scale, freq, ids, positions, H)
+  if (dtype == DLI_F32) {
+    if (even) DLI_SIN(float, true);
+    else DLI_SIN(float, false);
+  } else {
+    if (even) DLI_SIN(__nv_bfloat16, true);
+    else DLI_SIN(__nv_bfloat16, false);
+  }
+#undef DLI_SIN
+  return (int)cudaGetLastError();
+}
+
 // Token ids that were sampled on the device one step earlier and never travelled to the host:
 // ids[i] = source[src[i]] wherever src[i] >= 0.
 __global__ void patch_tokens_kernel(int* __restrict__ ids, const int* __restrict__ source, const int* __restrict__ src, int n) {

@@ -33,10 +33,11 @@ __device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* 
 // Groups: `groups` equal runs of neighbouring experts; a group's mark is the sum of its two largest choice scores (its
 // one score if it has one expert); only the `keep` groups with the largest marks stay eligible.  The `top` eligible experts
 // with the largest choice scores are chosen (ties: the lower index), in that order; weights = s[chosen] / (sum + 1e-20) * scale.
+// softmax != 0: choice = z + correction instead, and weights = softmax over the chosen experts' choices * scale.
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x,
                                                                   const float* __restrict__ router, const float* __restrict__ correction,
-                                                                  int W, int E, int top, int groups, int keep, float scale) {
+                                                                  int W, int E, int top, int groups, int keep, float scale, int softmax) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float sm[];  // x [W] | score [E] | choice [E] | mark [groups]
@@ -53,9 +54,9 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restric
   for (int e = warp; e < E; e += blockDim.x >> 5) {
     const float z = warp_dot<float>(router + (size_t)e * W, xs, W, lane, vec);
     if (lane == 0) {
-      const float s = 1.f / (1.f + expf(-z));
+      const float s = softmax ? z + correction[e] : 1.f / (1.f + expf(-z));
       score[e] = s;
-      choice[e] = s + correction[e];
+      choice[e] = softmax ? s : s + correction[e];
     }
   }
   __syncthreads();
@@ -92,7 +93,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restric
       if (mark[e / per] == CUDART_INF_F) choice[e] = -CUDART_INF_F;
     __syncwarp();
   }
-  float total = 0.f;
+  float total = 0.f, largest = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -CUDART_INF_F;
     int at = -1;
@@ -111,13 +112,18 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restric
       picked[k] = at;
       choice[at] = -CUDART_INF_F;
     }
-    total += score[at];
+    if (softmax) {  // the first one chosen has the largest logit
+      if (k == 0) largest = score[at];
+      total += expf(score[at] - largest);
+    } else {
+      total += score[at];
+    }
     __syncwarp();
   }
-  const float f = scale / (total + 1e-20f);
+  const float f = scale / (softmax ? total : total + 1e-20f);
   for (int k = lane; k < top; k += 32) {
     ids[t * top + k] = picked[k];
-    weights[t * top + k] = score[picked[k]] * f;
+    weights[t * top + k] = (softmax ? expf(score[picked[k]] - largest) : score[picked[k]]) * f;
   }
 }
 
@@ -193,7 +199,7 @@ inline cudaError_t allow_smem(K kernel, size_t smem, MaxPerDevice& set) {
 }  // namespace
 
 DLI_EXPORT int dli_moe_route(int* ids, float* weights, const void* x, const float* router, const float* correction, int n, int W, int E, int top,
-                             int groups, int keep, float scale, int dtype, cudaStream_t stream) {
+                             int groups, int keep, float scale, int softmax, int dtype, cudaStream_t stream) {
   if (n == 0) return 0;
   if (W < 1 || E < 1 || top < 1 || top > MAX_TOP || groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups))
     return DLI_ERR_UNSUPPORTED;
@@ -205,12 +211,12 @@ DLI_EXPORT int dli_moe_route(int* ids, float* weights, const void* x, const floa
     static MaxPerDevice set;
     if ((e = allow_smem(moe_route_kernel<float>, smem, set)) != cudaSuccess) return (int)e;
     e = launch_pdl((moe_route_kernel<float>), dim3(n), dim3(threads), smem, stream, 1, ids, weights, (const float*)x, router, correction, W, E,
-                   top, groups, keep, scale);
+                   top, groups, keep, scale, softmax);
   } else {
     static MaxPerDevice set;
     if ((e = allow_smem(moe_route_kernel<__nv_bfloat16>, smem, set)) != cudaSuccess) return (int)e;
     e = launch_pdl((moe_route_kernel<__nv_bfloat16>), dim3(n), dim3(threads), smem, stream, 1, ids, weights, (const __nv_bfloat16*)x, router,
-                   correction, W, E, top, groups, keep, scale);
+                   correction, W, E, top, groups, keep, scale, softmax);
   }
   return (int)e;
 }

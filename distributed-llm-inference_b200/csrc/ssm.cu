@@ -391,7 +391,8 @@ store_state:
 // norm, out = y / sqrt(mean(y^2) + eps) * w * silu(z).
 template <typename T>
 __global__ void gated_group_rmsnorm_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ u, long long u_stride,
-                                           int z_col, const float* __restrict__ w, int inner, int parts, float eps, int gate_after) {
+                                           int z_col, const float* __restrict__ w, const float* __restrict__ divisor, int inner, int parts, float eps,
+                                           int gate_after) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[33];
@@ -399,12 +400,13 @@ __global__ void gated_group_rmsnorm_kernel(T* __restrict__ out, const float* __r
   const int size = inner / parts, c0 = part * size;
   const float* yrow = y + (size_t)t * inner + c0;
   const T* zrow = u + (size_t)t * u_stride + z_col + c0;
+  const float f = divisor ? 1.f / divisor[(size_t)t * parts + part] : 1.f;  // every number of the part, before anything else
   float q = 0.f;
   for (int i = threadIdx.x; i < size; i += blockDim.x) {
-    const float gv = gate_after ? yrow[i] : yrow[i] * norm_gate(to_float(zrow[i]), gate_after);
+    const float gv = gate_after ? yrow[i] * f : yrow[i] * f * norm_gate(to_float(zrow[i]), gate_after);
     q = fmaf(gv, gv, q);
   }
-  const float r = 1.f / sqrtf(block_sum(q, red) / (float)size + eps);
+  const float r = f / sqrtf(block_sum(q, red) / (float)size + eps);
   for (int i = threadIdx.x; i < size; i += blockDim.x) {
     const float gate = norm_gate(to_float(zrow[i]), gate_after);
     out[(size_t)t * inner + c0 + i] = from_float<T>(gate_after ? yrow[i] * r * w[c0 + i] * gate : yrow[i] * gate * r * w[c0 + i]);
@@ -416,8 +418,8 @@ __global__ void gated_group_rmsnorm_kernel(T* __restrict__ out, const float* __r
 template <typename T, int THREADS, int CHUNKS>
 __global__ void __launch_bounds__(THREADS) gated_group_rmsnorm_vec_kernel(T* __restrict__ out, const float* __restrict__ y,
                                                                           const T* __restrict__ u, long long u_stride, int z_col,
-                                                                          const float* __restrict__ w, int inner, int parts, float eps,
-                                                                          int gate_after) {
+                                                                          const float* __restrict__ w, const float* __restrict__ divisor,
+                                                                          int inner, int parts, float eps, int gate_after) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[33];
@@ -425,6 +427,7 @@ __global__ void __launch_bounds__(THREADS) gated_group_rmsnorm_vec_kernel(T* __r
   const int size = inner / parts, c0 = part * size;
   const float* yrow = y + (size_t)t * inner + c0;
   const T* zrow = u + (size_t)t * u_stride + z_col + c0;
+  const float f = divisor ? 1.f / divisor[(size_t)t * parts + part] : 1.f;  // every number of the part, before anything else
   float gv[CHUNKS][8];
   float q = 0.f;
 #pragma unroll
@@ -434,6 +437,8 @@ __global__ void __launch_bounds__(THREADS) gated_group_rmsnorm_vec_kernel(T* __r
       float z[8];
       load8(yrow + col, gv[c]);
       load8(zrow + col, z);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) gv[c][k] *= f;
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const float gate = norm_gate(z[k], gate_after);
@@ -593,8 +598,8 @@ DLI_EXPORT int dli_ssm_scan(float* y, const void* xbc, const void* u, long long 
                                     q_start, state_slot, num_seqs, heads, P, N, groups, max_len, stream);
 }
 
-DLI_EXPORT int dli_gated_group_rmsnorm(void* out, const float* y, const void* u, long long u_stride, int z_col, const float* w, int n,
-                                       int inner, int parts, float eps, int gate_after, int dtype, cudaStream_t stream) {
+DLI_EXPORT int dli_gated_group_rmsnorm(void* out, const float* y, const void* u, long long u_stride, int z_col, const float* w,
+                                       const float* divisor, int n, int inner, int parts, float eps, int gate_after, int dtype, cudaStream_t stream) {
   if (n == 0) return 0;
   if (parts < 1 || parts > 65535 || inner % parts) return DLI_ERR_UNSUPPORTED;
   const int size = inner / parts;
@@ -604,7 +609,7 @@ DLI_EXPORT int dli_gated_group_rmsnorm(void* out, const float* y, const void* u,
       (((uintptr_t)out | (uintptr_t)y | (uintptr_t)u | (uintptr_t)w) & 15) == 0) {
 #define DLI_GN_VEC(T, THREADS, CHUNKS)                                                                                               \
   return (int)launch_pdl((gated_group_rmsnorm_vec_kernel<T, THREADS, CHUNKS>), grid, dim3(THREADS), 0, stream, 1, (T*)out, y, (const T*)u, \
-                         u_stride, z_col, w, inner, parts, eps, gate_after)
+                         u_stride, z_col, w, divisor, inner, parts, eps, gate_after)
 #define DLI_GN_SIZES(T)                       \
   if (size <= 256) DLI_GN_VEC(T, 32, 1);      \
   if (size <= 512) DLI_GN_VEC(T, 64, 1);      \
@@ -623,9 +628,9 @@ DLI_EXPORT int dli_gated_group_rmsnorm(void* out, const float* y, const void* u,
   const int threads = size >= 1024 ? 256 : 128;
   if (dtype == DLI_F32)
     e = launch_pdl((gated_group_rmsnorm_kernel<float>), grid, dim3(threads), 0, stream, 1, (float*)out, y, (const float*)u, u_stride, z_col, w,
-                   inner, parts, eps, gate_after);
+                   divisor, inner, parts, eps, gate_after);
   else
     e = launch_pdl((gated_group_rmsnorm_kernel<__nv_bfloat16>), grid, dim3(threads), 0, stream, 1, (__nv_bfloat16*)out, y,
-                   (const __nv_bfloat16*)u, u_stride, z_col, w, inner, parts, eps, gate_after);
+                   (const __nv_bfloat16*)u, u_stride, z_col, w, divisor, inner, parts, eps, gate_after);
   return (int)e;
 }

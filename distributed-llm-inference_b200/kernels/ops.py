@@ -72,6 +72,27 @@ def _sink_heads(sink, num_heads: int) -> c_void_p:
     return _ptr(sink)
 
 
+def _bend(softcap: float | None, slopes: torch.Tensor | None, num_heads: int) -> tuple[float, c_void_p]:
+    """The attention kernels' arguments for scores that are bent before the softmax: the soft cap (0: none) and the float32 slope
+    per query head that is taken off per key of distance (null: none)."""
+    if slopes is not None:
+        _need(slopes, "slopes", torch.float32)
+        if slopes.numel() != num_heads:
+            raise KernelError("slopes need one number for every query head")
+    return (float(softcap) if softcap else 0.0), _ptr(slopes)
+
+
+# Kernels whose scores pass through the soft cap and the distance penalty are libraries of their own (the plain ones do not carry
+# the instructions); the float32 kernel takes both as arguments.
+_BENT = {"BENT_SCORES": 1}
+
+
+def _bent_defines(softcap: float | None, slopes: torch.Tensor | None, more: dict | None = None) -> dict | None:
+    if softcap or slopes is not None:
+        return {**(more or {}), **_BENT}
+    return more
+
+
 def _need(t: torch.Tensor, name: str, dtype: torch.dtype | None = None) -> None:
     if not t.is_cuda:
         raise KernelError(f"{name} must be a CUDA tensor: the engine has no CPU path")
@@ -110,6 +131,18 @@ def embedding(h: torch.Tensor, table: torch.Tensor, ids: torch.Tensor) -> None:
         raise KernelError("embedding: shapes or dtype do not agree")
     f = _fn("elementwise.cu", "dli_embedding", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(h), _ptr(table), _ptr(ids), n, H, DT_CODE[table.dtype], _stream()), "embedding")
+
+
+def sinusoid_embedding(h: torch.Tensor, table: torch.Tensor, scale: float, freq: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor) -> None:
+    """h[t, c] = float32(table[ids[t], c]) * scale + (sin for even c, cos for odd c)(positions[t] * f[c // 2]); ``freq`` [2, pairs]
+    holds f as a float32 and the remainder that its rounding left out."""
+    _need(h, "h", torch.float32), _need(table, "table"), _need(freq, "freq", torch.float32), _need(ids, "ids", torch.int32)
+    _need(positions, "positions", torch.int32)
+    n, H = h.shape
+    if table.shape[1] != H or ids.numel() != n or positions.numel() != n or tuple(freq.shape) != (2, (H + 1) // 2) or table.dtype not in DT_CODE:
+        raise KernelError("sinusoid_embedding: shapes or dtype do not agree")
+    f = _fn("elementwise.cu", "dli_sinusoid_embedding", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(h), _ptr(table), float(scale), _ptr(freq), _ptr(ids), _ptr(positions), n, H, DT_CODE[table.dtype], _stream()), "sinusoid_embedding")
 
 
 def patch_tokens(ids: torch.Tensor, source: torch.Tensor, src: torch.Tensor) -> None:
@@ -303,8 +336,11 @@ def paged_attention_simt(
     scale: float,
     window: int | None = None,
     sink: float | torch.Tensor | None = None,
+    softcap: float | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> None:
-    """Causal attention of every token over its sequence's pages, on CUDA cores.  ``sink``: see ``_sink``.
+    """Causal attention of every token over its sequence's pages, on CUDA cores.  ``sink``: see ``_sink``.  ``softcap`` c: a score s
+    (after the scale) becomes c tanh(s / c); ``slopes``: then slopes[h] * (position - key position) is taken off.
 
     out [n, nh * d]; queries are the first nh * d columns of qkv; pools [pages, nkv, page_size, d];
     block_tables [seqs, max_blocks]; a token at position p reads keys max(0, p - window + 1) .. p.
@@ -320,11 +356,13 @@ def paged_attention_simt(
         raise KernelError(f"paged_attention_simt: head_dim {d} (<= {SIMT_MAX_HEAD_DIM}) / heads {num_heads} per kv head {nkv} not supported")
     f = _fn(
         "attention_simt.cu", "dli_paged_attention_simt",
-        [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6 + [c_float, c_float, c_void_p, c_int, c_void_p],
+        [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6
+        + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p],
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), block_tables.shape[1],
-          _ptr(seq_of_token), _ptr(positions), n, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads), DT_CODE[out.dtype], _stream()),
+          _ptr(seq_of_token), _ptr(positions), n, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
+          *_bend(softcap, slopes, num_heads), DT_CODE[out.dtype], _stream()),
         "paged_attention_simt",
     )
 
@@ -349,6 +387,8 @@ def paged_prefill_tc(
     window: int | None = None,
     query_tiles: int = 0,
     sink: float | torch.Tensor | None = None,
+    softcap: float | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> None:
     """bfloat16 attention for prompt portions on tcgen05 tensor cores with TMA-fed pages
     (head size 64 or 128; page sizes 8, 16, 32, 64, 128).  Arguments as paged_attention_mma.
@@ -366,13 +406,16 @@ def paged_prefill_tc(
         raise KernelError("paged_prefill_tc: sequence range outside the batch")
     f = _fn(
         "attention_tc.cu", "dli_paged_prefill_tc",
-        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_float, c_void_p, c_int, c_void_p],
+        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8
+        + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p],
+        _bent_defines(softcap, slopes),
     )
     if query_tiles not in (0, 1, 2):
         raise KernelError("paged_prefill_tc: query_tiles is 0 (choose), 1 or 2")
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), pages, _ptr(block_tables), block_tables.shape[1],
-          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, max_q_len, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads), query_tiles, _stream()),
+          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, max_q_len, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
+          *_bend(softcap, slopes, num_heads), query_tiles, _stream()),
         "paged_prefill_tc",
     )
 
@@ -399,6 +442,8 @@ def paged_decode_tma(
     scratch: tuple[torch.Tensor, torch.Tensor] | None = None,
     max_kv_len: int = 0,
     sink: float | torch.Tensor | None = None,
+    softcap: float | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> None:
     """bfloat16 attention of single-token sequences whose keys and values arrive by TMA (head size
     64 or 128; page sizes 8, 16, 32, ...).  Arguments as paged_attention_mma with max_q_len = 1.
@@ -426,16 +471,17 @@ def paged_decode_tma(
     f = _fn(
         "attention_tc.cu", "dli_paged_decode_tma",
         [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8
-        + [c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p],
+        + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p],
+        _bent_defines(softcap, slopes),
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), pages, _ptr(block_tables), block_tables.shape[1],
           _ptr(q_start), _ptr(kv_len), seq0, num_seqs, first_row, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
-          splits, _ptr(acc), _ptr(ml), int(max_kv_len), _stream()),
+          *_bend(softcap, slopes, num_heads), splits, _ptr(acc), _ptr(ml), int(max_kv_len), _stream()),
         "paged_decode_tma",
     )
     global launch_count
-    if splits > 1 and not _fn("attention_tc.cu", "dli_decode_tma_merges_in_cluster", [c_int, c_int, c_int])(num_heads, nkv, splits):
+    if splits > 1 and not _fn("attention_tc.cu", "dli_decode_tma_merges_in_cluster", [c_int, c_int, c_int], _bent_defines(softcap, slopes))(num_heads, nkv, splits):
         launch_count += 1  # the merge kernel; otherwise the splits merge inside the kernel, as one cluster
 
 
@@ -445,8 +491,9 @@ def paged_prefill_tc_error() -> int:
     return _fn("attention_tc.cu", "dli_paged_prefill_tc_error", [])()
 
 
-def _library_in_use(source: str) -> bool:
-    return any(key.startswith(source + ":") for key in _fns)
+def _library_in_use(source: str, defines: dict | None = None) -> bool:
+    tail = f":{sorted((defines or {}).items())}"
+    return any(key.startswith(source + ":") and key.endswith(tail) for key in _fns)
 
 
 def device_wait_errors(clear: bool = True) -> dict[str, int]:
@@ -455,16 +502,17 @@ def device_wait_errors(clear: bool = True) -> dict[str, int]:
     in mapped host memory, so reading them costs no copy; read them once the step's results have
     reached the host.  With ``clear`` a code that was read is forgotten."""
     found = {}
-    for source, read, forget in (("skinny_gemm.cu", "dli_skinny_gemm_error", "dli_skinny_gemm_clear_error"),
-                                 ("dense_gemm.cu", "dli_dense_gemm_error", "dli_dense_gemm_clear_error"),
-                                 ("attention_tc.cu", "dli_paged_prefill_tc_error", "dli_paged_prefill_tc_clear_error")):
-        if not _library_in_use(source):
+    for source, read, forget, defines in (("skinny_gemm.cu", "dli_skinny_gemm_error", "dli_skinny_gemm_clear_error", None),
+                                          ("dense_gemm.cu", "dli_dense_gemm_error", "dli_dense_gemm_clear_error", None),
+                                          ("attention_tc.cu", "dli_paged_prefill_tc_error", "dli_paged_prefill_tc_clear_error", None),
+                                          ("attention_tc.cu", "dli_paged_prefill_tc_error", "dli_paged_prefill_tc_clear_error", _BENT)):
+        if not _library_in_use(source, defines):
             continue
-        code = _fn(source, read, [])()
+        code = _fn(source, read, [], defines)()
         if code:
             found[source] = int(code)
             if clear:
-                _fn(source, forget, [])()
+                _fn(source, forget, [], defines)()
     return found
 
 
@@ -541,6 +589,8 @@ def paged_attention_mma(
     splits: int = 1,
     scratch: tuple[torch.Tensor, torch.Tensor] | None = None,
     sink: float | torch.Tensor | None = None,
+    softcap: float | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> None:
     """bfloat16 tensor-core attention for the sequences [seq0, seq0 + num_seqs) of a batch.
 
@@ -572,13 +622,13 @@ def paged_attention_mma(
     f = _fn(
         "attention_mma.cu", "dli_paged_attention_mma",
         [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]
-        + [c_int] * 8 + [c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
-        {"HEAD_DIM": d},
+        + [c_int] * 8 + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
+        _bent_defines(softcap, slopes, {"HEAD_DIM": d}),
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), block_tables.shape[1],
           _ptr(q_start), _ptr(kv_len), seq0, num_seqs, max_q_len, first_row, num_heads, nkv, page_size, int(window or 0),
-          scale, _sink(sink), _sink_heads(sink, num_heads), splits, _ptr(acc), _ptr(ml), _stream()),
+          scale, _sink(sink), _sink_heads(sink, num_heads), *_bend(softcap, slopes, num_heads), splits, _ptr(acc), _ptr(ml), _stream()),
         "paged_attention_mma",
     )
     global launch_count
@@ -996,6 +1046,49 @@ def qk_norm_rotary_store(proj: torch.Tensor, wq: torch.Tensor | None, wk: torch.
     return q
 
 
+def qk_norm_mix_store(q_out: torch.Tensor, qkv: torch.Tensor, bias: torch.Tensor | None, wq: torch.Tensor | None, wk: torch.Tensor | None, eps: float | None,
+                      positions: torch.Tensor, temp: tuple[float, float], source: torch.Tensor | None, lam: float | None, slots: torch.Tensor | None,
+                      k_pool: torch.Tensor | None, v_pool: torch.Tensor | None, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
+                      page_size: int) -> None:
+    """What lies between the q | k | v product and the attention kernel of a layer without rotation.  qkv [n, nh d + nkv d + nkv dv]
+    (float32 sums or the activation dtype) plus ``bias`` (float32, or None).  q and k are each divided by the RMS of their whole
+    part and multiplied by wq, wk (``eps`` None: not); q also by 1 + temp[0] ln(floor((p + 1) / temp[1]) + 1) at position p.
+    ``source`` [n, nkv dv] float32: with ``lam`` None this layer's values are left there; else the values become
+    (1 - lam) v + lam source.  Rows of D = the pools' row size (or q_out's) leave, padded with zeros: q -> q_out [n, nh D],
+    k -> k_pool, v -> v_pool [pages, nkv, page_size, D] at ``slots`` (None: not written)."""
+    _need(q_out, "q_out"), _need(qkv, "qkv"), _need(positions, "positions", torch.int32)
+    n = qkv.shape[0]
+    nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * value_dim
+    D = q_out.shape[1] // num_heads
+    if (q_out.dtype not in DT_CODE or qkv.dtype not in (q_out.dtype, torch.float32) or tuple(qkv.shape) != (n, nq + nk + nv) or positions.numel() != n
+            or tuple(q_out.shape) != (n, num_heads * D) or D < max(head_dim, value_dim) or num_heads % num_kv_heads):
+        raise KernelError("qk_norm_mix_store: shapes or dtype do not agree")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != nq + nk + nv:
+            raise KernelError("qk_norm_mix_store: one bias per column of the product")
+    if eps is not None:
+        _need(wq, "wq", torch.float32), _need(wk, "wk", torch.float32)
+        if wq.numel() != nq or wk.numel() != nk:
+            raise KernelError("qk_norm_mix_store: one weight per column of q and of k")
+    if source is not None:
+        _need(source, "source", torch.float32)
+        if tuple(source.shape) != (n, nv):
+            raise KernelError("qk_norm_mix_store: the source must be [n, kv_heads * value_dim]")
+    elif lam is not None:
+        raise KernelError("qk_norm_mix_store: mixing needs the source's values")
+    if slots is not None:
+        _need(slots, "slots", torch.int32), _need(k_pool, "k_pool", q_out.dtype), _need(v_pool, "v_pool", q_out.dtype)
+        if tuple(k_pool.shape[1:]) != (num_kv_heads, page_size, D) or k_pool.shape != v_pool.shape or slots.numel() != n:
+            raise KernelError("qk_norm_mix_store: pool layout must be [pages, kv_heads, page_size, row]")
+    f = _fn("attention_prep.cu", "dli_qk_norm_mix_store", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float, c_float, c_void_p,
+                                                          c_float, c_void_p, c_void_p, c_void_p] + [c_int] * 11 + [c_void_p])
+    _check(f(_ptr(q_out), _ptr(qkv), _ptr(bias), _ptr(wq), _ptr(wk), -1.0 if eps is None else float(eps), _ptr(positions), float(temp[0]), float(temp[1]),
+             _ptr(source), 0.0 if lam is None else float(lam), _ptr(slots), _ptr(k_pool), _ptr(v_pool), n, num_heads, num_kv_heads, head_dim, value_dim, D,
+             page_size, 0 if source is None else (1 if lam is None else 2), int(eps is not None), DT_CODE[qkv.dtype], DT_CODE[q_out.dtype], _stream()),
+           "qk_norm_mix_store")
+
+
 def sigmoid_gate(out: torch.Tensor, gate: torch.Tensor) -> None:
     """out *= sigmoid(gate), element by element; ``gate`` [n, cols] may be a column slice of a wider matrix."""
     _need(out, "out")
@@ -1165,20 +1258,25 @@ def ssm_scan(y: torch.Tensor, xbc: torch.Tensor, u: torch.Tensor, dt_col: int, d
 
 
 def gated_group_rmsnorm(out: torch.Tensor, y: torch.Tensor, u: torch.Tensor, z_col: int, weight: torch.Tensor, parts: int, eps: float,
-                        gate_after: bool = False, gate: str = "silu") -> None:
+                        gate_after: bool = False, gate: str = "silu", divisor: torch.Tensor | None = None) -> None:
     """out = g / sqrt(mean(g^2) + eps) * weight with g = y * silu(z), the mean taken over each of ``parts`` equal runs
     of the row; z is columns z_col .. of u; y float32.  ``gate_after``: the gate stays out of the norm,
     out = y / sqrt(mean(y^2) + eps) * weight * silu(z); with ``gate`` = ``"sigmoid"`` (only behind the norm) the gate is
-    the logistic function of z instead of SiLU."""
+    the logistic function of z instead of SiLU.  ``divisor`` [n, parts] float32 (or None): every run of y is divided by its
+    number first."""
     if gate not in ("silu", "sigmoid") or (gate == "sigmoid" and not gate_after):
         raise KernelError("gated_group_rmsnorm: gate is silu, or sigmoid behind the norm")
     _columns(u, "gated_group_rmsnorm"), _need(out, "out", u.dtype), _need(y, "y", torch.float32), _need(weight, "weight", torch.float32)
     n, inner = y.shape
     if tuple(out.shape) != (n, inner) or u.shape[0] != n or z_col + inner > u.shape[1] or weight.numel() != inner or inner % parts:
         raise KernelError("gated_group_rmsnorm: shapes do not agree")
-    f = _fn("ssm.cu", "dli_gated_group_rmsnorm", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p])
+    if divisor is not None:
+        _need(divisor, "divisor", torch.float32)
+        if tuple(divisor.shape) != (n, parts):
+            raise KernelError("gated_group_rmsnorm: one divisor per run of the row")
+    f = _fn("ssm.cu", "dli_gated_group_rmsnorm", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p])
     mode = 2 if gate == "sigmoid" else int(gate_after)
-    _check(f(_ptr(out), _ptr(y), _ptr(u), u.stride(0), z_col, _ptr(weight), n, inner, parts, eps, mode, DT_CODE[u.dtype], _stream()),
+    _check(f(_ptr(out), _ptr(y), _ptr(u), u.stride(0), z_col, _ptr(weight), _ptr(divisor), n, inner, parts, eps, mode, DT_CODE[u.dtype], _stream()),
            "gated_group_rmsnorm")
 
 
@@ -1561,6 +1659,56 @@ def decay_recurrence(o: torch.Tensor, rows: torch.Tensor, state: torch.Tensor, q
              0 if mode == "bonus" else 1, int(rows_per_lane), _stream()), "decay_recurrence")
 
 
+# ------------------------------------------------------------------ matrix memory with exponential gates
+
+MATRIX_MEMORY_MAX_HEAD_DIM = 512
+MATRIX_MEMORY_CHUNK_MAX_HEAD_DIM = 256  # the tensor-core kernel keeps a state column block in registers
+MATRIX_MEMORY_CHUNK_MIN_TOKENS = 17  # shorter portions are walked token after token
+
+
+def matrix_memory_form(dtype: torch.dtype, d: int, max_len: int) -> str:
+    """Which kernel serves a step: ``"chunk"`` (bfloat16 portions, tiles of tokens on the tensor cores) or ``"walk"`` (token after
+    token on the CUDA cores: decode steps, float32, larger heads)."""
+    if dtype == torch.bfloat16 and d <= MATRIX_MEMORY_CHUNK_MAX_HEAD_DIM and max_len >= MATRIX_MEMORY_CHUNK_MIN_TOKENS:
+        return "chunk"
+    return "walk"
+
+
+def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: float,
+                       state: torch.Tensor, top: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, max_len: int = 1 << 30,
+                       form: str | None = None) -> None:
+    """A matrix memory with exponential gates over every sequence's tokens of this step, from and to its slot of ``state``
+    [slots, heads, dv + 1, d] (float32; S transposed, the last row is n) and ``top`` [slots, heads, dv + 1] (m, a copy per column).
+    u [n, .]: q | k | v in its leading columns (heads of d, d, dv); gates [n, 2 heads] float32: the input gates' sums, then the
+    forget gates'; ``gate_bias`` [2 heads].  Per head i = cap tanh((gate + bias) / cap), f = logsigmoid(cap tanh(...)),
+    m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone.  Left: o [n, heads dv] = S^T q / sqrt(d)
+    and divisor [n, heads] = max(|n . q| / sqrt(d), exp(-m)) + 1e-6, both float32.  ``form``: ``"walk"``, ``"chunk"``, or None (chosen)."""
+    _columns(u, "matrix_memory_scan"), _need(o, "o", torch.float32), _need(divisor, "divisor", torch.float32)
+    _need(gates, "gates", torch.float32), _need(gate_bias, "gate_bias", torch.float32)
+    _need(state, "state", torch.float32), _need(top, "top", torch.float32)
+    _need(q_start, "q_start", torch.int32), _need(state_slot, "state_slot", torch.int32)
+    _, heads, dv1, d = state.shape
+    dv, n = dv1 - 1, u.shape[0]
+    if (tuple(o.shape) != (n, heads * dv) or tuple(divisor.shape) != (n, heads) or u.shape[1] < heads * (2 * d + dv) or tuple(gates.shape) != (n, 2 * heads)
+            or gate_bias.numel() != 2 * heads or tuple(top.shape) != tuple(state.shape[:3]) or d > MATRIX_MEMORY_MAX_HEAD_DIM
+            or q_start.numel() != state_slot.numel() + 1 or not cap > 0):
+        raise KernelError(f"matrix_memory_scan: shapes do not agree (or the head size is above {MATRIX_MEMORY_MAX_HEAD_DIM})")
+    form = form or matrix_memory_form(u.dtype, d, max_len)
+    args = (_ptr(o), _ptr(divisor), _ptr(u), u.stride(0), _ptr(gates), _ptr(gate_bias), float(cap), _ptr(state), _ptr(top), _ptr(q_start), _ptr(state_slot),
+            state_slot.numel(), heads, d, dv, int(max_len))
+    types = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 5
+    if form == "chunk":
+        if u.dtype != torch.bfloat16 or d > MATRIX_MEMORY_CHUNK_MAX_HEAD_DIM:
+            raise KernelError("matrix_memory_scan: the tensor-core form takes bfloat16 heads of at most 256")
+        f = _fn("matrix_memory_tc.cu", "dli_matrix_memory_chunk", types + [c_void_p], {"KEY_DIM": -(-d // 16) * 16})
+        _check(f(*args, _stream()), "matrix_memory_scan")
+    elif form == "walk":
+        f = _fn("matrix_memory.cu", "dli_matrix_memory_walk", types + [c_int, c_void_p])
+        _check(f(*args, DT_CODE[u.dtype], _stream()), "matrix_memory_scan")
+    else:
+        raise KernelError("matrix_memory_scan: form is walk or chunk")
+
+
 # ------------------------------------------------------------------ routed mixture of gated feed-forwards
 
 MOE_MAX_TOP = 32
@@ -1575,21 +1723,25 @@ def moe_grouped_supported(tokens: int, W: int, ff: int, dtype: torch.dtype) -> b
 MOE_PAIR_CHUNK = 8192  # tokens a launch of the pair kernels takes (their grids count (token, expert) pairs along y)
 
 
+MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1}
+
+
 def moe_route(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, group_count: int,
-              group_keep: int, scale: float) -> None:
+              group_keep: int, scale: float, score: str = "sigmoid") -> None:
     """Which experts every token uses, and with what weights.  z = x router^T (float32), s = sigmoid(z), choice = s + correction.
     With ``group_count`` > 1 the experts form equal groups of neighbours, a group's mark is the sum of its two largest choice scores,
     and only experts of the ``group_keep`` best groups are eligible.  ids [n, top] int32: the eligible experts with the largest choice
-    scores, best first (ties: the lower index); weights [n, top] float32 = s[ids] / (their sum + 1e-20) * scale."""
+    scores, best first (ties: the lower index); weights [n, top] float32 = s[ids] / (their sum + 1e-20) * scale.
+    ``score`` = ``"softmax_chosen"``: choice = z + correction, and the weights are softmax(choice[ids]) * scale."""
     _need(ids, "ids", torch.int32), _need(weights, "weights", torch.float32), _need(x, "x"), _need(router, "router", torch.float32)
     _need(correction, "correction", torch.float32)
     n, W = x.shape
     E, top = router.shape[0], ids.shape[1]
     if (x.dtype not in DT_CODE or router.shape[1] != W or correction.numel() != E or tuple(ids.shape) != (n, top) or tuple(weights.shape) != (n, top)
-            or top > MOE_MAX_TOP or group_count < 1 or E % group_count or not 1 <= group_keep <= group_count or top > group_keep * (E // group_count)):
+            or top > MOE_MAX_TOP or group_count < 1 or E % group_count or not 1 <= group_keep <= group_count or top > group_keep * (E // group_count) or score not in MOE_SCORES):
         raise KernelError("moe_route: shapes, dtype or groups do not agree")
-    f = _fn("moe.cu", "dli_moe_route", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 6 + [c_float, c_int, c_void_p])
-    _check(f(_ptr(ids), _ptr(weights), _ptr(x), _ptr(router), _ptr(correction), n, W, E, top, group_count, group_keep, float(scale), DT_CODE[x.dtype],
+    f = _fn("moe.cu", "dli_moe_route", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 6 + [c_float, c_int, c_int, c_void_p])
+    _check(f(_ptr(ids), _ptr(weights), _ptr(x), _ptr(router), _ptr(correction), n, W, E, top, group_count, group_keep, float(scale), MOE_SCORES[score], DT_CODE[x.dtype],
              _stream()), "moe_route")
 
 

@@ -10,7 +10,7 @@ from ..cache.needs import PagedKVNeed
 from ..kernels import attention as attn_kernels
 from ..kernels import ops
 from ..cache.needs import StateNeed
-from ..kernels.gemm import heads_product, last_product, project, project_bias
+from ..kernels.gemm import decode_product, heads_product, last_product, project, project_bias
 from ..weights.loader import TensorDecl
 from .base import Part, build_part, register_part, tensor_name
 
@@ -234,12 +234,7 @@ class ConvAttention(Part):
         nm = self.names
         self.w_in = torch.cat([tensors[nm[r]] for r in ("q", "k", "v")], 0).contiguous()
         self.w_conv = torch.cat([tensors[nm[r + "_conv"]] for r in ("q", "k", "v")], 0).t().contiguous()  # [taps, channels]
-        wo = tensors[nm["o"]]
-        if self.row != self.dv:  # the attention kernels leave rows of ``row`` numbers per head: zero columns where the padding lies
-            padded = torch.zeros((self.hidden, self.nh, self.row), dtype=wo.dtype, device=wo.device)
-            padded[:, :, : self.dv] = wo.view(self.hidden, self.nh, self.dv)
-            wo = padded.view(self.hidden, self.nh * self.row)
-        self.wo = wo.contiguous()
+        self.wo = zero_padded_heads(tensors[nm["o"]], self.nh, self.dv, self.row)
         if self.bias:
             self.b_in = torch.cat([tensors[nm[r + "_bias"]] for r in ("q", "k", "v")], 0).contiguous()
             self.bo = tensors[nm["o_bias"]]
@@ -265,6 +260,135 @@ class ConvAttention(Part):
         out = torch.empty((n, self.nh * self.row), dtype=x.dtype, device=x.device)
         attn_kernels.paged_attention(out, q, cache, batch, self.nh, self.scale, self.window, splits=batch.launch_keys.get(id(self)))
         return project_bias(out, self.wo, self.bo)
+
+
+def zero_padded_heads(wo: torch.Tensor, heads: int, dv: int, row: int) -> torch.Tensor:
+    """An output projection [H, heads * dv] for attention outputs that come in rows of ``row`` >= dv numbers a head: zero
+    columns where the padding lies."""
+    if row == dv:
+        return wo.contiguous()
+    padded = torch.zeros((wo.shape[0], heads, row), dtype=wo.dtype, device=wo.device)
+    padded[:, :, :dv] = wo.view(wo.shape[0], heads, dv)
+    return padded.view(wo.shape[0], heads * row)
+
+
+@register_part("mixer", "capped_attention")
+class CappedAttention(Part):
+    """Causal grouped-query softmax attention without rotation, whose scores are bent before the softmax, with options other
+    designs can switch:
+
+    * ``bias``: q, k and v have biases, added in the projection;
+    * ``qk_norm_eps`` (or None): q and k are each divided by the RMS of their whole projection (all heads together) and
+      multiplied by a weight of that size;
+    * ``temp_coef`` / ``temp_every``: the (normed) queries of position p are multiplied by
+      1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (0: none);
+    * ``softcap`` (or None): scores s = scale (q . k) become softcap * tanh(s / softcap);
+    * ``slopes`` (or None): then slope_h * (i - j) is taken off the score of query position i and key position j, a slope per head;
+    * ``head_sinks``: a learned score per head (tensor ``sink``) whose exponential joins every softmax denominator and carries no
+      value; it is neither scaled nor capped and has no distance;
+    * ``window``: position i sees j with 0 <= i - j < window;
+    * ``value_mix``: ``"source"`` — this layer's values are kept for the layers behind it; ``"mix"`` — its values become
+      (1 - lambda) v + lambda v_source, lambda a learned number (tensor ``vmix``), v_source the source layer's values of the same
+      token, and that is what is cached; None — neither;
+    * ``value_dim``: the values' size may differ from the keys'.  Pages hold rows of max(head_dim, value_dim) numbers (rounded up to a
+      multiple of 16 in bfloat16, for the tensor-core kernels), padded with zeros; the output projection's matrix is padded with
+      zero columns to match, once, at load.
+
+    One product yields q | k | v; one kernel adds the biases (for a decode step's few tokens, whose product leaves float32 sums),
+    norms, applies the temperature, mixes the values and writes the pages.
+    params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window, bias, qk_norm_eps, temp_coef, temp_every,
+    softcap, slopes, head_sinks, value_mix, tensors (names of q, k, v, o, q_bias, k_bias, v_bias, q_norm, k_norm, sink, vmix)."""
+
+    graph_capturable = True
+
+    def __init__(self, spec, env) -> None:
+        super().__init__(spec, env)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.nh, self.nkv, self.d = int(p["num_heads"]), int(p["num_kv_heads"]), int(p["head_dim"])
+        self.dv = int(p.get("value_dim") or self.d)
+        self.row = max(self.d, self.dv)  # what a page keeps per token and KV head, for keys and for values
+        if env.dtype == torch.bfloat16:
+            self.row = -(-self.row // 16) * 16
+        self.scale, self.window = float(p["scale"]), p.get("window")
+        self.bias = bool(p.get("bias", False))
+        self.eps = None if p.get("qk_norm_eps") is None else float(p["qk_norm_eps"])
+        self.temp = (float(p.get("temp_coef") or 0.0), float(p.get("temp_every") or 1.0))
+        self.softcap = None if p.get("softcap") is None else float(p["softcap"])
+        self.slopes = None if p.get("slopes") is None else torch.tensor(p["slopes"], dtype=torch.float64).to(torch.float32).to(env.device)
+        self.head_sinks = bool(p.get("head_sinks", False))
+        self.value_mix = p.get("value_mix")
+        if self.nh % self.nkv or (self.slopes is not None and self.slopes.numel() != self.nh) or self.value_mix not in (None, "source", "mix"):
+            raise ValueError("capped_attention: num_heads must be a multiple of num_kv_heads, slopes one per head, value_mix source, mix or absent")
+        defaults = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "q_bias": "q_proj.bias",
+                    "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks",
+                    "vmix": "value_mix"}
+        self.names = {role: tensor_name(spec, role, default) for role, default in defaults.items()}
+        self.sizes = {"q": self.nh * self.d, "k": self.nkv * self.d, "v": self.nkv * self.dv}
+        self.w_in = self.b_in = self.b_in32 = self.wo = self.wq_norm = self.wk_norm = self.sinks = None
+        self.lam = 0.0
+
+    def declare(self):
+        nm, H = self.names, self.hidden
+        out = {nm["o"]: TensorDecl((H, self.nh * self.dv))}
+        for role, size in self.sizes.items():
+            out[nm[role]] = TensorDecl((size, H))
+            if self.bias:
+                out[nm[role + "_bias"]] = TensorDecl((size,), "vector32")
+        if self.eps is not None:
+            out[nm["q_norm"]] = TensorDecl((self.sizes["q"],), "vector32")
+            out[nm["k_norm"]] = TensorDecl((self.sizes["k"],), "vector32")
+        if self.head_sinks:
+            out[nm["sink"]] = TensorDecl((self.nh,), "vector32")
+        # the source's own lambda mixes nothing; a checkpoint may hold one
+        out[nm["vmix"]] = TensorDecl((), "vector32", unused=self.value_mix != "mix")
+        return out
+
+    def load(self, tensors):
+        nm = self.names
+        self.w_in = torch.cat([tensors[nm[r]] for r in ("q", "k", "v")], 0).contiguous()
+        self.wo = zero_padded_heads(tensors[nm["o"]], self.nh, self.dv, self.row)
+        if self.bias:
+            self.b_in32 = torch.cat([tensors[nm[r + "_bias"]] for r in ("q", "k", "v")], 0).contiguous()
+            self.b_in = self.b_in32.to(self.env.dtype)
+        if self.eps is not None:
+            self.wq_norm, self.wk_norm = tensors[nm["q_norm"]], tensors[nm["k_norm"]]
+        if self.head_sinks:
+            self.sinks = tensors[nm["sink"]]
+        if self.value_mix == "mix":
+            self.lam = float(tensors[nm["vmix"]].item())
+
+    def cache_need(self):
+        return PagedKVNeed(self.nkv, self.row, self.window)
+
+    def decode_launch_key(self, num_seqs: int, max_kv_len: int, page_size: int):
+        seen = min(max_kv_len, self.window + 64) if self.window else max_kv_len
+        return attn_kernels.decode_splits(num_seqs, self.nh, self.nkv, self.row, page_size, seen)
+
+    def forward(self, x: torch.Tensor, batch, cache) -> torch.Tensor:
+        n = x.shape[0]
+        if decode_product(x):  # few tokens: the product's float32 sums as they are, the bias joins them in the next kernel
+            qkv, bias = project(x, self.w_in, out_dtype=torch.float32), self.b_in32
+        else:
+            qkv, bias = project_bias(x, self.w_in, self.b_in), None
+        group = batch.group(cache.group)
+        q = torch.empty((n, self.nh * self.row), dtype=x.dtype, device=x.device)
+        mixed = self.value_mix == "mix"
+        source = None
+        if self.value_mix == "source":
+            source = batch.scratch["value_source"] = torch.empty((n, self.sizes["v"]), dtype=torch.float32, device=x.device)
+        elif mixed:
+            source = batch.scratch["value_source"]
+        ops.qk_norm_mix_store(q, qkv, bias, self.wq_norm, self.wk_norm, self.eps, batch.positions, self.temp, source, self.lam if mixed else None,
+                              group.slots if cache.writes else None, cache.k if cache.writes else None, cache.v if cache.writes else None,
+                              self.nh, self.nkv, self.d, self.dv, cache.page_size)
+        out = torch.empty((n, self.nh * self.row), dtype=x.dtype, device=x.device)
+        splits = batch.launch_keys.get(id(self))
+        if splits is None and batch.num_single:
+            splits = self.decode_launch_key(batch.num_single, batch.max_kv_len_single, cache.page_size)
+        attn_kernels.paged_attention(out, q, cache, batch, self.nh, self.scale, self.window, splits=splits, sink=self.sinks, softcap=self.softcap,
+                                     slopes=self.slopes)
+        return project(out, self.wo)
 
 
 @register_part("mixer", "latent_attention")

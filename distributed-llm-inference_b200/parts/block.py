@@ -134,9 +134,9 @@ class SandwichBlock(Part):
 
 @register_part("arrangement", "parallel")
 class ParallelBlock(Part):
-    """x = x + (mixer(norm_a(x)) + ffn(norm_f(x))): both branches read the same x, each behind a norm of its own, and
-    their outputs are added to the stream together.  Roles: mixer_norm, mixer, and — a layer may have no
-    feed-forward — ffn_norm, ffn.  The two outputs stay pending on the stream as a ``PendingSum``; the norm in front
+    """x = x + (mixer(norm_a(x)) + ffn(norm_f(x))): both branches read the same x, each behind a norm of its own — or, without
+    the role ffn_norm, both behind the one norm — and their outputs are added to the stream together.  Roles: mixer_norm,
+    mixer, and — a layer may have no feed-forward — ffn, ffn_norm.  The two outputs stay pending on the stream as a ``PendingSum``; the norm in front
     of the next layer's branches adds them, and where both norms divide by the same root mean square
     (``add_norm_pair``) one kernel adds the pending outputs and writes both branches' inputs."""
 
@@ -147,17 +147,25 @@ class ParallelBlock(Part):
         self.mixer_norm = build_part("norm", spec.parts["mixer_norm"], env)
         self.mixer = build_part("mixer", spec.parts["mixer"], env)
         self.has_ffn = "ffn" in spec.parts
+        self.own_ffn_norm = "ffn_norm" in spec.parts
         if self.has_ffn:
-            self.ffn_norm = build_part("norm", spec.parts["ffn_norm"], env)
+            self.ffn_norm = build_part("norm", spec.parts["ffn_norm"], env) if self.own_ffn_norm else self.mixer_norm
             self.ffn = build_part("feed_forward", spec.parts["ffn"], env)
 
     def children(self):
-        return [self.mixer_norm, self.mixer] + ([self.ffn_norm, self.ffn] if self.has_ffn else [])
+        own = [self.ffn_norm] if self.has_ffn and self.own_ffn_norm else []
+        return [self.mixer_norm, self.mixer] + (own + [self.ffn] if self.has_ffn else [])
 
     def cache_need(self):
         return self.mixer.cache_need()
 
     def forward(self, stream: ResidualStream, batch, cache) -> None:
+        if self.has_ffn and not self.own_ffn_norm:  # one norm, one kernel: it adds what the layer before left pending
+            y = normed_input(self.mixer_norm, stream.h, stream.take_pending(), None)
+            stream.pending = None
+            a = self.mixer.forward(y, batch, cache)
+            stream.pending = PendingSum(a, self.ffn.forward(y))
+            return
         pair = getattr(self.mixer_norm, "add_norm_pair", None) if self.has_ffn else None
         if pair is not None and not isinstance(stream.take_pending(), (PendingSum, torch.Tensor, type(None))):
             stream.settle()

@@ -106,11 +106,16 @@ class DenseActMLP(Part):
 class RoutedGLU(Part):
     """A mixture of ``num_experts`` small gated feed-forwards down_e(act(gate_e(x)) * up_e(x)), of which each token uses ``top``.
 
-    The router's logits z = W_r x and everything that follows them are float32.  Scores are sigmoid(z) (``score``:
-    ``"sigmoid"``).  The experts are CHOSEN by score + correction (a learned number per expert that steers the choice and
-    nothing else); they are WEIGHTED by their scores without it, divided by their sum (+ 1e-20) and multiplied by ``route_scale``.
+    The router's logits z = W_r x and everything that follows them are float32.  ``score``:
+
+    * ``"sigmoid"``: scores are sigmoid(z).  The experts are CHOSEN by score + correction (a learned number per expert that steers
+      the choice and nothing else); they are WEIGHTED by their scores without it, divided by their sum (+ 1e-20) and multiplied
+      by ``route_scale``;
+    * ``"softmax_chosen"``: the tensor ``correction`` is a bias of the logits, z = W_r x + b.  The experts with the largest logits
+      are chosen, their weights are the softmax over the chosen experts' logits alone, times ``route_scale``.
+
     With ``group_count`` > 1 the experts form that many equal groups of neighbours; a group's mark is the sum of its two
-    largest choice scores, and only experts of the ``group_keep`` best groups can be chosen.  The output is the weighted
+    largest choice scores (or logits), and only experts of the ``group_keep`` best groups can be chosen.  The output is the weighted
     sum of the chosen experts' outputs, added up in float32 in the order of the choice.
 
     One kernel routes; the tokens of every expert are then gathered by a counting sort on the device (no shape depends on
@@ -129,8 +134,9 @@ class RoutedGLU(Part):
         self.route_scale = float(p.get("route_scale", 1.0))
         self.group_count, self.group_keep = int(p.get("group_count") or 1), int(p.get("group_keep") or 1)
         self.activation = p.get("activation", "silu")
-        if p.get("score", "sigmoid") != "sigmoid":
-            raise ValueError(f"routed_glu: score={p['score']!r} (known: sigmoid)")
+        self.score = p.get("score", "sigmoid")
+        if self.score not in ops.MOE_SCORES:
+            raise ValueError(f"routed_glu: score={self.score!r} (known: {', '.join(ops.MOE_SCORES)})")
         if self.activation not in ops.GLU_ACTIVATIONS:
             raise ValueError(f"activation {self.activation!r} is not supported (known: {sorted(ops.GLU_ACTIVATIONS)})")
         per = self.experts // self.group_count
@@ -161,7 +167,7 @@ class RoutedGLU(Part):
         n = x.shape[0]
         ids = torch.empty((n, self.top), dtype=torch.int32, device=x.device)
         weights = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
-        ops.moe_route(ids, weights, x, self.w_router, self.correction, self.group_count, self.group_keep, self.route_scale)
+        ops.moe_route(ids, weights, x, self.w_router, self.correction, self.group_count, self.group_keep, self.route_scale, self.score)
         out = torch.empty((n, self.hidden), dtype=x.dtype, device=x.device)
         ops.moe_experts(out, x, ids, weights, self.w_gate_up, self.w_down, self.activation)
         return out

@@ -35,6 +35,38 @@ class TokenEmbedding(Part):
         return h
 
 
+@register_part("embedding", "sinusoid_embedding")
+class SinusoidEmbedding(Part):
+    """h = table[token] * scale + s(position): a fixed vector of sines (even places) and cosines (odd places) of the token's
+    position is added, the places 2i and 2i + 1 sharing the frequency position_base^(-2i / hidden_size).  The frequencies are
+    made on the host in float64 and kept as a float32 and its remainder, so that the angles of far positions keep float32's
+    precision.  params: vocab_size, hidden_size, tensor, scale, position_base."""
+
+    graph_capturable = True
+
+    def __init__(self, spec, env) -> None:
+        super().__init__(spec, env)
+        p = spec.params
+        self.vocab, self.hidden = int(p["vocab_size"]), int(p["hidden_size"])
+        self.scale, base = float(p.get("scale", 1.0)), float(p["position_base"])
+        self.name = tensor_name(spec, "weight", "weight")
+        freq = torch.tensor([base ** (-2.0 * i / self.hidden) for i in range((self.hidden + 1) // 2)], dtype=torch.float64)
+        head = freq.to(torch.float32)
+        self.freq = torch.stack([head, (freq - head.double()).to(torch.float32)]).contiguous().to(env.device)  # [2, pairs]
+        self.weight: torch.Tensor | None = None
+
+    def declare(self):
+        return {self.name: TensorDecl((self.vocab, self.hidden))}
+
+    def load(self, tensors):
+        self.weight = tensors[self.name]
+
+    def forward_step(self, batch, cache) -> ResidualStream:
+        h = torch.empty((batch.token_ids.numel(), self.hidden), dtype=torch.float32, device=batch.token_ids.device)
+        ops.sinusoid_embedding(h, self.weight, self.scale, self.freq, batch.token_ids, batch.positions)
+        return ResidualStream(h)
+
+
 @register_part("embedding", "pair_hash_embedding")
 class PairHashEmbedding(Part):
     """h = table[token] * scale + pair_table[row]: beside the token's own row, a row of a second table chosen by a hash of

@@ -1,4 +1,4 @@
-"""Recurrent mixers (state-space, delta rule): per-request state of fixed size instead of keys and values in pages."""
+"""Recurrent mixers (state-space, delta rule, matrix memory): per-request state of fixed size instead of keys and values in pages."""
 
 from __future__ import annotations
 
@@ -391,4 +391,69 @@ class ChannelDeltaRule(Part):
         ops.decay_recurrence(o, rows, state, batch.q_start, batch.state_slot, self.kv_heads, "delta", None, max_len=batch.max_q_len)
         gated = torch.empty((n, self.inner), dtype=x.dtype, device=x.device)
         ops.gated_group_rmsnorm(gated, o, g, 0, w["norm"], self.heads, self.eps, gate_after=True, gate="sigmoid")
+        return project(gated, w["o"])
+
+
+@register_part("mixer", "matrix_memory")
+class MatrixMemory(Part):
+    """A matrix memory with exponential gates (the matrix cell of xLSTM), on any mix of prompt portions and decoded tokens.
+
+    One product yields q | k | v | g (q and k: ``num_heads`` heads of ``head_dim``; v and g: heads of ``value_dim``), a second one
+    the two gates' float32 sums.  Per head and token, with c = ``gate_cap``, a log input gate i = c tanh((W_i x + b_i) / c) and a
+    log forget gate f = logsigmoid(c tanh((W_f x + b_f) / c)), a running maximum m that starts at 0, and q times head_dim^-1/2:
+
+        m' = max(f + m, i);    S <- exp(f + m - m') S + exp(i - m') k v^T;    n <- exp(f + m - m') n + exp(i - m') k;    m <- m'
+        o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)
+
+    Each head's o is divided by its root mean square (``eps``), multiplied by a weight and by sigmoid(g), and goes through the
+    output projection.  A request keeps S with n as one more value column (a column of values that are 1), and m, in its state
+    slot, all float32; everything starts at zero.  The gates' sums, gates, exponentials, maxima, state and read-outs are float32.
+
+    params: hidden_size, num_heads, head_dim, value_dim, gate_cap, eps, tensors (names of q, k, v, i, i_bias, f, f_bias, g, norm, o)."""
+
+    graph_capturable = True
+
+    def __init__(self, spec, env) -> None:
+        super().__init__(spec, env)
+        p = spec.params
+        self.hidden, self.heads = int(p["hidden_size"]), int(p["num_heads"])
+        self.d, self.dv = int(p["head_dim"]), int(p["value_dim"])
+        self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
+        if self.d > ops.MATRIX_MEMORY_MAX_HEAD_DIM:
+            raise ValueError(f"matrix_memory: head_dim={self.d} is above the scan kernel's {ops.MATRIX_MEMORY_MAX_HEAD_DIM}")
+        self.inner = self.heads * self.dv
+        self.g_col = 2 * self.heads * self.d + self.inner
+        defaults = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "i": "i_gate.weight", "i_bias": "i_gate.bias",
+                    "f": "f_gate.weight", "f_bias": "f_gate.bias", "g": "g_proj.weight", "norm": "norm.weight", "o": "o_proj.weight"}
+        self.names = {role: tensor_name(spec, role, default) for role, default in defaults.items()}
+        self.w: dict[str, torch.Tensor] = {}
+
+    def declare(self):
+        nm, H, qk = self.names, self.hidden, self.heads * self.d
+        return {nm["q"]: TensorDecl((qk, H)), nm["k"]: TensorDecl((qk, H)), nm["v"]: TensorDecl((self.inner, H)), nm["g"]: TensorDecl((self.inner, H)),
+                nm["i"]: TensorDecl((self.heads, H)), nm["f"]: TensorDecl((self.heads, H)), nm["o"]: TensorDecl((H, self.inner)),
+                nm["i_bias"]: TensorDecl((self.heads,), "vector32"), nm["f_bias"]: TensorDecl((self.heads,), "vector32"),
+                nm["norm"]: TensorDecl((self.inner,), "vector32")}
+
+    def load(self, tensors):
+        t = {role: tensors[name] for role, name in self.names.items()}
+        self.w = {"in": torch.cat([t["q"], t["k"], t["v"], t["g"]], 0).contiguous(), "gates": torch.cat([t["i"], t["f"]], 0).contiguous(),
+                  "gate_bias": torch.cat([t["i_bias"], t["f_bias"]], 0).contiguous(), "norm": t["norm"], "o": t["o"]}
+
+    def cache_need(self):
+        """S and n (kept transposed: a value column's head_dim numbers together, n behind the last one), and m — one copy
+        per value column, so that each column's owner reads and writes its own."""
+        return (StateNeed((self.heads, self.dv + 1, self.d), torch.float32), StateNeed((self.heads, self.dv + 1), torch.float32))
+
+    def forward(self, x: torch.Tensor, batch, cache) -> torch.Tensor:
+        w = self.w
+        n = x.shape[0]
+        state, top = cache.states
+        u = project(x, w["in"])  # q | k | v | g
+        gates = project(x, w["gates"], out_dtype=torch.float32)  # i | f
+        o = torch.empty((n, self.inner), dtype=torch.float32, device=x.device)
+        divisor = torch.empty((n, self.heads), dtype=torch.float32, device=x.device)
+        ops.matrix_memory_scan(o, divisor, u, gates, w["gate_bias"], self.cap, state, top, batch.q_start, batch.state_slot, max_len=batch.max_q_len)
+        gated = torch.empty((n, self.inner), dtype=x.dtype, device=x.device)
+        ops.gated_group_rmsnorm(gated, o, u, self.g_col, w["norm"], self.heads, self.eps, gate_after=True, gate="sigmoid", divisor=divisor)
         return project(gated, w["o"])

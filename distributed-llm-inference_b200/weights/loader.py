@@ -32,6 +32,8 @@ class TensorDecl:
     # name of another declared tensor this one must equal if the file stores it anyway
     # (a tied head some checkpoints serialise): the duplicate is checked and dropped
     optional_alias_of: str | None = None
+    # a tensor the model does not read: the checkpoint may hold it (then its shape is checked) or not
+    unused: bool = False
 
 
 def safetensor_files(model_dir: Path) -> list[Path]:
@@ -68,7 +70,7 @@ def load_tensors(
             where[name] = f  # a later shard wins, as a merged dict would
 
     aliases = {n: d.optional_alias_of for n, d in expected.items() if d.optional_alias_of}
-    required = {n for n in expected if n not in aliases}
+    required = {n for n, d in expected.items() if n not in aliases and not d.unused}
     missing = sorted(required - where.keys())
     unexpected = sorted(where.keys() - expected.keys())
     wrong = []

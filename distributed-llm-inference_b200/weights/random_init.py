@@ -36,7 +36,7 @@ def random_tensors(
     (Streams differ between CPU and CUDA generators; a folder is always written from the CPU.)"""
     out: dict[str, torch.Tensor] = {}
     for name, decl in sorted(expected.items()):
-        if decl.optional_alias_of:
+        if decl.optional_alias_of or decl.unused:
             continue
         g = _generator(seed, name, device)
         if any(d is None for d in decl.shape):

@@ -25,6 +25,13 @@ def embedding(h, table, ids):
     h.copy_(table[ids.long()].float())
 
 
+def sinusoid_embedding(h, table, scale, freq, ids, positions):
+    H = h.shape[1]
+    ang = (positions.double()[:, None] * freq.double().sum(0)[None, :]).float()
+    s = torch.stack([ang.sin(), ang.cos()], -1).reshape(h.shape[0], -1)[:, :H]
+    h.copy_(table[ids.long()].float() * scale + s)
+
+
 def patch_tokens(ids, source, src):
     pick = src >= 0
     ids[pick] = source[src[pick].long()]
@@ -104,7 +111,8 @@ def scale_softcap(logits, scale, cap):
         logits.copy_(cap * torch.tanh(logits / cap))
 
 
-def paged_attention_simt(out, qkv, k_pool, v_pool, block_tables, seq_of_token, positions, num_heads, scale, window=None, sink=None):
+def paged_attention_simt(out, qkv, k_pool, v_pool, block_tables, seq_of_token, positions, num_heads, scale, window=None, sink=None,
+                         softcap=None, slopes=None):
     n = out.shape[0]
     _, nkv, page_size, d = k_pool.shape
     fan = num_heads // nkv
@@ -120,6 +128,10 @@ def paged_attention_simt(out, qkv, k_pool, v_pool, block_tables, seq_of_token, p
         v = v_pool[pages, :, (keys % page_size).long(), :].float()
         k, v = k.repeat_interleave(fan, 1), v.repeat_interleave(fan, 1)  # [keys, nh, d]
         s = torch.einsum("hd,khd->hk", q[t], k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if slopes is not None:
+            s = s - slopes[:, None] * (p - keys)[None, :].float()
         if isinstance(sink, torch.Tensor):  # a learned score per head
             s = torch.cat([s, sink.float().view(num_heads, 1)], -1)
         elif sink is not None:  # one more term in the denominator, without a value
@@ -128,7 +140,7 @@ def paged_attention_simt(out, qkv, k_pool, v_pool, block_tables, seq_of_token, p
         out[t] = torch.einsum("hk,khd->hd", w, v).reshape(-1).to(out.dtype)
 
 
-def _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink=None):
+def _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink=None, **bend):
     """The bfloat16 attention kernels' common contract: sequences [seq0, seq0 + num_seqs); a sequence's
     tokens sit in rows q_start[s] .. q_start[s + 1] at positions kv_len[s] - q_len .. kv_len[s] - 1."""
     rows, seqs, pos = [], [], []
@@ -142,25 +154,25 @@ def _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_s
     idx = torch.tensor(rows)
     part = torch.empty((len(rows), out.shape[1]), dtype=out.dtype)
     paged_attention_simt(part, qkv[idx], k_pool, v_pool, block_tables, torch.tensor(seqs, dtype=torch.int32),
-                         torch.tensor(pos, dtype=torch.int32), num_heads, scale, window, sink)
+                         torch.tensor(pos, dtype=torch.int32), num_heads, scale, window, sink, **bend)
     out[idx] = part
 
 
 def paged_attention_mma(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, max_q_len, first_row, num_heads, scale,
-                        window=None, splits=1, scratch=None, sink=None):
+                        window=None, splits=1, scratch=None, sink=None, **bend):
     assert splits == 1 or (max_q_len == 1 and scratch is not None)
-    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink)
+    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink, **bend)
 
 
 def paged_decode_tma(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, first_row, num_heads, scale,
-                     window=None, splits=1, scratch=None, max_kv_len=0, sink=None):
+                     window=None, splits=1, scratch=None, max_kv_len=0, sink=None, **bend):
     assert splits == 1 or scratch is not None
-    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink)
+    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink, **bend)
 
 
 def paged_prefill_tc(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, max_q_len, num_heads, scale,
-                     window=None, query_tiles=0, sink=None):
-    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink)
+                     window=None, query_tiles=0, sink=None, **bend):
+    _attend(out, qkv, k_pool, v_pool, block_tables, q_start, kv_len, seq0, num_seqs, num_heads, scale, window, sink, **bend)
 
 
 # ---- layer norm around the residual stream, activations
@@ -228,6 +240,35 @@ def qk_norm_rotary_store(proj, wq, wk, eps, positions, inv_freq, slots, k_pool, 
         k_pool[page, :, off, :] = qk[:, num_heads:].to(k_pool.dtype)
         v_pool[page, :, off, :] = v.reshape(n, num_kv_heads, head_dim).to(v_pool.dtype)
     return qk[:, :num_heads].reshape(n, nq).to(proj.dtype)
+
+
+def qk_norm_mix_store(q_out, qkv, bias, wq, wk, eps, positions, temp, source, lam, slots, k_pool, v_pool, num_heads, num_kv_heads, head_dim, value_dim,
+                      page_size):
+    n = qkv.shape[0]
+    nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * value_dim
+    D = q_out.shape[1] // num_heads
+    x = qkv.float() + (bias if bias is not None else 0.0)
+    q, k, v = x[:, :nq], x[:, nq : nq + nk], x[:, nq + nk :]
+    if eps is not None:
+        q = q * torch.rsqrt((q * q).mean(-1, keepdim=True) + eps) * wq
+        k = k * torch.rsqrt((k * k).mean(-1, keepdim=True) + eps) * wk
+    if temp[0]:
+        q = q * (1 + temp[0] * torch.log(torch.floor((positions + 1).float() / temp[1]) + 1))[:, None]
+    if source is not None and lam is None:
+        source.copy_(v)
+    elif source is not None:
+        v = (1 - lam) * v + lam * source
+
+    def padded(a, heads, d):
+        out = torch.zeros((n, heads, D))
+        out[..., :d] = a.reshape(n, heads, d)
+        return out
+
+    q_out.copy_(padded(q, num_heads, head_dim).reshape(n, -1).to(q_out.dtype))
+    if slots is not None:
+        page, off = (slots // page_size).long(), (slots % page_size).long()
+        k_pool[page, :, off, :] = padded(k, num_kv_heads, head_dim).to(k_pool.dtype)
+        v_pool[page, :, off, :] = padded(v, num_kv_heads, value_dim).to(v_pool.dtype)
 
 
 def latent_prep(q_out, proj, w_norm, eps, positions, inv_freq, slots, k_pool, num_heads, head_dim, rot_dim, kv_rank, rotary_dim, page_size, amp=1.0):
@@ -305,8 +346,10 @@ def ssm_scan(y, xbc, u, dt_col, dt_bias, a_log, d_skip, state, q_start, state_sl
             y[t] = (torch.einsum("hpn,hn->hp", state[slot], C) + d_skip[:, None] * x).reshape(-1)
 
 
-def gated_group_rmsnorm(out, y, u, z_col, weight, parts, eps, gate_after=False, gate="silu"):
+def gated_group_rmsnorm(out, y, u, z_col, weight, parts, eps, gate_after=False, gate="silu", divisor=None):
     n, inner = y.shape
+    if divisor is not None:
+        y = (y.view(n, parts, inner // parts) / divisor[:, :, None]).reshape(n, inner)
     z = u[:, z_col : z_col + inner].float()
     gate = torch.sigmoid(z) if gate == "sigmoid" else _silu(z)
     g = (y if gate_after else y * gate).view(n, parts, inner // parts)
@@ -700,11 +743,35 @@ def decay_recurrence(o, rows, state, q_start, state_slot, kq_heads, mode, bonus=
                 o[t] = torch.einsum("hvd,hd->hv", S, a).reshape(-1)
 
 
-def moe_route(ids, weights, x, router, correction, group_count, group_keep, scale):
+def matrix_memory_scan(o, divisor, u, gates, gate_bias, cap, state, top, q_start, state_slot, max_len=0, form=None):
+    _, heads, dv1, d = state.shape
+    dv = dv1 - 1
+    z = cap * torch.tanh((gates + gate_bias) / cap)
+    log_in, log_forget = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+    for s in range(state_slot.numel()):
+        slot = int(state_slot[s])
+        for t in range(int(q_start[s]), int(q_start[s + 1])):
+            q = u[t, : heads * d].float().view(heads, d)
+            k = u[t, heads * d : 2 * heads * d].float().view(heads, d)
+            v = torch.cat([u[t, 2 * heads * d : 2 * heads * d + heads * dv].float().view(heads, dv), torch.ones(heads, 1)], 1)  # n: one more value column
+            m0 = top[slot, :, 0]
+            m = torch.maximum(log_forget[t] + m0, log_in[t])
+            keep, take = torch.exp(log_forget[t] + m0 - m), torch.exp(log_in[t] - m)
+            state[slot] = state[slot] * keep[:, None, None] + take[:, None, None] * v[:, :, None] * k[:, None, :]
+            top[slot] = m[:, None]
+            out = torch.einsum("hvd,hd->hv", state[slot], q) * d**-0.5
+            o[t] = out[:, :dv].reshape(-1)
+            divisor[t] = torch.maximum(out[:, dv].abs(), torch.exp(-m)) + 1e-6
+
+
+def moe_route(ids, weights, x, router, correction, group_count, group_keep, scale, score="sigmoid"):
     n, top = ids.shape
     E = router.shape[0]
-    s = torch.sigmoid(x.float() @ router.t())
+    s = x.float() @ router.t()
+    if score == "sigmoid":
+        s = torch.sigmoid(s)
     choice = s + correction
+    logits = choice
     if group_count > 1:
         per = E // group_count
         marks = choice.view(n, group_count, per).topk(min(2, per), -1).values.sum(-1)
@@ -715,6 +782,9 @@ def moe_route(ids, weights, x, router, correction, group_count, group_keep, scal
     picked = torch.sort(-choice, dim=-1, stable=True).indices[:, :top]
     w = s.gather(1, picked)
     ids.copy_(picked.to(torch.int32))
+    if score == "softmax_chosen":
+        weights.copy_(torch.softmax(logits.gather(1, picked), -1) * scale)
+        return
     weights.copy_(w / (w.sum(-1, keepdim=True) + 1e-20) * scale)
 
 
@@ -747,7 +817,7 @@ def batched_project(x, weight):
     return torch.bmm(x.float(), weight.float()).to(x.dtype)
 
 
-OPS = {"embedding": embedding, "patch_tokens": patch_tokens, "copy_page": copy_page, "add_rmsnorm": add_rmsnorm,
+OPS = {"embedding": embedding, "sinusoid_embedding": sinusoid_embedding, "qk_norm_mix_store": qk_norm_mix_store, "matrix_memory_scan": matrix_memory_scan, "patch_tokens": patch_tokens, "copy_page": copy_page, "add_rmsnorm": add_rmsnorm,
        "rotary_table": rotary_table, "rotary_store": rotary_store, "silu_mul": silu_mul, "paged_attention_simt": paged_attention_simt,
        "paged_attention_mma": paged_attention_mma, "paged_decode_tma": paged_decode_tma, "paged_prefill_tc": paged_prefill_tc,
        "skinny_gemm_slices": skinny_gemm_slices, "skinny_gemm": skinny_gemm, "skinny_gemm_residual": skinny_gemm_residual,
