@@ -105,4 +105,4 @@ def write_safetensors(path: str | Path, tensors: dict[str, torch.Tensor], metada
         fh.write(blob)
         for name in ordered:
             t = tensors[name].detach().contiguous().cpu()
-            fh.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            fh.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
