@@ -987,6 +987,144 @@ def lokolorn_kernels(size, pk, tokens=4096, seqs=64):
     return out
 
 
+def gedunex_sizes(width, heads, kv_heads, dim, memory_heads, memory_dim, window, ff, experts, top, lk, vocab=32000):
+    """A Gedunex model of eight layers (windowed attention with capped scores and mixed values, matrix memory, in turn) whose routed
+    feed-forward activates as many numbers a token as a dense one of size ``ff`` (``top`` experts of ff / top), and the Lokolorn
+    configuration of the same width, heads, experts and number of layer runs (``lk``: its sizes)."""
+    def mlp():
+        return {"kind": "moe", "expert": {"ff": ff // top}, "router": {"experts": experts, "top": top}}
+
+    att = {"type": "attention", "mlp": mlp(), "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim**-0.5, "softcap": 30.0,
+                                                        "mask": {"size": window}, "q_temp": {"coef": 0.1, "every": 4096}, "v_mix": True}}
+    mem = {"type": "mlstm", "mlp": mlp(), "mixer": {"heads": memory_heads, "dim": memory_dim, "vdim": memory_dim, "gate_cap": 12.0}}
+    gd = {"architecture": "Gedunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "layers": [att, mem] * 4}
+    lokolorn, _ = lokolorn_sizes(vocab=vocab, **lk)
+    return gd, lokolorn
+
+
+GEDUNEX_SIZES = {
+    name: dict(width=s["width"], heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"], memory_heads=s["delta_heads"], memory_dim=s["delta_dim"],
+               window=s["window"], ff=s["ff"], experts=s["experts"], top=s["top"], lk=s)
+    for name, s in LOKOLORN_SIZES.items()
+}
+
+
+def gedunex_kernels(size, pk, tokens=4096, seqs=64):
+    """Every kernel of the Gedunex parts beside its like, at one size: a prompt portion of ``tokens`` tokens and a decode step of ``seqs``
+    sequences.  us, the bytes (or operations) the kernel has to move, and the share of the measured HBM peak (of the measured bf16 rate
+    for attention, of the CUDA cores' float32 rate for the recurrences)."""
+    import torch
+
+    from dli_b200.kernels import attention as attn
+    from dli_b200.kernels import gemm, ops
+
+    dev, bf = "cuda", torch.bfloat16
+    W, nh, nkv, d = size["width"], size["heads"], size["kv_heads"], size["dim"]
+    Hm, dm, E, top = size["memory_heads"], size["memory_dim"], size["experts"], size["top"]
+    out = {}
+
+    def record(name, us, nbytes, like=None, flops=None, tensor=False):
+        rec = {"us": round(us, 1), "gb_s": round(nbytes / us / 1e3, 1), "hbm_frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)}
+        if flops is not None and tensor:
+            rec["tflops_bf16"] = round(flops / us / 1e6, 1)
+            rec["bf16_frac"] = round(flops / us / 1e6 / pk["bf16_tflops"], 3)
+        elif flops is not None:
+            rec["tflops_fp32"] = round(flops / us / 1e6, 2)
+            rec["simt_frac"] = round(flops / us / 1e6 / SIMT_FP32_TFLOPS, 3)
+        if like:
+            rec["like"] = like
+        out[name] = rec
+
+    for label, n, S in (("portion", tokens, 1), ("decode", seqs, seqs)):
+        q_len, context = n // S, (n if S == 1 else 2048)
+        q_start = torch.arange(S + 1, dtype=torch.int32, device=dev) * q_len
+        seq_of = torch.repeat_interleave(torch.arange(S, dtype=torch.int32), q_len).to(dev)
+        slot = torch.arange(S, dtype=torch.int32, device=dev)
+        positions = (torch.arange(n, dtype=torch.int32) % q_len + (0 if S == 1 else context - 1)).to(dev)
+        # embedding
+        table, ids = torch.randn(32000, W, device=dev).to(bf), torch.randint(0, 32000, (n,), dtype=torch.int32, device=dev)
+        h, freq = torch.empty(n, W, device=dev), torch.rand(2, W // 2, device=dev)
+        record(f"{label}.sinusoid_embedding", time_kernel(lambda: ops.sinusoid_embedding(h, table, 8.0, freq, ids, positions)), n * W * 6, "embedding")
+        record(f"{label}.embedding", time_kernel(lambda: ops.embedding(h, table, ids)), n * W * 6)
+        # what lies between the q | k | v product and the attention kernel (a decode step's product leaves float32 sums)
+        C = (nh + 2 * nkv) * d
+        pages = -(-context // 16) * S + 1
+        kp, vp = (torch.randn(pages, nkv, 16, d, device=dev).to(bf) for _ in range(2))
+        slots = torch.arange(n, dtype=torch.int32, device=dev)
+        proj = torch.randn(n, C, device=dev).to(bf)
+        wq, wk, src = torch.ones(nh * d, device=dev), torch.ones(nkv * d, device=dev), torch.randn(n, nkv * d, device=dev)
+        q = torch.empty(n, nh * d, dtype=bf, device=dev)
+        record(f"{label}.qk_norm_mix_store",
+               time_kernel(lambda: ops.qk_norm_mix_store(q, proj, None, wq, wk, 1e-6, positions, (0.1, 4096.0), src, 0.5, slots, kp, vp, nh, nkv, d, d, 16)),
+               n * (C * 4 + nkv * d * 4), "qk_norm_rotary_store")
+        inv = (1.0 / (10000.0 ** (torch.arange(0, d, 2).float() / d))).to(dev)
+        record(f"{label}.qk_norm_rotary_store", time_kernel(lambda: ops.qk_norm_rotary_store(proj, wq, wk, 1e-6, positions, inv, slots, kp, vp, nh, nkv, d, d, 16,
+                                                                                             True, False)), n * C * 4)
+        # attention with bent scores beside the same kernels without
+        tables = (torch.randperm(pages - 1, device=dev)[: -(-context // 16) * S].view(S, -1)).to(torch.int32)
+
+        class Group:
+            block_tables = tables
+
+        class Batch:
+            num_single, num_seqs, max_q_len, max_kv_len = (S if q_len == 1 else 0), S, q_len, context
+            max_kv_len_single = context if q_len == 1 else 0
+
+            def group(self, i):
+                return Group
+
+        Batch.q_start, Batch.kv_len, Batch.seq_of_token, Batch.positions = q_start, torch.full((S,), context, dtype=torch.int32, device=dev), seq_of, positions
+
+        class Cache:
+            k, v, page_size, group = kp, vp, 16, 0
+
+        o = torch.empty(n, nh * d, dtype=bf, device=dev)
+        sinks, slopes = torch.zeros(nh, device=dev), torch.tensor([2.0 ** (-8.0 * (i + 1) / nh) for i in range(nh)], device=dev)
+        for wname, window in (("", None), (f"_window{size['window']}", size["window"])):
+            def seen(p):
+                return p + 1 if window is None else min(p + 1, window)
+
+            pairs = sum(seen(p) for p in range(n)) if S == 1 else S * seen(context - 1)
+            moved = (n if S == 1 else S * seen(context - 1)) * nkv * d * 4 + n * nh * d * 4
+            bent = {"softcap": 30.0, "slopes": slopes}
+            splits = attn.decode_splits(S, nh, nkv, d, 16, context if window is None else min(context, window + 64)) if q_len == 1 else None
+            us = time_kernel(lambda: attn.paged_attention(o, q, Cache, Batch(), nh, d**-0.5, window, splits=splits, sink=sinks, **bent))
+            record(f"{label}.bent_attention{wname}", us, moved, f"sink_attention{wname}", flops=4.0 * pairs * nh * d, tensor=True)
+            us = time_kernel(lambda: attn.paged_attention(o, q, Cache, Batch(), nh, d**-0.5, window, splits=splits, sink=sinks))
+            record(f"{label}.sink_attention{wname}", us, moved, flops=4.0 * pairs * nh * d, tensor=True)
+        # matrix memory: gates' product, scan, norm; its likes: the two delta rules
+        inner = Hm * dm
+        x = torch.randn(n, W, device=dev).to(bf)
+        wg = torch.randn(2 * Hm, W, device=dev).to(bf)
+        record(f"{label}.gates_product", time_kernel(lambda: gemm.project(x, wg, out_dtype=torch.float32)), n * W * 2 + 2 * Hm * W * 2)
+        u = torch.randn(n, 4 * inner, device=dev).to(bf)
+        gates, gb = torch.randn(n, 2 * Hm, device=dev), torch.cat([torch.zeros(Hm, device=dev), torch.full((Hm,), 4.0, device=dev)])
+        st, mt = torch.zeros(S, Hm, dm + 1, dm, device=dev), torch.zeros(S, Hm, dm + 1, device=dev)
+        om, div = torch.empty(n, inner, device=dev), torch.empty(n, Hm, device=dev)
+        state_bytes, flops = S * Hm * dm * dm * 8, 5.0 * n * Hm * dm * dm
+        record(f"{label}.matrix_memory", time_kernel(lambda: ops.matrix_memory_scan(om, div, u, gates, gb, 12.0, st, mt, q_start, slot, max_len=q_len)),
+               state_bytes + n * inner * 10, "delta_rule_scan", flops=flops)
+        qkv = torch.randn(n, 3 * inner, device=dev).to(bf)
+        u3 = torch.randn(n, 4 * inner + 2 * Hm, device=dev).to(bf)
+        dt1, al1, st2 = torch.zeros(Hm, device=dev), torch.full((Hm,), -3.0, device=dev), torch.zeros(S, Hm, dm, dm, device=dev)
+        us = time_kernel(lambda: ops.delta_rule_scan(om, qkv, u3, 4 * inner, 4 * inner + Hm, dt1, al1, st2, seq_of, q_start, slot, Hm, dm, 1e-6, max_len=q_len))
+        record(f"{label}.delta_rule_scan", us, state_bytes + n * inner * 10, flops=8.0 * n * Hm * dm * dm)
+        rows = torch.rand(n, ops.decay_recurrence_row(Hm, Hm, dm, dm), device=dev)
+        us = time_kernel(lambda: ops.decay_recurrence(om, rows, st2, q_start, slot, Hm, "delta", None, max_len=q_len))
+        record(f"{label}.recurrence_delta", us, state_bytes + n * inner * 20, flops=8.0 * n * Hm * dm * dm)
+        gated, nw = torch.empty(n, inner, dtype=bf, device=dev), torch.ones(inner, device=dev)
+        record(f"{label}.head_norm_with_divisor", time_kernel(lambda: ops.gated_group_rmsnorm(gated, om, u, 0, nw, Hm, 1e-6, gate_after=True, gate="sigmoid", divisor=div)),
+               n * inner * 8, "head_norm")
+        record(f"{label}.head_norm", time_kernel(lambda: ops.gated_group_rmsnorm(gated, om, u, 0, nw, Hm, 1e-6, gate_after=True, gate="sigmoid")), n * inner * 8)
+        # router
+        router, rb = torch.randn(E, W, device=dev) * 0.05, torch.randn(E, device=dev) * 0.1
+        ids2, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        record(f"{label}.route_softmax_chosen", time_kernel(lambda: ops.moe_route(ids2, wts, x, router, rb, 1, 1, 1.0, "softmax_chosen")), n * W * 2 + E * W * 4,
+               "route_sigmoid")
+        record(f"{label}.route_sigmoid", time_kernel(lambda: ops.moe_route(ids2, wts, x, router, rb, 4, 2, 2.5)), n * W * 2 + E * W * 4)
+    return out
+
+
 SIMT_FP32_TFLOPS = 148 * 128 * 2 * 1.9e9 / 1e12  # CUDA-core multiply-adds of a B200 at 1.9 GHz: the scan's ceiling (no float32 tensor-core path)
 
 
@@ -996,6 +1134,7 @@ DESIGNS = {
     "sugonex": (SUGONEX_SIZES, sugonex_sizes, "pazenex", sugonex_kernels),
     "pokadra": (POKADRA_SIZES, pokadra_sizes, "pazenex", pokadra_kernels),
     "lokolorn": (LOKOLORN_SIZES, lokolorn_sizes, "sugonex", lokolorn_kernels),
+    "gedunex": (GEDUNEX_SIZES, gedunex_sizes, "lokolorn", gedunex_kernels),
 }
 
 
@@ -1237,7 +1376,7 @@ def main() -> int:
     ap.add_argument("--phase", default="all", choices=["all", "decode", "prefill", "sample"],
                     help="profiling runs: only the device-timed decode steps, only the prefill step, or only the sampling kernel (prints a short line)")
     ap.add_argument("--no-graphs", action="store_true", help="profiling runs: launch the step's kernels one by one")
-    ap.add_argument("--design", default=None, choices=["pazenex", "sugonex", "pokadra", "lokolorn"],
+    ap.add_argument("--design", default=None, choices=["pazenex", "sugonex", "pokadra", "lokolorn", "gedunex"],
                     help="another measurement: this architecture beside Llama at equal sizes, and its kernels beside their likes (prints its own line)")
     ap.add_argument("--size", default=None, choices=list(DESIGN_SIZES), help="--design: one size only (every design has these names)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN,

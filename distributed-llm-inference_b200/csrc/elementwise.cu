@@ -50,7 +50,7 @@ DLI_EXPORT int dli_embedding(float* h, const void* table, const int* ids, int n,
 
 // h[t] = table[ids[t]] * scale + the position's vector of sines (even places) and cosines (odd places).  A thread makes a pair of
 // places with one sincosf: the angle a is the rounded product position * frequency, e what that rounding and the frequency's
-// own left out, and sin(a + e) = sin a + e cos a, cos(a + e) = cos a - e sin a to float32.
+// own left out; sin(a + e) and cos(a + e) to the second order in e (which stays below 0.004 up to position 100,000).
 template <typename T, bool PAIRS>
 __global__ void sinusoid_embedding_kernel(float* __restrict__ h, const T* __restrict__ table, float scale, const float* __restrict__ freq,
                                           const int* __restrict__ ids, const int* __restrict__ positions, int H) {
@@ -65,7 +65,8 @@ __global__ void sinusoid_embedding_kernel(float* __restrict__ h, const T* __rest
     const float e = fmaf(pos, f, -a) + pos * freq[pairs + i];
     float sn, cs;
     sincosf(a, &sn, &cs);
-    const float s0 = fmaf(e, cs, sn), c0 = fmaf(-e, sn, cs);
+    const float h2 = 0.5f * e * e;
+    const float s0 = fmaf(e, cs, fmaf(-h2, sn, sn)), c0 = fmaf(-e, sn, fmaf(-h2, cs, cs));
     if (PAIRS) {
       float x0, x1;
       if constexpr (sizeof(T) == 2) {
