@@ -14,6 +14,12 @@
 // A warp owns 16 value columns of one head of one sequence; S^T of those columns stays in its registers as the accumulator of
 // mma.sync m16n8k16 over all tiles (the layout of an accumulator of S^T is that of the B operand of Q S, so nothing moves).  The
 // vector n is one more value column, whose value is always 1.  Tokens arrive by cp.async a tile ahead; a CTA's warps share them.
+//
+// A few long sequences leave most of the GPU idle, because a sequence's tiles follow one another.  They are then cut into segments of
+// whole tiles, in two launches: the first computes what every segment but the last adds to a state (L, its maximum, the sum B of its
+// log forget gates; no read-outs), the second starts every segment from the states in front of it,
+//   m' = max(m + B, m_L),   S <- exp(m + B - m') S + exp(m_L - m') L,   segment after segment,
+// and walks all segments side by side.
 #include "common.cuh"
 #include "matrix_memory.cuh"
 #include <math_constants.h>
@@ -54,6 +60,9 @@ struct Params {
   const int* q_start;
   const int* state_slot;
   int heads, d, dv, warps, vec;
+  int segments;           // of a sequence; with more than one:
+  float* part;            // [seqs][segments][heads][dv + 1][d]: slot 0 the state at the start, slot g + 1 what segment g adds
+  float* part_m;          // [seqs][segments][heads][dv + 1][2]: its maximum, the sum of its log forget gates (a copy per column)
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -92,12 +101,17 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t&
   lo = pack2(x - m.x, y - m.y);
 }
 
+// LOCAL: the first of the two launches over segments (what a segment adds to a state, no read-outs).
+template <bool LOCAL>
 __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(const Params p) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(128) unsigned char smem[];
-  const int seq = blockIdx.z, head = blockIdx.y;
-  const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
+  const int launched = LOCAL ? p.segments - 1 : p.segments;
+  const int seq = blockIdx.z / launched, seg = blockIdx.z - seq * launched, head = blockIdx.y;
+  const int first = p.q_start[seq], last = p.q_start[seq + 1];
+  const int per_segment = ((last - first + TOKENS - 1) / TOKENS + p.segments - 1) / p.segments * TOKENS;
+  const int t0 = first + seg * per_segment, t1 = min(last, t0 + per_segment);  // this CTA's tokens
   if (t1 <= t0) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthreads = p.warps * 32;
   const int d = p.d, dv = p.dv, cols = dv + 1, heads = p.heads;
@@ -119,7 +133,7 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
         const int r = e / (DK / 8), c = e - r * (DK / 8);
         const bool ok = base + r < t1 && c * 8 < d;
         const bf16* src = ubase + (ok ? (size_t)(base + r) * p.u_stride + c * 8 : 0);
-        cp_async16(smem_u32(sQ + r * QK_ROW + c * 16), src, ok ? 16 : 0);
+        if (!LOCAL) cp_async16(smem_u32(sQ + r * QK_ROW + c * 16), src, ok ? 16 : 0);
         cp_async16(smem_u32(sK + r * QK_ROW + c * 16), src + (size_t)heads * d, ok ? 16 : 0);
       }
       const int chunks = vcols / 8;
@@ -166,18 +180,41 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
 
   // ---- the state: S^T, rows = this warp's value columns, columns = key rows, in accumulators of 16 x 8
   const size_t sbase = ((size_t)p.state_slot[seq] * heads + head) * cols;
+  auto pbase = [&](int slot) { return (((size_t)seq * p.segments + slot) * heads + head) * cols; };
   float S[DK / 8][4];
   const int row_lo = col0 + (lane >> 2), row_hi = row_lo + 8, kcol = (lane & 3) * 2;
+  auto each = [&](auto&& fn) {  // fn(accumulator j, element e, offset of that number in a [dv + 1][d] block) for the numbers that exist
 #pragma unroll
-  for (int j = 0; j < DK / 8; ++j) {
-    const int i = j * 8 + kcol;
+    for (int j = 0; j < DK / 8; ++j)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int col = e < 2 ? row_lo : row_hi, ii = i + (e & 1);
-      S[j][e] = (col < cols && ii < d) ? p.state[(sbase + col) * d + ii] : 0.f;
+      for (int e = 0; e < 4; ++e) {
+        const int col = e < 2 ? row_lo : row_hi, i = j * 8 + kcol + (e & 1);
+        if (col < cols && i < d) fn(j, e, (size_t)col * d + i);
+      }
+  };
+#pragma unroll
+  for (int j = 0; j < DK / 8; ++j) S[j][0] = S[j][1] = S[j][2] = S[j][3] = 0.f;
+  float m0 = -CUDART_INF_F, forgot = 0.f;  // forgot: the sum of the log forget gates so far (LOCAL)
+  if (LOCAL) {
+    if (seg == 0 && active) {  // the state at the start, set aside: the second launch's last segment writes over it
+      float* dst = p.part + pbase(0) * d;
+      const float* src = p.state + sbase * d;
+      each([&](int, int, size_t at) { dst[at] = src[at]; });
+      if (lane < 16 && col0 + lane < cols) p.part_m[(pbase(0) + col0 + lane) * 2] = p.top[sbase + col0 + lane];
+    }
+  } else if (active) {
+    const float* src = p.segments == 1 ? p.state + sbase * d : p.part + pbase(0) * d;
+    each([&](int j, int e, size_t at) { S[j][e] = src[at]; });
+    m0 = p.segments == 1 ? p.top[sbase + col0] : p.part_m[(pbase(0) + col0) * 2];
+    for (int g = 1; g <= seg; ++g) {
+      const float* meta = p.part_m + (pbase(g) + col0) * 2;
+      const float mb = m0 + meta[1], next = fmaxf(mb, meta[0]);
+      const float keep = expf(mb - next), take = expf(meta[0] - next);
+      const float* add = p.part + pbase(g) * d;
+      each([&](int j, int e, size_t at) { S[j][e] = fmaf(keep, S[j][e], take * add[at]); });
+      m0 = next;
     }
   }
-  float m0 = active ? p.top[sbase + col0] : 0.f;
   const float bias_i = p.bias[head], bias_f = p.bias[heads + head];
   const float scale = 1.f / sqrtf((float)d);
   float raw[4];
@@ -239,6 +276,7 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
       const uint32_t q_addr = smem_u32(sQ) + (lane & 15) * QK_ROW + (lane >> 4) * 16;
       const float m02 = m0 * LOG2E;
 
+      if constexpr (!LOCAL) {
       // ---- what the state at the tile's start gives: O = Q S0, 64 tokens x 16 columns
       float O[TOKENS / 16][2][4];
 #pragma unroll
@@ -252,18 +290,16 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
         split3(S[2 * kk + 1][0], S[2 * kk + 1][1], B[0][1], B[1][1], B[2][1]);
         split3(S[2 * kk][2], S[2 * kk][3], B[0][2], B[1][2], B[2][2]);
         split3(S[2 * kk + 1][2], S[2 * kk + 1][3], B[0][3], B[1][3], B[2][3]);
+        uint32_t a[TOKENS / 16][4];
 #pragma unroll
-        for (int mt = 0; mt < TOKENS / 16; ++mt) {
-          if (mt * 16 < len) {
-            uint32_t a[4];
-            ldsm_x4(a, q_addr + mt * 16 * QK_ROW + kk * 32);
+        for (int mt = 0; mt < TOKENS / 16; ++mt) ldsm_x4(a[mt], q_addr + mt * 16 * QK_ROW + kk * 32);
 #pragma unroll
-            for (int s = 2; s >= 0; --s) {  // the small terms first
-              mma(O[mt][0], a, B[s][0], B[s][1]);
-              mma(O[mt][1], a, B[s][2], B[s][3]);
-            }
+        for (int s = 2; s >= 0; --s)  // the small terms first; eight accumulators in turn, so that no product waits for the one before
+#pragma unroll
+          for (int mt = 0; mt < TOKENS / 16; ++mt) {
+            mma(O[mt][0], a[mt], B[s][0], B[s][1]);
+            mma(O[mt][1], a[mt], B[s][2], B[s][3]);
           }
-        }
       }
 
       // ---- what the tile's own tokens give, sixteen rows at a time
@@ -302,6 +338,11 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
             P[j][2] = tok <= r_hi ? P[j][2] * ex2(a0 - g_hi) : 0.f;
             P[j][3] = tok + 1 <= r_hi ? P[j][3] * ex2(a1 - g_hi) : 0.f;
           }
+          float T[3][2][4];  // the three terms' sums apart: six accumulators in turn
+#pragma unroll
+          for (int s = 0; s < 3; ++s)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) T[s][0][e] = T[s][1][e] = 0.f;
 #pragma unroll
           for (int kk = 0; kk <= mt; ++kk) {
             uint32_t A[3][4], b[4];
@@ -312,10 +353,14 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
             ldsm_x4_trans(b, smem_u32(sV) + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * V_ROW + (lane >> 4) * 16);
 #pragma unroll
             for (int s = 2; s >= 0; --s) {
-              mma(O[mt][0], A[s], b[0], b[1]);
-              mma(O[mt][1], A[s], b[2], b[3]);
+              mma(T[s][0], A[s], b[0], b[1]);
+              mma(T[s][1], A[s], b[2], b[3]);
             }
           }
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) O[mt][nt][e] += (T[2][nt][e] + T[1][nt][e]) + T[0][nt][e];
         }
       }
 
@@ -348,6 +393,7 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
         }
       }
 
+      }
       // ---- the state at the tile's end: S^T <- exp(m0 - g_C) S^T + (w V)^T K, w_j = exp(a_j - g_C)
       const float eC = ex2(m02 - gC);
 #pragma unroll
@@ -364,48 +410,78 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) matrix_memory_chunk_kernel(con
             const float2 x = unpack2(v[e]);
             split3(x.x * (e < 2 ? w0 : w8), x.y * (e < 2 ? w1 : w9), A[0][e], A[1][e], A[2][e]);
           }
+          constexpr int GROUP = (DK / 16) % 4 == 0 ? 4 : ((DK / 16) % 3 == 0 ? 3 : ((DK / 16) % 2 == 0 ? 2 : 1));
 #pragma unroll
-          for (int jp = 0; jp < DK / 16; ++jp) {
-            uint32_t b[4];
-            ldsm_x4_trans(b, smem_u32(sK) + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QK_ROW + (jp * 16 + (lane >> 4) * 8) * 2);
+          for (int j0 = 0; j0 < DK / 16; j0 += GROUP) {  // 2 GROUP accumulators in turn
+            uint32_t b[GROUP][4];
 #pragma unroll
-            for (int s = 2; s >= 0; --s) {
-              mma(S[2 * jp], A[s], b[0], b[1]);
-              mma(S[2 * jp + 1], A[s], b[2], b[3]);
-            }
+            for (int g = 0; g < GROUP; ++g)
+              ldsm_x4_trans(b[g], smem_u32(sK) + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * QK_ROW + ((j0 + g) * 16 + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int s = 2; s >= 0; --s)
+#pragma unroll
+              for (int g = 0; g < GROUP; ++g) {
+                mma(S[2 * (j0 + g)], A[s], b[g][0], b[g][1]);
+                mma(S[2 * (j0 + g) + 1], A[s], b[g][2], b[g][3]);
+              }
           }
         }
       }
     }
     m0 = (bC + gC) * (1.f / LOG2E);
+    if (LOCAL) forgot += bC * (1.f / LOG2E);
     if (base + TOKENS < t1) load_gates(base + TOKENS, raw);
     __syncthreads();  // this stage is copied into again in the round after next; sA and sG are written anew
   }
   cp_async_wait<0>();
   if (!active) return;
-#pragma unroll
-  for (int j = 0; j < DK / 8; ++j) {
-    const int i = j * 8 + kcol;
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int col = e < 2 ? row_lo : row_hi, ii = i + (e & 1);
-      if (col < cols && ii < d) p.state[(sbase + col) * d + ii] = S[j][e];
+  if (LOCAL) {
+    float* dst = p.part + pbase(seg + 1) * d;
+    each([&](int j, int e, size_t at) { dst[at] = S[j][e]; });
+    if (lane < 16 && col0 + lane < cols) {
+      p.part_m[(pbase(seg + 1) + col0 + lane) * 2] = m0;
+      p.part_m[(pbase(seg + 1) + col0 + lane) * 2 + 1] = forgot;
     }
+  } else if (t1 == last) {
+    float* dst = p.state + sbase * d;
+    each([&](int j, int e, size_t at) { dst[at] = S[j][e]; });
+    if (lane < 16 && col0 + lane < cols) p.top[sbase + col0 + lane] = m0;
   }
-  if (lane < 16 && col0 + lane < cols) p.top[sbase + col0 + lane] = m0;
 }
 
 }  // namespace
 
+namespace {
+// CTAs of a sequence's head, and warps of a CTA (even shares of the value columns' tiles of sixteen)
+inline void shares(int dv, int& ctas, int& warps) {
+  const int tiles = (dv + 1 + 15) / 16;
+  ctas = (tiles + MAX_WARPS - 1) / MAX_WARPS;
+  warps = (tiles + ctas - 1) / ctas;
+}
+}  // namespace
+
+// Into how many segments the sequences of a step are cut: as many as give every SM two CTAs, none shorter than four tiles.
+DLI_EXPORT int dli_matrix_memory_segments(int num_seqs, int heads, int dv, int max_len) {
+  int ctas, warps;
+  shares(dv, ctas, warps);
+  long long fill = 2LL * sm_count() / ((long long)ctas * heads * (num_seqs > 0 ? num_seqs : 1));
+  const int most = (max_len + TOKENS - 1) / TOKENS / 4;
+  if (fill > most) fill = most;
+  return fill < 1 ? 1 : (fill > 64 ? 64 : (int)fill);
+}
+
+// segments > 1: part [num_seqs segments heads (dv + 1) d] and part_m [num_seqs segments heads (dv + 1) 2] are scratch.
 DLI_EXPORT int dli_matrix_memory_chunk(float* o, float* divisor, const void* u, long long u_stride, const float* gates, const float* bias, float cap,
                                        float* state, float* top, const int* q_start, const int* state_slot, int num_seqs, int heads, int d, int dv,
-                                       int max_len, cudaStream_t stream) {
-  (void)max_len;
+                                       int segments, float* part, float* part_m, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
-  if (heads < 1 || heads > 65535 || num_seqs > 65535 || d < 1 || d > DK || dv < 1 || !(cap > 0.f)) return DLI_ERR_UNSUPPORTED;
+  if (heads < 1 || heads > 65535 || segments < 1 || (long long)num_seqs * segments > 65535 || d < 1 || d > DK || dv < 1 || !(cap > 0.f) ||
+      (segments > 1 && (!part || !part_m)))
+    return DLI_ERR_UNSUPPORTED;
   static OncePerDevice configured;
   if (!configured.here()) {
-    cudaError_t e = cudaFuncSetAttribute(matrix_memory_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaError_t e = cudaFuncSetAttribute(matrix_memory_chunk_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(matrix_memory_chunk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return (int)e;
     configured.here() = true;
   }
@@ -413,7 +489,13 @@ DLI_EXPORT int dli_matrix_memory_chunk(float* o, float* divisor, const void* u, 
   p.o = o; p.divisor = divisor; p.u = (const bf16*)u; p.u_stride = u_stride; p.gates = gates; p.bias = bias; p.cap = cap;
   p.state = state; p.top = top; p.q_start = q_start; p.state_slot = state_slot; p.heads = heads; p.d = d; p.dv = dv;
   p.vec = (d % 8) == 0 && (dv % 8) == 0 && (u_stride % 8) == 0 && ((uintptr_t)u & 15) == 0;
-  const int tiles = (dv + 1 + 15) / 16, ctas = (tiles + MAX_WARPS - 1) / MAX_WARPS;
-  p.warps = (tiles + ctas - 1) / ctas;  // even shares
-  return (int)launch_pdl(matrix_memory_chunk_kernel, dim3(ctas, heads, num_seqs), dim3(p.warps * 32), (size_t)SMEM, stream, 1, p);
+  p.segments = segments; p.part = part; p.part_m = part_m;
+  int ctas;
+  shares(dv, ctas, p.warps);
+  if (segments > 1) {
+    const cudaError_t e = launch_pdl((matrix_memory_chunk_kernel<true>), dim3(ctas, heads, num_seqs * (segments - 1)), dim3(p.warps * 32), (size_t)SMEM,
+                                     stream, 1, p);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl((matrix_memory_chunk_kernel<false>), dim3(ctas, heads, num_seqs * segments), dim3(p.warps * 32), (size_t)SMEM, stream, 1, p);
 }

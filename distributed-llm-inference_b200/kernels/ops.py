@@ -1676,13 +1676,14 @@ def matrix_memory_form(dtype: torch.dtype, d: int, max_len: int) -> str:
 
 def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: float,
                        state: torch.Tensor, top: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, max_len: int = 1 << 30,
-                       form: str | None = None) -> None:
+                       form: str | None = None, segments: int = 0) -> None:
     """A matrix memory with exponential gates over every sequence's tokens of this step, from and to its slot of ``state``
     [slots, heads, dv + 1, d] (float32; S transposed, the last row is n) and ``top`` [slots, heads, dv + 1] (m, a copy per column).
     u [n, .]: q | k | v in its leading columns (heads of d, d, dv); gates [n, 2 heads] float32: the input gates' sums, then the
     forget gates'; ``gate_bias`` [2 heads].  Per head i = cap tanh((gate + bias) / cap), f = logsigmoid(cap tanh(...)),
     m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone.  Left: o [n, heads dv] = S^T q / sqrt(d)
-    and divisor [n, heads] = max(|n . q| / sqrt(d), exp(-m)) + 1e-6, both float32.  ``form``: ``"walk"``, ``"chunk"``, or None (chosen)."""
+    and divisor [n, heads] = max(|n . q| / sqrt(d), exp(-m)) + 1e-6, both float32.  ``form``: ``"walk"``, ``"chunk"``, or None (chosen).
+    ``segments`` (of the form ``"chunk"``; 0: chosen): into how many runs of tiles a sequence is cut that are walked side by side."""
     _columns(u, "matrix_memory_scan"), _need(o, "o", torch.float32), _need(divisor, "divisor", torch.float32)
     _need(gates, "gates", torch.float32), _need(gate_bias, "gate_bias", torch.float32)
     _need(state, "state", torch.float32), _need(top, "top", torch.float32)
@@ -1695,16 +1696,25 @@ def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, 
         raise KernelError(f"matrix_memory_scan: shapes do not agree (or the head size is above {MATRIX_MEMORY_MAX_HEAD_DIM})")
     form = form or matrix_memory_form(u.dtype, d, max_len)
     args = (_ptr(o), _ptr(divisor), _ptr(u), u.stride(0), _ptr(gates), _ptr(gate_bias), float(cap), _ptr(state), _ptr(top), _ptr(q_start), _ptr(state_slot),
-            state_slot.numel(), heads, d, dv, int(max_len))
-    types = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 5
+            state_slot.numel(), heads, d, dv)
+    types = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 4
     if form == "chunk":
         if u.dtype != torch.bfloat16 or d > MATRIX_MEMORY_CHUNK_MAX_HEAD_DIM:
             raise KernelError("matrix_memory_scan: the tensor-core form takes bfloat16 heads of at most 256")
-        f = _fn("matrix_memory_tc.cu", "dli_matrix_memory_chunk", types + [c_void_p], {"KEY_DIM": -(-d // 16) * 16})
-        _check(f(*args, _stream()), "matrix_memory_scan")
+        lib = {"KEY_DIM": -(-d // 16) * 16}
+        if segments < 1:
+            segments = _fn("matrix_memory_tc.cu", "dli_matrix_memory_segments", [c_int] * 4, lib)(state_slot.numel(), heads, dv, int(min(max_len, n)))
+        part = part_m = None
+        if segments > 1:
+            rows = state_slot.numel() * segments * heads * dv1
+            part, part_m = torch.empty(rows * d, dtype=torch.float32, device=o.device), torch.empty(rows * 2, dtype=torch.float32, device=o.device)
+        f = _fn("matrix_memory_tc.cu", "dli_matrix_memory_chunk", types + [c_int, c_void_p, c_void_p, c_void_p], lib)
+        _check(f(*args, segments, _ptr(part), _ptr(part_m), _stream()), "matrix_memory_scan")
+        global launch_count
+        launch_count += segments > 1  # two launches
     elif form == "walk":
-        f = _fn("matrix_memory.cu", "dli_matrix_memory_walk", types + [c_int, c_void_p])
-        _check(f(*args, DT_CODE[u.dtype], _stream()), "matrix_memory_scan")
+        f = _fn("matrix_memory.cu", "dli_matrix_memory_walk", types + [c_int, c_int, c_void_p])
+        _check(f(*args, int(max_len), DT_CODE[u.dtype], _stream()), "matrix_memory_scan")
     else:
         raise KernelError("matrix_memory_scan: form is walk or chunk")
 

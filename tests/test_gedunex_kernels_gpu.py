@@ -108,12 +108,12 @@ def test_matrix_memory(sizes, dtype, form):
     q_start = _i32([0] + torch.tensor(lens).cumsum(0).tolist())
     slots = _i32([3, 0, 4, 1, 2])
 
-    def run(module, where, form=None, one_by_one=False):
+    def run(module, where, form=None, one_by_one=False, **more):
         o, div = torch.zeros(n, heads * dv, device=where), torch.zeros(n, heads, device=where)
         s, m = state.clone().to(where), top.clone().to(where)
         ud, gd, bd = u.to(where), gates.to(where), bias.to(where)
         if not one_by_one:
-            module.matrix_memory_scan(o, div, ud, gd, bd, 9.0, s, m, q_start.to(where), slots.to(where), max_len=max(lens), **({"form": form} if form else {}))
+            module.matrix_memory_scan(o, div, ud, gd, bd, 9.0, s, m, q_start.to(where), slots.to(where), max_len=max(lens), **({"form": form} if form else {}), **more)
         else:
             for i in range(max(lens)):  # the i-th token of every sequence that has one
                 seqs = [k for k, L in enumerate(lens) if i < L]
@@ -125,9 +125,9 @@ def test_matrix_memory(sizes, dtype, form):
         return o, div, s, m
 
     want = run(ref, "cpu")
-    got = run(ops, "cuda", form)
-    for a, b, what in zip(got, want, ("o", "divisor", "state", "top")):
-        _close(a, b, 2e-5, what)
+    for more in ({},) if form == "walk" else ({}, {"segments": 1}, {"segments": 2}, {"segments": 7}):  # (seven: more than a sequence has tiles)
+        for a, b, what in zip(run(ops, "cuda", form, **more), want, ("o", "divisor", "state", "top")):
+            _close(a, b, 2e-5, f"{what} {more}")
     if form == "walk":
         for a, b, what in zip(run(ops, "cuda", one_by_one=True), want, ("o", "divisor", "state", "top")):
             _close(a, b, 2e-5, f"token by token: {what}")
@@ -142,14 +142,15 @@ def test_matrix_memory_with_gates_at_their_extremes():
     gates[50:120, heads:] = -60.0
     q_start, slots = _i32([0, n]), _i32([2])
     out = []
-    for module, where in ((ref, "cpu"), (ops, "cuda")):
+    for module, where, more in ((ref, "cpu", {}), (ops, "cuda", {"segments": 1}), (ops, "cuda", {"segments": 3}), (ops, "cuda", {"form": "walk"})):
         o, div = torch.zeros(n, heads * dv, device=where), torch.zeros(n, heads, device=where)
         s, m = state.clone().to(where), top.clone().to(where)
-        module.matrix_memory_scan(o, div, u.to(where), gates.to(where), bias.to(where), 15.0, s, m, q_start.to(where), slots.to(where), max_len=n)
+        module.matrix_memory_scan(o, div, u.to(where), gates.to(where), bias.to(where), 15.0, s, m, q_start.to(where), slots.to(where), max_len=n, **more)
         out.append((o.view(n, heads, dv) / div[:, :, None], m, s))
-    for a, b, what in zip(out[1], out[0], ("o / divisor", "top", "state")):
-        assert torch.isfinite(a).all()
-        _close(a, b, 1e-3, what)
+    for got in out[1:]:
+        for a, b, what in zip(got, out[0], ("o / divisor", "top", "state")):
+            assert torch.isfinite(a).all()
+            _close(a, b, 1e-3, what)
 
 
 @pytest.mark.parametrize("dtype,tol", DTYPES)
