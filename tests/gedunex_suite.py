@@ -64,8 +64,8 @@ CONFIGS = {
                      attention(heads=2, kv_heads=2, dim=8, vdim=8, window=5)]),
     "memory_first": config([memory(heads=1, dim=20, vdim=7, cap=4.0), attention(v_mix=False, window=None, temp=None), attention(heads=8, kv_heads=4, dim=16, vdim=24, scale=0.8),
                             attention(heads=4, kv_heads=4, dim=32, vdim=24, softcap=None)], mlps=(None, dense(32), moe(ff=16, experts=4, top=1)), width=40, eps=1e-6),
-    "no_mixing": config([attention(v_mix=False), memory(heads=4, dim=16, vdim=16), attention(heads=4, kv_heads=1, dim=64, vdim=48, scale=0.15, softcap=20.0, v_mix=False)],
-                        mlps=(moe(ff=64, experts=12, top=4), None), width=64, vocab=130, scale=1.0),
+    "no_mixing": config([attention(v_mix=False), memory(heads=4, dim=16, vdim=16), attention(heads=6, kv_heads=2, dim=64, vdim=40, scale=0.15, softcap=18.0, v_mix=False)],
+                        mlps=(moe(ff=64, experts=10, top=4), None), width=64, vocab=130, scale=1.0),
     "only_attention": config([attention(temp=(1.5, 1)), attention(heads=3, kv_heads=1, dim=16, vdim=16, temp=(0.2, 7.5)), attention(heads=12, kv_heads=2, dim=24, vdim=8, window=70)],
                              mlps=(moe(ff=24, experts=5, top=5),), vocab=61),
     "only_memory": config([memory(), memory(heads=2, dim=40, vdim=33, cap=2.0), memory(heads=5, dim=8, vdim=8, cap=30.0)], mlps=(dense(64), None)),
@@ -182,7 +182,7 @@ def case_each_mechanism_alone(tmp_path, device, dtype):
         "cap": attention(softcap=2.0, window=None, temp=None, v_mix=False, scale=1.5),
         "window": attention(softcap=None, window=6, temp=None, v_mix=False),
         "temperature": attention(softcap=None, window=None, temp=(2.0, 3), v_mix=False),
-        "rows_64": attention(heads=4, kv_heads=1, dim=56, vdim=64, scale=0.2, window=30),
+        "rows_64": attention(heads=5, kv_heads=1, dim=56, vdim=64, scale=0.2, window=30),
         "rows_64_many_heads": attention(heads=20, kv_heads=1, dim=64, vdim=32, scale=0.2, window=25),
         "rows_128": attention(heads=4, kv_heads=2, dim=128, vdim=120, scale=0.1, window=None),
         "rows_128_capless": attention(heads=2, kv_heads=2, dim=128, vdim=128, scale=0.1, softcap=None),

@@ -95,7 +95,7 @@ def _memory_inputs(dtype, heads, d, dv, n, seed=7):
 
 @pytest.mark.parametrize("form", ["walk", "chunk"])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("sizes", [(4, 12, 10), (2, 32, 32), (3, 9, 7), (2, 48, 64), (2, 128, 128), (1, 136, 40), (2, 64, 63), (1, 256, 48), (2, 16, 130), (1, 24, 15), (1, 40, 16)])
+@pytest.mark.parametrize("sizes", [(4, 12, 10), (2, 32, 32), (3, 9, 7), (2, 48, 56), (2, 128, 128), (1, 136, 40), (2, 64, 63), (1, 256, 48), (2, 16, 130), (1, 24, 15), (1, 40, 16)])
 def test_matrix_memory(sizes, dtype, form):
     """Portions of 1, 70, 3, 128 and 33 tokens from states that are not zero, in scattered slots; the state afterwards; then the
     same tokens one at a time.  Both forms are float32 in effect, whatever the inputs' dtype: the tolerances are float32's."""
@@ -155,7 +155,7 @@ def test_matrix_memory_with_gates_at_their_extremes():
 
 @pytest.mark.parametrize("dtype,tol", DTYPES)
 def test_router_by_softmax_over_the_chosen(dtype, tol):
-    for W, E, top in ((48, 6, 2), (64, 12, 3), (50, 7, 7), (128, 40, 6), (256, 16, 1), (32, 1, 1)):
+    for W, E, top in ((48, 6, 2), (64, 13, 3), (50, 7, 7), (128, 40, 6), (256, 16, 1), (32, 1, 1)):
         router, bias = _rand(E, W, seed=1, scale=2.0 / W**0.5), _rand(E, seed=2)
         for n in (1, 5, 300):
             x = _rand(n, W, seed=10 + n).to(dtype)
@@ -211,7 +211,7 @@ def _paged_batch(nh, nkv, d, dtype, page, lens, kv, seed):
 
 @pytest.mark.parametrize("bend", ["cap and slopes", "slopes", "cap"])
 @pytest.mark.parametrize("window", [None, 64, 150])
-@pytest.mark.parametrize("dtype,d,heads", [(torch.float32, 24, (4, 2)), (torch.bfloat16, 48, (4, 2)), (torch.bfloat16, 64, (4, 1)), (torch.bfloat16, 64, (20, 1)),
+@pytest.mark.parametrize("dtype,d,heads", [(torch.float32, 24, (4, 2)), (torch.bfloat16, 48, (4, 2)), (torch.bfloat16, 64, (5, 1)), (torch.bfloat16, 64, (20, 1)),
                                            (torch.bfloat16, 96, (6, 3)), (torch.bfloat16, 128, (4, 2)), (torch.bfloat16, 128, (3, 3)), (torch.bfloat16, 20, (2, 1))])
 def test_bent_scores_in_every_attention_kernel(dtype, d, heads, window, bend):
     """A soft cap that bites, slopes from steep to nearly flat, a sink per head, over portions and single tokens, with and without
