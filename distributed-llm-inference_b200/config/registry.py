@@ -15,6 +15,7 @@ from typing import Any, Callable
 from .gedunex import GedunexConfig, gedunex_model_spec
 from .llama import LlamaConfig, UnsupportedModelError, llama_model_spec
 from .lokolorn import LokolornConfig, lokolorn_model_spec
+from .novunex import NovunexConfig, novunex_model_spec
 from .pazenex import PazenexConfig, pazenex_model_spec
 from .pokadra import PokadraConfig, pokadra_model_spec
 from .spec import ModelSpec
@@ -68,3 +69,4 @@ register_architecture(Architecture("Sugonex", SugonexConfig.from_dict, sugonex_m
 register_architecture(Architecture("Pokadra", PokadraConfig.from_dict, pokadra_model_spec))
 register_architecture(Architecture("Lokolorn", LokolornConfig.from_dict, lokolorn_model_spec))
 register_architecture(Architecture("Gedunex", GedunexConfig.from_dict, gedunex_model_spec))
+register_architecture(Architecture("Novunex", NovunexConfig.from_dict, novunex_model_spec))

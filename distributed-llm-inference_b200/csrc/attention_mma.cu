@@ -1,5 +1,5 @@
 // Paged causal GQA attention in bfloat16 on tensor cores, for one head size (-DHEAD_DIM=...,
-// a multiple of 16 up to 256).  One kernel serves prompt portions and single decoded tokens:
+// a multiple of 16 up to 256) and, where values have a size of their own, one value size (-DVALUE_DIM=..., likewise).  One kernel serves prompt portions and single decoded tokens:
 //
 //   * a CTA owns a tile of up to 64 rows; a row is one (token, query head) pair, and all rows
 //     of a tile share one KV head, so a key/value tile fetched once serves the whole GQA group;
@@ -26,30 +26,38 @@
 #error "compile with -DHEAD_DIM=<multiple of 16>"
 #endif
 
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+
 using namespace dli;
 typedef __nv_bfloat16 bf16;
 
 namespace {
 
 constexpr int D = HEAD_DIM;
+constexpr int DV = VALUE_DIM;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head size must be a multiple of 16 up to 256");
+static_assert(DV % 16 == 0 && DV >= 16 && DV <= 256, "value size must be a multiple of 16 up to 256");
 constexpr int BLOCK_N = 64;             // keys per tile
 constexpr int NWARPS = 4;
 constexpr int BLOCK_M = 16 * NWARPS;    // rows per tile
 constexpr int THREADS = 32 * NWARPS;
 constexpr int CHUNKS = D / 8;           // 16-byte chunks per row
 constexpr int ROW_BYTES = D * 2 + 16;   // padded row
-constexpr int TILE_BYTES = BLOCK_N * ROW_BYTES;
+constexpr int VROW_BYTES = DV * 2 + 16;
+constexpr int TILE_BYTES = BLOCK_N * ROW_BYTES;    // keys
+constexpr int VTILE_BYTES = BLOCK_N * VROW_BYTES;  // values
 constexpr int STAGES = 2;
-constexpr int SMEM_BYTES = BLOCK_M * ROW_BYTES + 2 * STAGES * TILE_BYTES;
+constexpr int SMEM_BYTES = BLOCK_M * ROW_BYTES + STAGES * (TILE_BYTES + VTILE_BYTES);
 constexpr int SMEM_BYTES_SHARED = BLOCK_M * ROW_BYTES + STAGES * TILE_BYTES;  // one pool serves as keys and values
 
 struct Params {
-  bf16* out;                 // [n, nh * D]
+  bf16* out;                 // [n, nh * DV]
   const bf16* q;             // rows of q_stride elements; head h at column h * D
   long long q_stride;
   const bf16* k_pool;        // [pages, nkv, page_size, D]
-  const bf16* v_pool;
+  const bf16* v_pool;        // [pages, nkv, page_size, DV]
   const int* block_tables;   // [seqs, max_blocks]
   int max_blocks;
   const int* q_start;        // [seqs + 1]
@@ -61,7 +69,7 @@ struct Params {
   float sink_log2;           // score of a sink (a term of the denominator without a value) times log2(e); -inf: none
   const float* sink_heads;   // if not null: a sink score per query head (natural units), instead of sink_log2
   int tokens_per_tile, heads_per_chunk, head_chunks, splits;
-  float* part_acc;           // [n * nh, splits, D]   (splits > 1)
+  float* part_acc;           // [n * nh, splits, DV]   (splits > 1)
   float* part_ml;            // [n * nh, splits, 2]
 };
 
@@ -106,10 +114,49 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // `nthreads` threads take part, thread `t` of them.  When the 16-byte chunks of a row divide
 // the thread count, a thread keeps its chunk column and walks down the rows, stepping through
 // the block table without a division per copy.
+template <int ROWS, int WIDTH>
+__device__ __forceinline__ void load_rows(unsigned char* dst, const bf16* __restrict__ pool, const int* __restrict__ table, int base, int lo, int hi, int nkv,
+                                          int kvh, int page_size, int t, int nthreads) {
+  constexpr int C = WIDTH / 8, PITCH = WIDTH * 2 + 16;
+  if ((nthreads % C) == 0) {
+    const int step = nthreads / C;
+    const int c = t % C;
+    int r = t / C;
+    int key = base + r;
+    int blk = key / page_size, off = key - blk * page_size;
+    for (; r < ROWS; r += step) {
+      const bool ok = key >= lo && key < hi;
+      size_t src = 0;
+      if (ok) src = (((size_t)table[blk] * nkv + kvh) * page_size + off) * WIDTH + c * 8;
+      cp_async16(smem_u32(dst + r * PITCH + c * 16), pool + src, ok ? 16 : 0);
+      key += step;
+      off += step;
+      while (off >= page_size) { off -= page_size; ++blk; }
+    }
+  } else {
+    for (int idx = t; idx < ROWS * C; idx += nthreads) {
+      const int r = idx / C, c = idx - r * C;
+      const int key = base + r;
+      const bool ok = key >= lo && key < hi;
+      size_t src = 0;
+      if (ok) {
+        const int blk = key / page_size;
+        src = (((size_t)table[blk] * nkv + kvh) * page_size + (key - blk * page_size)) * WIDTH + c * 8;
+      }
+      cp_async16(smem_u32(dst + r * PITCH + c * 16), pool + src, ok ? 16 : 0);
+    }
+  }
+}
 template <int ROWS, bool SHARED = false>
 __device__ __forceinline__ void load_kv_tile(unsigned char* dK, unsigned char* dV, const bf16* __restrict__ k_pool,
                                              const bf16* __restrict__ v_pool, const int* __restrict__ table, int base, int lo, int hi,
                                              int nkv, int kvh, int page_size, int t, int nthreads) {
+  if (D != DV || SHARED) {
+    load_rows<ROWS, D>(dK, k_pool, table, base, lo, hi, nkv, kvh, page_size, t, nthreads);
+    if (!SHARED) load_rows<ROWS, DV>(dV, v_pool, table, base, lo, hi, nkv, kvh, page_size, t, nthreads);
+    return;
+  }
+  // rows of one size: one look-up and one address serve both copies
   if ((nthreads % CHUNKS) == 0) {
     const int step = nthreads / CHUNKS;
     const int c = t % CHUNKS;
@@ -121,7 +168,7 @@ __device__ __forceinline__ void load_kv_tile(unsigned char* dK, unsigned char* d
       size_t src = 0;
       if (ok) src = (((size_t)table[blk] * nkv + kvh) * page_size + off) * D + c * 8;
       cp_async16(smem_u32(dK + r * ROW_BYTES + c * 16), k_pool + src, ok ? 16 : 0);
-      if (!SHARED) cp_async16(smem_u32(dV + r * ROW_BYTES + c * 16), v_pool + src, ok ? 16 : 0);
+      cp_async16(smem_u32(dV + r * ROW_BYTES + c * 16), v_pool + src, ok ? 16 : 0);
       key += step;
       off += step;
       while (off >= page_size) { off -= page_size; ++blk; }
@@ -137,20 +184,20 @@ __device__ __forceinline__ void load_kv_tile(unsigned char* dK, unsigned char* d
         src = (((size_t)table[blk] * nkv + kvh) * page_size + (key - blk * page_size)) * D + c * 8;
       }
       cp_async16(smem_u32(dK + r * ROW_BYTES + c * 16), k_pool + src, ok ? 16 : 0);
-      if (!SHARED) cp_async16(smem_u32(dV + r * ROW_BYTES + c * 16), v_pool + src, ok ? 16 : 0);
+      cp_async16(smem_u32(dV + r * ROW_BYTES + c * 16), v_pool + src, ok ? 16 : 0);
     }
   }
 }
 
 // One tile of NK keys for the 16 rows of a warp: S = Q K^T, mask, online softmax, O += P V.
-// q16: the warp's 16 query rows; tK, tV: the tile's keys and values (rows of ROW_BYTES);
+// q16: the warp's 16 query rows; tK, tV: the tile's keys (rows of ROW_BYTES) and values (rows of VROW_BYTES);
 // base: position of the tile's first key; rvalid / rpos: validity and position of the two
 // rows this thread holds (lane / 4 and lane / 4 + 8).
 template <int NK>
 __device__ __forceinline__ void tile_update(const unsigned char* sQ, const unsigned char* tK, const unsigned char* tV, int base,
                                             const bool (&rvalid)[2], const int (&rpos)[2], int window, float scale_log2,
                                             const ScoreBend& bend, const float (&slope)[2], float (&m)[2], float (&l)[2],
-                                            float (&o)[D / 8][4], int lane) {
+                                            float (&o)[DV / 8][4], int lane) {
   // ---- S = Q K^T
   float sc[NK / 8][4];
 #pragma unroll
@@ -210,7 +257,7 @@ __device__ __forceinline__ void tile_update(const unsigned char* sQ, const unsig
     }
   }
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j) {
+  for (int j = 0; j < DV / 8; ++j) {
     o[j][0] *= corr[0]; o[j][1] *= corr[0];
     o[j][2] *= corr[1]; o[j][3] *= corr[1];
   }
@@ -224,11 +271,11 @@ __device__ __forceinline__ void tile_update(const unsigned char* sQ, const unsig
     a[2] = pack_bf16(sc[2 * kk + 1][0], sc[2 * kk + 1][1]);
     a[3] = pack_bf16(sc[2 * kk + 1][2], sc[2 * kk + 1][3]);
 #pragma unroll
-    for (int jp = 0; jp < D / 16; ++jp) {
+    for (int jp = 0; jp < DV / 16; ++jp) {
       uint32_t b[4];
       const int key = kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
       const int dim = jp * 16 + (lane >> 4) * 8;
-      ldmatrix_x4_trans(b, smem_u32(tV + key * ROW_BYTES + dim * 2));
+      ldmatrix_x4_trans(b, smem_u32(tV + key * VROW_BYTES + dim * 2));
       mma_bf16(o[2 * jp], a, b[0], b[1]);
       mma_bf16(o[2 * jp + 1], a, b[2], b[3]);
     }
@@ -282,7 +329,7 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
   }
 
   auto load_tile = [&](int stage, int t) {
-    load_kv_tile<BLOCK_N, SHARED>(sK + stage * TILE_BYTES, sV + stage * TILE_BYTES, p.k_pool, p.v_pool, table, t * BLOCK_N, lo, hi, p.nkv, kvh,
+    load_kv_tile<BLOCK_N, SHARED>(sK + stage * TILE_BYTES, sV + stage * VTILE_BYTES, p.k_pool, p.v_pool, table, t * BLOCK_N, lo, hi, p.nkv, kvh,
                                   p.page_size, tid, THREADS);
   };
 
@@ -307,9 +354,9 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
 
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F};
   float l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+  for (int j = 0; j < DV / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
   if (num_tiles > 0) load_tile(0, t_begin);
   cp_async_commit();
@@ -322,7 +369,7 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
     __syncthreads();
 
     if (warp_active)
-      tile_update<BLOCK_N>(sQ + warp * 16 * ROW_BYTES, sK + stage * TILE_BYTES, sV + stage * TILE_BYTES, (t_begin + it) * BLOCK_N,
+      tile_update<BLOCK_N>(sQ + warp * 16 * ROW_BYTES, sK + stage * TILE_BYTES, sV + stage * VTILE_BYTES, (t_begin + it) * BLOCK_N,
                            rvalid, rpos, p.window, p.scale_log2, p.bend, slope, m, l, o, lane);
     __syncthreads();  // the stage is overwritten by the load issued next iteration
   }
@@ -342,16 +389,16 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Para
     const size_t row = (size_t)(q0 + tok0 + tok) * p.nh + head0 + hd;  // (token, head) row of the batch
     if (p.splits == 1) {
       const float inv = 1.f / (l[rr] + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + hd), m[rr]));
-      bf16* dst = p.out + row * D;
+      bf16* dst = p.out + row * DV;
 #pragma unroll
-      for (int j = 0; j < D / 8; ++j) {
+      for (int j = 0; j < DV / 8; ++j) {
         const int dim = j * 8 + (lane & 3) * 2;
         *reinterpret_cast<__nv_bfloat162*>(dst + dim) = __floats2bfloat162_rn(o[j][2 * rr] * inv, o[j][2 * rr + 1] * inv);
       }
     } else {
-      float* dst = p.part_acc + (row * p.splits + split) * D;
+      float* dst = p.part_acc + (row * p.splits + split) * DV;
 #pragma unroll
-      for (int j = 0; j < D / 8; ++j) {
+      for (int j = 0; j < DV / 8; ++j) {
         const int dim = j * 8 + (lane & 3) * 2;
         *reinterpret_cast<float2*>(dst + dim) = make_float2(o[j][2 * rr], o[j][2 * rr + 1]);
       }
@@ -375,19 +422,21 @@ struct DecodeShape {
   static constexpr int STAGES = PIPE;
   static constexpr bool SHARED = ONE_POOL;            // the values are read from the keys' rows: no value stages
   static constexpr int TILE = KEYS * ROW_BYTES;
-  static constexpr int WARP = (ONE_POOL ? 1 : 2) * PIPE * TILE;  // K and V stages of one warp
-  static constexpr int MERGE = NWARPS * 16 * (D + 2) * 4;  // per warp: o[16][D], m[16], l[16]
+  static constexpr int VTILE = KEYS * VROW_BYTES;
+  static constexpr int WARP = PIPE * (TILE + (ONE_POOL ? 0 : VTILE));  // K and V stages of one warp
+  static constexpr int MERGE = NWARPS * 16 * (DV + 2) * 4;  // per warp: o[16][DV], m[16], l[16]
   static constexpr int SMEM = 16 * ROW_BYTES + (NWARPS * WARP > MERGE ? NWARPS * WARP : MERGE);
 };
 typedef DecodeShape<16, 2> DecodeMany;
-typedef DecodeShape<(D <= 128 ? 32 : 16), (D <= 64 ? 3 : 2)> DecodeFew;
+constexpr int WIDER = D > DV ? D : DV;
+typedef DecodeShape<(WIDER <= 128 ? 32 : 16), (WIDER <= 64 ? 3 : 2)> DecodeFew;
 typedef DecodeShape<16, 2, true> DecodeManyShared;
 typedef DecodeShape<(D <= 128 ? 32 : 16), (D <= 128 ? 3 : 2), true> DecodeFewShared;
 
 // grid (splits, sequences, kv heads * chunks of 16 query heads); every sequence brings one token.
 template <typename Shape>
 __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params p) {
-  constexpr int DEC_N = Shape::N, DEC_STAGES = Shape::STAGES, DEC_TILE_BYTES = Shape::TILE, DEC_WARP_BYTES = Shape::WARP;
+  constexpr int DEC_N = Shape::N, DEC_STAGES = Shape::STAGES, DEC_TILE_BYTES = Shape::TILE, DEC_VTILE_BYTES = Shape::SHARED ? Shape::TILE : Shape::VTILE, DEC_WARP_BYTES = Shape::WARP;
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(128) unsigned char smem[];
@@ -426,7 +475,7 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
   unsigned char* wK = sKV + warp * DEC_WARP_BYTES;
   unsigned char* wV = Shape::SHARED ? wK : wK + DEC_STAGES * DEC_TILE_BYTES;
   auto load_tile = [&](int stage, int t) {
-    load_kv_tile<DEC_N, Shape::SHARED>(wK + stage * DEC_TILE_BYTES, wV + stage * DEC_TILE_BYTES, p.k_pool, p.v_pool, table, t * DEC_N, lo, hi, p.nkv,
+    load_kv_tile<DEC_N, Shape::SHARED>(wK + stage * DEC_TILE_BYTES, wV + stage * DEC_VTILE_BYTES, p.k_pool, p.v_pool, table, t * DEC_N, lo, hi, p.nkv,
                                        kvh, p.page_size, lane, 32);
   };
 
@@ -441,9 +490,9 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
 #endif
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F};
   float l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+  for (int j = 0; j < DV / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
   // this warp's tiles: t_begin + warp, + NWARPS, ...
   const int my_tiles = (t_end - t_begin - warp + NWARPS - 1) / NWARPS;
@@ -458,7 +507,7 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
     cp_async_commit();
     cp_async_wait<DEC_STAGES - 1>();
     __syncwarp();
-    tile_update<DEC_N>(sQ, wK + stage * DEC_TILE_BYTES, wV + stage * DEC_TILE_BYTES, (t_begin + warp + it * NWARPS) * DEC_N, rvalid,
+    tile_update<DEC_N>(sQ, wK + stage * DEC_TILE_BYTES, wV + stage * DEC_VTILE_BYTES, (t_begin + warp + it * NWARPS) * DEC_N, rvalid,
                        rpos, p.window, p.scale_log2, p.bend, slope, m, l, o, lane);
     __syncwarp();  // the stage is overwritten by the load issued next iteration
   }
@@ -471,14 +520,14 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
 
   // ---- merge the four warps' partial results in shared memory
   __syncthreads();  // every warp is done with its key and value stages
-  float* mo = reinterpret_cast<float*>(sKV);          // [NWARPS][16][D]
-  float* mm = mo + NWARPS * 16 * D;                    // [NWARPS][16]
+  float* mo = reinterpret_cast<float*>(sKV);          // [NWARPS][16][DV]
+  float* mm = mo + NWARPS * 16 * DV;                    // [NWARPS][16]
   float* ml = mm + NWARPS * 16;                        // [NWARPS][16]
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
-    float* dst = mo + (warp * 16 + rows[rr]) * D;
+    float* dst = mo + (warp * 16 + rows[rr]) * DV;
 #pragma unroll
-    for (int j = 0; j < D / 8; ++j)
+    for (int j = 0; j < DV / 8; ++j)
       *reinterpret_cast<float2*>(dst + j * 8 + (lane & 3) * 2) = make_float2(o[j][2 * rr], o[j][2 * rr + 1]);
     if ((lane & 3) == 0) {
       mm[warp * 16 + rows[rr]] = m[rr];
@@ -486,8 +535,8 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
     }
   }
   __syncthreads();
-  for (int idx = tid; idx < nheads * D; idx += THREADS) {
-    const int r = idx / D, dcol = idx - r * D;
+  for (int idx = tid; idx < nheads * DV; idx += THREADS) {
+    const int r = idx / DV, dcol = idx - r * DV;
     float mx = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < NWARPS; ++w) mx = fmaxf(mx, mm[w * 16 + r]);
@@ -497,13 +546,13 @@ __global__ void __launch_bounds__(THREADS) paged_decode_mma_kernel(const Params 
       const float mw = mm[w * 16 + r];
       const float f = (mw == -CUDART_INF_F) ? 0.f : exp2f(mw - mx);
       L += ml[w * 16 + r] * f;
-      acc += mo[(w * 16 + r) * D + dcol] * f;
+      acc += mo[(w * 16 + r) * DV + dcol] * f;
     }
     const size_t row = (size_t)token * p.nh + head0 + r;
     if (p.splits == 1) {
-      p.out[row * D + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
+      p.out[row * DV + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
     } else {
-      p.part_acc[(row * p.splits + split) * D + dcol] = acc;
+      p.part_acc[(row * p.splits + split) * DV + dcol] = acc;
       if (dcol == 0) {
         p.part_ml[(row * p.splits + split) * 2] = mx;
         p.part_ml[(row * p.splits + split) * 2 + 1] = L;
@@ -529,13 +578,13 @@ __global__ void merge_splits_kernel(bf16* __restrict__ out, const float* __restr
   }
   L += sink_term(sink_of(sink_heads, sink_log2, (int)(row % nh)), mmax);
   const float inv = 1.f / L;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  for (int d = threadIdx.x; d < DV; d += blockDim.x) {
     float acc = 0.f;
     for (int i = 0; i < splits; ++i) {
       const float mi = ml[2 * i];
-      if (mi != -CUDART_INF_F) acc += part_acc[(row * splits + i) * D + d] * exp2f(mi - mmax);
+      if (mi != -CUDART_INF_F) acc += part_acc[(row * splits + i) * DV + d] * exp2f(mi - mmax);
     }
-    out[row * D + d] = __float2bfloat16_rn(acc * inv);
+    out[row * DV + d] = __float2bfloat16_rn(acc * inv);
   }
 }
 
@@ -543,7 +592,7 @@ __global__ void merge_splits_kernel(bf16* __restrict__ out, const float* __restr
 
 // One launch for the sequences [seq0, seq0 + num_seqs) of a batch, each of which brings at most
 // max_q_len tokens.  With splits > 1 every one of them must bring exactly one token; part_acc and
-// part_ml are scratch of (rows * splits * D) and (rows * splits * 2) floats, rows counted from
+// part_ml are scratch of (rows * splits * DV) and (rows * splits * 2) floats, rows counted from
 // token 0 of the batch up to the last token of these sequences.
 DLI_EXPORT int dli_paged_attention_mma(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                        const int* block_tables, int max_blocks, const int* q_start, const int* kv_len,
@@ -583,6 +632,7 @@ DLI_EXPORT int dli_paged_attention_mma(void* out, const void* q, long long q_str
   p.head_chunks = (G + p.heads_per_chunk - 1) / p.heads_per_chunk;
   p.tokens_per_tile = BLOCK_M / p.heads_per_chunk;
   p.splits = splits; p.part_acc = part_acc; p.part_ml = part_ml;
+  if (D != DV && k_pool == v_pool) return DLI_ERR_UNSUPPORTED;
   const bool one_pool = k_pool == v_pool;  // the values lie in the keys' rows: a tile is copied once and serves both products
   if (max_q_len == 1) {
     const dim3 grid(splits, num_seqs, nkv * ((G + 15) / 16));
@@ -606,7 +656,7 @@ DLI_EXPORT int dli_paged_attention_mma(void* out, const void* q, long long q_str
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   if (splits > 1) {
-    launch_pdl((merge_splits_kernel), dim3(num_seqs * nh), dim3(D < 128 ? 64 : 128), 0, stream, 1, (bf16*)out, part_acc, part_ml, first_row * nh, splits, p.sink_log2, sink_heads, nh);
+    launch_pdl((merge_splits_kernel), dim3(num_seqs * nh), dim3(DV < 128 ? 64 : 128), 0, stream, 1, (bf16*)out, part_acc, part_ml, first_row * nh, splits, p.sink_log2, sink_heads, nh);
     e = cudaGetLastError();
   }
   return (int)e;
@@ -633,7 +683,7 @@ DLI_EXPORT int dli_paged_decode_attention_noalloc(void* out, const void* q, long
   if (splits < 1 || nh < 1 || first_row < 0) return DLI_ERR_UNSUPPORTED;
   // rows are counted from token 0 of the batch, as the ordinary entry point indexes its scratch
   const unsigned long long rows = (unsigned long long)(first_row + num_seqs) * (unsigned long long)nh;
-  const unsigned long long need = rows * (unsigned long long)splits * (unsigned long long)(D + 2);
+  const unsigned long long need = rows * (unsigned long long)splits * (unsigned long long)(DV + 2);
   if (need > DLI_NOALLOC_SCRATCH_FLOATS) return DLI_ERR_SCRATCH_TOO_SMALL;
 
   // set-up, once per device: the device address of the array, looked up with that device current
@@ -649,7 +699,7 @@ DLI_EXPORT int dli_paged_decode_attention_noalloc(void* out, const void* q, long
     base[dev] = p;
   }
   float* part_acc = base[dev];
-  float* part_ml = part_acc + rows * (unsigned long long)splits * (unsigned long long)D;
+  float* part_ml = part_acc + rows * (unsigned long long)splits * (unsigned long long)DV;
   if (splits == 1) part_acc = part_ml = nullptr;  // no partial results: the kernel writes the output itself
   return dli_paged_attention_mma(out, q, q_stride, k_pool, v_pool, block_tables, max_blocks, q_start, kv_len, seq0, num_seqs, 1,
                                  first_row, nh, nkv, page_size, window, scale, -INFINITY, nullptr, 0.f, nullptr, splits, part_acc, part_ml, stream);

@@ -1,5 +1,5 @@
 // What lies between an attention mixer's projections and its attention kernel when queries and keys are
-// normed over their whole projection, or when the keys and values are one cached latent; and what lies behind the
+// normed over their whole projection or head by head, or when the keys and values are one cached latent; and what lies behind the
 // attention kernel when its output is gated.
 // float32 and bfloat16 instantiations; all arithmetic is float32.
 #include "common.cuh"
@@ -8,24 +8,39 @@ using namespace dli;
 
 namespace {
 
-// One block per token.  proj row: q (nh * d columns) | k (nkv * d columns), then whatever else the product made.
-//   q <- q / rms(q over all nh * d) * wq,  k <- k / rms(k over all nkv * d) * wk      (normed != 0)
+// Norms of q and k before the rotation: none, over the whole projection (all heads together), or over each head.
+enum { NORM_NONE = 0, NORM_PROJECTION = 1, NORM_HEAD = 2 };
+
+struct QkStoreArgs {
+  long long proj_stride;
+  const float* wq;  // NORM_PROJECTION: nh * d and nkv * d numbers; NORM_HEAD: d numbers each
+  const float* wk;
+  float eps;
+  const int* positions;
+  const float* inv_freq;
+  const int* slots;
+  int nh, nkv, d, dv;  // heads; size of a query or key, of a value
+  int kd, vd;          // rows as they leave (kd >= d, vd >= dv, padded with zeros)
+  int rot, page_size, write_kv, norm, values_from_keys;
+};
+
+// One block per token.  proj row: q (nh * d columns) | k (nkv * d columns) | v (nkv * dv columns), then whatever else the product
+// made; without write_kv only q is read.
+//   q <- q / rms(q) * wq,  k <- k / rms(k) * wk      (rms over what `norm` says)
 //   rotary (rotate-half pairing, first `rot` dimensions of each head, angle float32(position) * inv_freq[i])
-//   q -> q_out [n, nh * d];  k -> k_pool at the token's slot;
-//   v_pool gets the keys as projected (values_from_keys != 0) or the nkv * d columns behind k.
+//   q -> q_out [n, nh, kd];  k -> k_pool at the token's slot;
+//   v_pool gets the keys as projected (values_from_keys != 0; dv = d) or the nkv * dv columns behind k.
 template <typename T>
-__global__ void qk_norm_rotary_store_kernel(T* __restrict__ q_out, const T* __restrict__ proj, long long proj_stride,
-                                            const float* __restrict__ wq, const float* __restrict__ wk, float eps,
-                                            const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                            const int* __restrict__ slots, T* __restrict__ k_pool, T* __restrict__ v_pool, int nh,
-                                            int nkv, int d, int rot, int page_size, int write_kv, int normed, int values_from_keys) {
+__global__ void qk_norm_rotary_store_kernel(T* __restrict__ q_out, const T* __restrict__ proj, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                                            const QkStoreArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float row[];  // (nh + nkv) * d
+  extern __shared__ float row[];  // (nh + nkv) * d | 1 / rms of every head (NORM_HEAD)
   __shared__ float red[33];
-  const int t = blockIdx.x;
-  const int nq = nh * d, nk = nkv * d;
-  const T* src = proj + (size_t)t * proj_stride;
+  const int t = blockIdx.x, nh = a.nh, nkv = a.nkv, d = a.d;
+  const int nq = nh * d, nk = a.write_kv ? nkv * d : 0;
+  float* head_r = row + (nh + nkv) * d;
+  const T* src = proj + (size_t)t * a.proj_stride;
   float sq = 0.f, sk = 0.f;
   for (int e = threadIdx.x; e < nq + nk; e += blockDim.x) {
     const float x = to_float(src[e]);
@@ -33,65 +48,80 @@ __global__ void qk_norm_rotary_store_kernel(T* __restrict__ q_out, const T* __re
     if (e < nq) sq = fmaf(x, x, sq); else sk = fmaf(x, x, sk);
   }
   float rq = 1.f, rk = 1.f;
-  if (normed) {
-    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
-    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+  if (a.norm == NORM_PROJECTION) {
+    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
+    if (nk) rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
   } else {
     __syncthreads();
-  }
-  const float pos = (float)positions[t];
-  const int half = rot >> 1;
-  long long kv_base = 0;
-  if (write_kv) {
-    const int slot = slots[t];
-    kv_base = ((long long)(slot / page_size) * nkv * page_size + slot % page_size) * d;  // + kvh * page_size * d + i
-  }
-  for (int e = threadIdx.x; e < nq + nk; e += blockDim.x) {
-    const bool is_q = e < nq;
-    if (!is_q && !write_kv) continue;
-    const int c = is_q ? e : e - nq;          // column inside q or k
-    const int head = c / d, i = c - head * d;
-    const float r = is_q ? rq : rk;
-    const float* w = is_q ? wq : wk;
-    float x = row[e] * r * (normed ? w[c] : 1.f);
-    if (i < rot) {
-      const int j = i < half ? i : i - half;
-      const int pe = i < half ? e + half : e - half, pc = i < half ? c + half : c - half;
-      const float xp = row[pe] * r * (normed ? w[pc] : 1.f);
-      float sn, cs;
-      sincosf(pos * inv_freq[j], &sn, &cs);
-      x = i < half ? x * cs - xp * sn : x * cs + xp * sn;
+    if (a.norm == NORM_HEAD) {
+      for (int head = threadIdx.x >> 5; head < (nq + nk) / d; head += blockDim.x >> 5) {
+        float ss = 0.f;
+        for (int i = threadIdx.x & 31; i < d; i += 32) ss = fmaf(row[head * d + i], row[head * d + i], ss);
+        ss = warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) head_r[head] = 1.f / sqrtf(ss / (float)d + a.eps);
+      }
+      __syncthreads();
     }
-    if (is_q) {
-      q_out[(size_t)t * nq + c] = from_float<T>(x);
-    } else {
-      const long long at = kv_base + (long long)head * page_size * d + i;
-      k_pool[at] = from_float<T>(x);
-      v_pool[at] = values_from_keys ? src[e] : src[e + nk];
+  }
+  const float pos = (float)a.positions[t];
+  const int half = a.rot >> 1;
+  const int slot = a.write_kv ? a.slots[t] : 0;
+  const long long page = slot / a.page_size;
+  const int off = slot % a.page_size;
+  for (int e = threadIdx.x; e < (nq + nk) / d * a.kd; e += blockDim.x) {
+    const int head = e / a.kd, i = e - head * a.kd;
+    const bool is_q = head < nh;
+    const int hh = is_q ? head : head - nh;
+    float x = 0.f;
+    if (i < d) {
+      const float r = a.norm == NORM_HEAD ? head_r[head] : is_q ? rq : rk;
+      const float* w = (is_q ? a.wq : a.wk) + (a.norm == NORM_PROJECTION ? hh * d : 0);
+      const float* h = row + head * d;
+      x = h[i] * r * (a.norm ? w[i] : 1.f);
+      if (i < a.rot) {
+        const int j = i < half ? i : i - half, other = i < half ? i + half : i - half;
+        const float xp = h[other] * r * (a.norm ? w[other] : 1.f);
+        float sn, cs;
+        sincosf(pos * a.inv_freq[j], &sn, &cs);
+        x = i < half ? x * cs - xp * sn : x * cs + xp * sn;
+      }
     }
+    if (is_q) q_out[((size_t)t * nh + hh) * a.kd + i] = from_float<T>(x);
+    else k_pool[((page * nkv + hh) * a.page_size + off) * a.kd + i] = from_float<T>(x);
+  }
+  if (!a.write_kv) return;
+  const T* vsrc = src + nq + (a.values_from_keys ? 0 : nk);
+  for (int e = threadIdx.x; e < nkv * a.vd; e += blockDim.x) {
+    const int hh = e / a.vd, i = e - hh * a.vd;
+    v_pool[((page * nkv + hh) * a.page_size + off) * a.vd + i] = i < a.dv ? vsrc[hh * a.dv + i] : from_float<T>(0.f);
   }
 }
 
-// The same with 16-byte accesses, for d % 8 == 0, rot % 16 == 0 and 16-byte aligned rows.  A work item is a run of
+template <typename T>
+__device__ __forceinline__ void copy8(T* dst, const T* src) {
+#pragma unroll
+  for (int i = 0; i < (int)(8 * sizeof(T) / 16); ++i) reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+}
+
+// The same with 16-byte accesses, for d, dv, kd, vd % 8 == 0, rot % 16 == 0 and 16-byte aligned rows.  A work item is a run of
 // eight columns — together with its partner run, half the rotated span further, where it is rotated.  The token's
 // cosines and sines are computed once, in shared memory, not once per head.
 template <typename T>
-__global__ void qk_norm_rotary_store_vec_kernel(T* __restrict__ q_out, const T* __restrict__ proj, long long proj_stride,
-                                                const float* __restrict__ wq, const float* __restrict__ wk, float eps,
-                                                const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                                const int* __restrict__ slots, T* __restrict__ k_pool, T* __restrict__ v_pool, int nh,
-                                                int nkv, int d, int rot, int page_size, int write_kv, int normed, int values_from_keys) {
+__global__ void qk_norm_rotary_store_vec_kernel(T* __restrict__ q_out, const T* __restrict__ proj, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                                                const QkStoreArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float cs[];  // cos [rot / 2] | sin [rot / 2]
+  extern __shared__ float cs[];  // cos [rot / 2] | sin [rot / 2] | 1 / rms of every head (NORM_HEAD)
   __shared__ float red[33];
-  const int t = blockIdx.x;
-  const int nq = nh * d, nk = nkv * d, half = rot >> 1;
-  const T* src = proj + (size_t)t * proj_stride;
-  const float pos = (float)positions[t];
-  for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &cs[half + j], &cs[j]);
+  const int t = blockIdx.x, nh = a.nh, nkv = a.nkv, d = a.d;
+  const int nq = nh * d, nk = a.write_kv ? nkv * d : 0, half = a.rot >> 1;
+  const int heads = nh + (a.write_kv ? nkv : 0);
+  float* head_r = cs + a.rot;
+  const T* src = proj + (size_t)t * a.proj_stride;
+  const float pos = (float)a.positions[t];
+  for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * a.inv_freq[j], &cs[half + j], &cs[j]);
   float rq = 1.f, rk = 1.f;
-  if (normed) {
+  if (a.norm == NORM_PROJECTION) {
     float sq = 0.f, sk = 0.f;
     for (int e = threadIdx.x * 8; e < nq + nk; e += blockDim.x * 8) {
       float x[8];
@@ -101,69 +131,88 @@ __global__ void qk_norm_rotary_store_vec_kernel(T* __restrict__ q_out, const T* 
       for (int k = 0; k < 8; ++k) ss = fmaf(x[k], x[k], ss);
       if (e < nq) sq += ss; else sk += ss;
     }
-    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
-    rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+    rq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
+    if (nk) rk = 1.f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
+  } else if (a.norm == NORM_HEAD) {
+    // a head belongs to `lanes` neighbouring lanes (a power of two), each of which sums runs of eight
+    const int runs = d >> 3;
+    int lanes = 1;
+    while (lanes < runs && lanes < 32) lanes <<= 1;
+    const int lane = threadIdx.x & (lanes - 1), step = blockDim.x / lanes;
+    for (int first = 0; first < heads; first += step) {  // every thread takes part in every round: the shuffles need whole warps
+      const int head = first + threadIdx.x / lanes;
+      float ss = 0.f;
+      if (head < heads)
+        for (int i = lane; i < runs; i += lanes) {
+          float x[8];
+          load8(src + head * d + i * 8, x);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) ss = fmaf(x[k], x[k], ss);
+        }
+      for (int off = lanes >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+      if (lane == 0 && head < heads) head_r[head] = 1.f / sqrtf(ss / (float)d + a.eps);
+    }
+    __syncthreads();
   } else {
     __syncthreads();
   }
-  long long kv_base = 0;
-  if (write_kv) {
-    const int slot = slots[t];
-    kv_base = ((long long)(slot / page_size) * nkv * page_size + slot % page_size) * d;
-  }
-  // items per head: half / 8 rotated pairs, then (d - rot) / 8 runs that pass unrotated
-  const int pair_items = half >> 3, per_head = pair_items + ((d - rot) >> 3);
-  const int heads = nh + (write_kv ? nkv : 0);
+  const int slot = a.write_kv ? a.slots[t] : 0;
+  const long long page = slot / a.page_size;
+  const int off = slot % a.page_size;
+  // items per head: half / 8 rotated pairs, (d - rot) / 8 runs that pass unrotated, (kd - d) / 8 runs of zeros
+  const int pair_items = half >> 3, data_items = pair_items + ((d - a.rot) >> 3), per_head = data_items + ((a.kd - d) >> 3);
   for (int item = threadIdx.x; item < heads * per_head; item += blockDim.x) {
     const int head = item / per_head, it = item - head * per_head;
     const bool is_q = head < nh;
     const int hh = is_q ? head : head - nh;
-    const float r = is_q ? rq : rk;
-    const float* w = (is_q ? wq : wk) + hh * d;
+    const float r = a.norm == NORM_HEAD ? head_r[head] : is_q ? rq : rk;
+    const float* w = (is_q ? a.wq : a.wk) + (a.norm == NORM_PROJECTION ? hh * d : 0);
     const T* hsrc = src + head * d;  // q heads, then k heads, lie back to back
-    T* dst = is_q ? q_out + (size_t)t * nq + hh * d : k_pool + kv_base + (long long)hh * page_size * d;
-    T* vdst = is_q ? nullptr : v_pool + kv_base + (long long)hh * page_size * d;
-    const T* vsrc = values_from_keys ? hsrc : hsrc + nk;
+    T* dst = is_q ? q_out + ((size_t)t * nh + hh) * a.kd : k_pool + ((page * nkv + hh) * a.page_size + off) * a.kd;
     if (it < pair_items) {
       const int i = it * 8;
       float lo[8], hi[8], wl[8], wh[8], ol[8], oh[8];
       load8(hsrc + i, lo);
       load8(hsrc + i + half, hi);
-      if (vdst) {
-        *reinterpret_cast<uint4*>(vdst + i) = *reinterpret_cast<const uint4*>(vsrc + i);
-        *reinterpret_cast<uint4*>(vdst + i + half) = *reinterpret_cast<const uint4*>(vsrc + i + half);
-        if (sizeof(T) == 4) {
-          *reinterpret_cast<uint4*>(vdst + i + 4) = *reinterpret_cast<const uint4*>(vsrc + i + 4);
-          *reinterpret_cast<uint4*>(vdst + i + half + 4) = *reinterpret_cast<const uint4*>(vsrc + i + half + 4);
-        }
-      }
-      if (normed) {
+      if (a.norm) {
         load8(w + i, wl);
         load8(w + i + half, wh);
       }
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
-        const float a = lo[k] * r * (normed ? wl[k] : 1.f), b = hi[k] * r * (normed ? wh[k] : 1.f);
+        const float u = lo[k] * r * (a.norm ? wl[k] : 1.f), v = hi[k] * r * (a.norm ? wh[k] : 1.f);
         const float c = cs[i + k], sn = cs[half + i + k];
-        ol[k] = a * c - b * sn;
-        oh[k] = b * c + a * sn;
+        ol[k] = u * c - v * sn;
+        oh[k] = v * c + u * sn;
       }
       store8(dst + i, ol);
       store8(dst + i + half, oh);
-    } else {
-      const int i = rot + (it - pair_items) * 8;
+    } else if (it < data_items) {
+      const int i = a.rot + (it - pair_items) * 8;
       float x[8], wv[8];
       load8(hsrc + i, x);
-      if (vdst) {
-        *reinterpret_cast<uint4*>(vdst + i) = *reinterpret_cast<const uint4*>(vsrc + i);
-        if (sizeof(T) == 4) *reinterpret_cast<uint4*>(vdst + i + 4) = *reinterpret_cast<const uint4*>(vsrc + i + 4);
-      }
-      if (normed) {
+      if (a.norm) {
         load8(w + i, wv);
 #pragma unroll
         for (int k = 0; k < 8; ++k) x[k] = x[k] * r * wv[k];
       }
       store8(dst + i, x);
+    } else {
+      const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      store8(dst + d + (it - data_items) * 8, zero);
+    }
+  }
+  if (!a.write_kv) return;
+  const T* vsrc = src + nq + (a.values_from_keys ? 0 : nk);
+  const int vper = a.vd >> 3;
+  for (int item = threadIdx.x; item < nkv * vper; item += blockDim.x) {
+    const int hh = item / vper, i = (item - hh * vper) * 8;
+    T* dst = v_pool + ((page * nkv + hh) * a.page_size + off) * a.vd + i;
+    if (i < a.dv) {
+      copy8(dst, vsrc + hh * a.dv + i);
+    } else {
+      const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      store8(dst, zero);
     }
   }
 }
@@ -201,53 +250,49 @@ __global__ void sigmoid_gate_kernel(T* __restrict__ out, const T* __restrict__ g
 
 DLI_EXPORT int dli_qk_norm_rotary_store(void* q_out, const void* proj, long long proj_stride, const float* wq, const float* wk,
                                         float eps, const int* positions, const float* inv_freq, const int* slots, void* k_pool,
-                                        void* v_pool, int n, int nh, int nkv, int d, int rot, int page_size, int write_kv,
-                                        int normed, int values_from_keys, int dtype, cudaStream_t stream) {
+                                        void* v_pool, int n, int nh, int nkv, int d, int dv, int kd, int vd, int rot, int page_size, int write_kv,
+                                        int norm, int values_from_keys, int dtype, cudaStream_t stream) {
   if (n == 0) return 0;
-  const size_t smem = (size_t)(nh + nkv) * d * sizeof(float);
-  if (nh < 1 || nkv < 1 || d < 1 || rot < 0 || rot > d || (rot & 1) || smem > 200 * 1024 || (rot && !inv_freq) ||
-      (normed && (!wq || !wk)) || (write_kv && (!slots || !k_pool || !v_pool)))
+  const size_t smem = ((size_t)(nh + nkv) * d + nh + nkv) * sizeof(float);
+  if (nh < 1 || nkv < 1 || d < 1 || dv < 1 || kd < d || vd < dv || rot < 0 || rot > d || (rot & 1) || page_size < 1 || smem > 200 * 1024 ||
+      (rot && !inv_freq) || norm < NORM_NONE || norm > NORM_HEAD || (norm && (!wq || (write_kv && !wk))) || (values_from_keys && dv != d) ||
+      (write_kv && (!slots || !k_pool || !v_pool)))
     return DLI_ERR_UNSUPPORTED;
+  const QkStoreArgs a{proj_stride, wq, wk, eps, positions, inv_freq, slots, nh, nkv, d, dv, kd, vd, rot, page_size, write_kv, norm, values_from_keys};
   const int threads = (nh + nkv) * d >= 2048 ? 512 : 256;
-  cudaError_t e;
   const size_t esize = dtype == DLI_F32 ? 4 : 2;
-  const bool aligned = (d % 8) == 0 && (rot % 16) == 0 && (proj_stride % 8) == 0 && rot * sizeof(float) <= 48 * 1024 &&
+  const size_t vsmem = ((size_t)rot + nh + nkv) * sizeof(float);
+  const bool aligned = (d % 8) == 0 && (dv % 8) == 0 && (kd % 8) == 0 && (vd % 8) == 0 && (rot % 16) == 0 && (proj_stride % 8) == 0 && vsmem <= 47 * 1024 &&
                        (((uintptr_t)q_out | (uintptr_t)proj | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0 &&
                        ((size_t)d * esize) % 16 == 0;
   if (aligned) {
     const int items = (nh + nkv) * (d / 8);
     const int vt = items >= 256 ? 256 : (items >= 128 ? 128 : 64);
-    const size_t vsmem = (size_t)rot * sizeof(float);
     if (dtype == DLI_F32)
-      e = launch_pdl((qk_norm_rotary_store_vec_kernel<float>), dim3(n), dim3(vt), vsmem, stream, 1, (float*)q_out, (const float*)proj,
-                     proj_stride, wq, wk, eps, positions, inv_freq, slots, (float*)k_pool, (float*)v_pool, nh, nkv, d, rot, page_size,
-                     write_kv, normed, values_from_keys);
-    else
-      e = launch_pdl((qk_norm_rotary_store_vec_kernel<__nv_bfloat16>), dim3(n), dim3(vt), vsmem, stream, 1, (__nv_bfloat16*)q_out,
-                     (const __nv_bfloat16*)proj, proj_stride, wq, wk, eps, positions, inv_freq, slots, (__nv_bfloat16*)k_pool,
-                     (__nv_bfloat16*)v_pool, nh, nkv, d, rot, page_size, write_kv, normed, values_from_keys);
-    return (int)e;
+      return (int)launch_pdl((qk_norm_rotary_store_vec_kernel<float>), dim3(n), dim3(vt), vsmem, stream, 1, (float*)q_out, (const float*)proj, (float*)k_pool,
+                             (float*)v_pool, a);
+    return (int)launch_pdl((qk_norm_rotary_store_vec_kernel<__nv_bfloat16>), dim3(n), dim3(vt), vsmem, stream, 1, (__nv_bfloat16*)q_out,
+                           (const __nv_bfloat16*)proj, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, a);
   }
+  cudaError_t e;
   if (dtype == DLI_F32) {
     static MaxPerDevice set;
-    if ((int)smem > 48 * 1024 && set.here() < (int)smem) {
+    if ((int)smem > 47 * 1024 && set.here() < (int)smem) {
       e = cudaFuncSetAttribute(qk_norm_rotary_store_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
       set.here() = (int)smem;
     }
-    e = launch_pdl((qk_norm_rotary_store_kernel<float>), dim3(n), dim3(threads), smem, stream, 1, (float*)q_out, (const float*)proj,
-                   proj_stride, wq, wk, eps, positions, inv_freq, slots, (float*)k_pool, (float*)v_pool, nh, nkv, d, rot, page_size,
-                   write_kv, normed, values_from_keys);
+    e = launch_pdl((qk_norm_rotary_store_kernel<float>), dim3(n), dim3(threads), smem, stream, 1, (float*)q_out, (const float*)proj, (float*)k_pool,
+                   (float*)v_pool, a);
   } else {
     static MaxPerDevice set;
-    if ((int)smem > 48 * 1024 && set.here() < (int)smem) {
+    if ((int)smem > 47 * 1024 && set.here() < (int)smem) {
       e = cudaFuncSetAttribute(qk_norm_rotary_store_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
       set.here() = (int)smem;
     }
     e = launch_pdl((qk_norm_rotary_store_kernel<__nv_bfloat16>), dim3(n), dim3(threads), smem, stream, 1, (__nv_bfloat16*)q_out,
-                   (const __nv_bfloat16*)proj, proj_stride, wq, wk, eps, positions, inv_freq, slots, (__nv_bfloat16*)k_pool,
-                   (__nv_bfloat16*)v_pool, nh, nkv, d, rot, page_size, write_kv, normed, values_from_keys);
+                   (const __nv_bfloat16*)proj, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, a);
   }
   return (int)e;
 }

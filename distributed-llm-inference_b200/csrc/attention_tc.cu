@@ -1,5 +1,5 @@
 // Paged causal GQA attention for prompt portions on the fifth-generation tensor cores
-// (bfloat16, head size 64 — and 128 in the kernel with a thread per row —, page sizes 8..128 that divide 128).
+// (bfloat16; head sizes up to 64 or 128, for keys and values each, in multiples of 8; page sizes 8..128 that divide 128).
 //
 // A CTA owns 128 rows — (token, query head) pairs that share one KV head — and walks the keys
 // of its sequence in tiles of 128:
@@ -13,6 +13,10 @@
 //   * O += P V is a second group of tcgen05.mma (V is the MN-major operand, exactly as it lies in
 //     the pages), accumulated in tensor memory over all tiles; the threads rescale it in place only
 //     when a row's maximum has grown by more than 2^8, and read it once, at the end.
+//
+// That is the kernel for keys and values of 64 numbers; the one with a thread per row (below) takes keys and values of up to 128,
+// of sizes of their own: shared memory holds whole 128-byte slabs of 64 columns, and the columns that a pool's rows do not have
+// are zeros that TMA fills in, so that only what is stored crosses from memory.
 //
 // One warp issues the copies, one the matrix products; they meet each other and the softmax threads on
 // mbarriers only.  Keys, values, scores and probabilities are double-buffered, so the tensor cores work
@@ -54,6 +58,7 @@ struct Params {
   float sink_log2;  // score of a sink (a term of the denominator without a value) times log2(e); -inf: none
   const float* sink_heads;  // if not null: a sink score per query head (natural units), instead of sink_log2
   int tokens_per_tile, heads_per_chunk, head_chunks;
+  int d, dv;  // columns of a key and of a value row (the kernel with a thread per row; the other's are 64)
   int* error_flag;
 };
 
@@ -479,18 +484,22 @@ __global__ void __launch_bounds__(THREADS, 1) paged_prefill_tc_kernel(const __gr
 //   k_full, v_full [2]     TMA -> products              k_free, v_free [2]   products done -> TMA
 //   s_done [A, B]          S there                      s_read [A, B] (128)  S in registers
 //   p_ready [A, B] (128)   P written, output rescaled   o_done [A, B]        O += P V finished
-// Head size 64: two query tiles per CTA.  Head size 128: one (its Q, K and V tiles are twice as large), so the
-// group has no partner; a row of keys or values is then two 128-byte slabs, each with its own TMA box, the
-// score product runs over both, and the output product is one group of tcgen05.mma per slab of 64 columns.
-template <int HD>
+// HD and HV: keys' and values' columns as they lie in shared memory, whole 128-byte slabs of 64, each with its own TMA box; the
+// score product runs over the slabs of the keys, and the output product is one group of tcgen05.mma per slab of the values.
+// p.d and p.dv are the pools' columns (and those of the queries and of the output): at most HD and HV, multiples of 8; TMA fills what
+// lies beyond them with zeros.  Two query tiles per CTA, unless both are 128: then one (Q, K and V tiles are twice as large), and the
+// group has no partner.
+template <int HD, int HV>
 struct T2Cfg {
-  static_assert(HD == 64 || HD == 128, "head sizes with whole 128-byte slabs");
-  static constexpr int QT = HD == 64 ? 2 : 1;             // query tiles per CTA
-  static constexpr int SLABS = HD / 64;
+  static_assert((HD == 64 || HD == 128) && (HV == 64 || HV == 128), "head sizes with whole 128-byte slabs");
+  static constexpr int QT = HD == 64 || HV == 64 ? 2 : 1;  // query tiles per CTA
+  static constexpr int SLABS = HD / 64, VSLABS = HV / 64;
   static constexpr int THREADS = QT * ROWS + 128;         // softmax warpgroups and one whose warps issue the products (one per query tile) and the copies (keys, values)
-  static constexpr int KV_BYTES = SLABS * TILE_BYTES;     // one stage of keys or of values; also one Q tile
-  static constexpr int SMEM = QT * KV_BYTES + 4 * KV_BYTES + QT * 2 * TILE_BYTES + 256 + 1024;  // Q, K x2, V x2, P per query tile, barriers, alignment
-  static constexpr int TMEM = QT * KEYS + QT * HD <= 256 ? 256 : 512;
+  static constexpr int K_BYTES = SLABS * TILE_BYTES;      // one stage of keys; also one Q tile
+  static constexpr int V_BYTES = VSLABS * TILE_BYTES;     // one stage of values
+  static constexpr int SMEM = QT * K_BYTES + 2 * K_BYTES + 2 * V_BYTES + QT * 2 * TILE_BYTES + 256 + 1024;  // Q, K x2, V x2, P per query tile, barriers, alignment
+  static_assert(SMEM <= 227 * 1024, "one CTA fits an SM");
+  static constexpr int TMEM = QT * KEYS + QT * HV <= 256 ? 256 : 512;
 };
 
 // Pairs of float32 in a 64-bit register, for the instructions that work on both at once (sm_100).
@@ -522,19 +531,19 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
   return d;
 }
 
-template <int HD>
-__global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k,
-                                                                                  const __grid_constant__ CUtensorMap map_v, const Params p) {
-  using Cfg = T2Cfg<HD>;
-  constexpr int QT = Cfg::QT, SLABS = Cfg::SLABS, KV_BYTES = Cfg::KV_BYTES, T2_THREADS = Cfg::THREADS;
+template <int HD, int HV>
+__global__ void __launch_bounds__(T2Cfg<HD, HV>::THREADS, 1) paged_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k,
+                                                                                      const __grid_constant__ CUtensorMap map_v, const Params p) {
+  using Cfg = T2Cfg<HD, HV>;
+  constexpr int QT = Cfg::QT, SLABS = Cfg::SLABS, VSLABS = Cfg::VSLABS, K_BYTES = Cfg::K_BYTES, V_BYTES = Cfg::V_BYTES, T2_THREADS = Cfg::THREADS;
   constexpr int D = HD;  // shadows the one-tile kernel's head size within this kernel
   pdl_launch_dependents();
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* sQ = smem;                     // tile A (, tile B); a tile is SLABS slabs of [128 rows x 128 bytes]
-  unsigned char* sK = sQ + QT * KV_BYTES;       // two stages
-  unsigned char* sV = sK + 2 * KV_BYTES;        // two stages
-  unsigned char* sP = sV + 2 * KV_BYTES;        // per query tile (keys 0..63 | keys 64..127)
+  unsigned char* sK = sQ + QT * K_BYTES;        // two stages
+  unsigned char* sV = sK + 2 * K_BYTES;         // two stages
+  unsigned char* sP = sV + 2 * V_BYTES;         // per query tile (keys 0..63 | keys 64..127)
   uint64_t* bars = (uint64_t*)(sP + QT * 2 * TILE_BYTES);
   uint32_t* tmem_slot = (uint32_t*)(bars + 16);
   volatile int* failed = (volatile int*)(tmem_slot + 1);
@@ -586,11 +595,11 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     const int rr = idx / (D / 8), c = idx - rr * (D / 8);  // rr: row among those of all tiles; c: 16-byte chunk of the row
     const int rt = rr & (ROWS - 1), tok = (rr >> 7) * tpt + rt / Gc, hd = rt % Gc;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (rt / Gc < tpt && tok < ntok && hd < nheads)
-      v = *reinterpret_cast<const uint4*>(p.q + (size_t)(q0 + tok0 + tok) * p.q_stride + (size_t)(head0 + hd) * D + c * 8);
-    *reinterpret_cast<uint4*>(sQ + (rr >> 7) * KV_BYTES + (c >> 3) * TILE_BYTES + rt * 128 + (((c & 7) ^ (rt & 7)) << 4)) = v;
+    if (rt / Gc < tpt && tok < ntok && hd < nheads && c * 8 < p.d)
+      v = *reinterpret_cast<const uint4*>(p.q + (size_t)(q0 + tok0 + tok) * p.q_stride + (size_t)(head0 + hd) * p.d + c * 8);
+    *reinterpret_cast<uint4*>(sQ + (rr >> 7) * K_BYTES + (c >> 3) * TILE_BYTES + rt * 128 + (((c & 7) ^ (rt & 7)) << 4)) = v;
   }
-  for (int idx = tid; idx < 2 * KV_BYTES / 16; idx += T2_THREADS) reinterpret_cast<uint4*>(sV)[idx] = make_uint4(0, 0, 0, 0);
+  for (int idx = tid; idx < 2 * V_BYTES / 16; idx += T2_THREADS) reinterpret_cast<uint4*>(sV)[idx] = make_uint4(0, 0, 0, 0);
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();
@@ -614,6 +623,7 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     const uint32_t full = keys ? k_full : v_full, freed = keys ? k_free : v_free;
     unsigned char* stage0 = keys ? sK : sV;
     const CUtensorMap* map = keys ? &map_k : &map_v;
+    const int slabs = keys ? SLABS : VSLABS, stage_bytes = keys ? K_BYTES : V_BYTES;
     auto lookup = [&](int t) -> int {
       const int first = t * KEYS + page_i * p.page_size;
       const bool need = lane < 16 && t < t_end && page_i < pages && first < hi && first + p.page_size > lo;
@@ -630,12 +640,12 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
         if (*failed) break;
       }
       const int count = __popc(__ballot_sync(0xffffffffu, cur >= 0));
-      if (lane == 0) mbar_expect_tx(full + 8 * st, (uint32_t)(count * p.page_size * 128 * SLABS));
+      if (lane == 0) mbar_expect_tx(full + 8 * st, (uint32_t)(count * p.page_size * 128 * slabs));
       __syncwarp();
       if (cur >= 0) {
 #pragma unroll
-        for (int sl = 0; sl < SLABS; ++sl)
-          tma_load_2d(smem_u32(stage0 + st * KV_BYTES + sl * TILE_BYTES + page_i * p.page_size * 128), map, sl * 64, (cur * p.nkv + kvh) * p.page_size, full + 8 * st);
+        for (int sl = 0; sl < (SLABS > VSLABS ? SLABS : VSLABS); ++sl)
+          if (sl < slabs) tma_load_2d(smem_u32(stage0 + st * stage_bytes + sl * TILE_BYTES + page_i * p.page_size * 128), map, sl * 64, (cur * p.nkv + kvh) * p.page_size, full + 8 * st);
       }
     }
   } else if (warp == QT * ROWS / 32 || (QT == 2 && warp == QT * ROWS / 32 + 2)) {
@@ -649,13 +659,14 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     const int q = warp == QT * ROWS / 32 ? 0 : 1;  // this thread's query tile
     if (lane == 0) {
       const uint32_t idesc_s = instr_desc(ROWS, KEYS, 0), idesc_o = instr_desc(ROWS, 64, 1);
-      const uint32_t qa = smem_u32(sQ + q * KV_BYTES), pa = smem_u32(sP + q * 2 * TILE_BYTES);
+      const int k_steps = (p.d + 15) >> 4;  // (the columns of a last half step are zeros)
+      const uint32_t qa = smem_u32(sQ + q * K_BYTES), pa = smem_u32(sP + q * 2 * TILE_BYTES);
       auto scores = [&](int t) {  // S_q(t) = Q_q K(t)^T
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t k = smem_u32(sK + (t & 1) * KV_BYTES);
+        const uint32_t k = smem_u32(sK + (t & 1) * K_BYTES);
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk)
-          umma(tmem_s + q * KEYS, smem_desc_sw128(qa + (kk >> 2) * TILE_BYTES + (kk & 3) * 32), smem_desc_sw128(k + (kk >> 2) * TILE_BYTES + (kk & 3) * 32), idesc_s, kk != 0);
+          if (kk < k_steps) umma(tmem_s + q * KEYS, smem_desc_sw128(qa + (kk >> 2) * TILE_BYTES + (kk & 3) * 32), smem_desc_sw128(k + (kk >> 2) * TILE_BYTES + (kk & 3) * 32), idesc_s, kk != 0);
         umma_commit(s_done + 8 * q);
         umma_commit(k_free + 8 * (t & 1));  // this tile's product with K(t) is issued
       };
@@ -671,12 +682,12 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
         ok = wait_or_fail(p_ready + 8 * q, t & 1, failed, 19, p.error_flag) && wait_or_fail(v_full + 8 * (t & 1), (t >> 1) & 1, failed, 20, p.error_flag);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t v = smem_u32(sV + (t & 1) * KV_BYTES);
+        const uint32_t v = smem_u32(sV + (t & 1) * V_BYTES);
 #pragma unroll
-        for (int sl = 0; sl < SLABS; ++sl)  // 64 output columns at a time: the values' slab is the MN-major operand
+        for (int sl = 0; sl < VSLABS; ++sl)  // 64 output columns at a time: the values' slab is the MN-major operand
 #pragma unroll
           for (int k = 0; k < KEYS / 16; ++k)
-            umma(tmem_o + q * D + sl * 64, smem_desc_sw128(pa + (k >> 2) * TILE_BYTES + (k & 3) * 32), smem_desc_sw128(v + sl * TILE_BYTES + k * 2048), idesc_o, (t | k) != 0);
+            umma(tmem_o + q * HV + sl * 64, smem_desc_sw128(pa + (k >> 2) * TILE_BYTES + (k & 3) * 32), smem_desc_sw128(v + sl * TILE_BYTES + k * 2048), idesc_o, (t | k) != 0);
         umma_commit(o_done + 8 * q);
         umma_commit(v_free + 8 * (t & 1));  // this tile's product with V(t) is issued
       }
@@ -692,7 +703,7 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     const bool rvalid = rtok < ntok && (r % Gc) < nheads && r / Gc < tpt;
     const int rpos = pos0 + rtok;
     const uint32_t lane_bits = (uint32_t)((warp & 3) * 32) << 16;
-    const uint32_t my_s = tmem_s + q * KEYS + lane_bits, my_o = tmem_o + q * D + lane_bits;
+    const uint32_t my_s = tmem_s + q * KEYS + lane_bits, my_o = tmem_o + q * HV + lane_bits;
     const uint32_t my_s_done = s_done + 8 * q, my_s_read = s_read + 8 * q, my_p_ready = p_ready + 8 * q, my_o_done = o_done + 8 * q;
     constexpr float RESCALE_STEP = 8.f;
     float m = -CUDART_INF_F, m_ref = -CUDART_INF_F, l = 0.f;
@@ -763,7 +774,7 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
           if (ok) {
 #pragma unroll
-            for (int c = 0; c < D; c += 32) {
+            for (int c = 0; c < HV; c += 32) {
               uint32_t v[32];
               tmem_ld32_nowait(my_o + c, v);
               asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -821,16 +832,17 @@ __global__ void __launch_bounds__(T2Cfg<HD>::THREADS, 1) paged_prefill_tc2_kerne
     const float inv = 1.f / (l + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + (r % Gc)), m_ref * p.scale_log2));
     const size_t row = (size_t)(q0 + tok0 + rtok) * p.nh + head0 + (r % Gc);
 #pragma unroll
-    for (int c = 0; c < D; c += 32) {
+    for (int c = 0; c < HV; c += 32) {
       uint32_t v[32];
       if (ok) {
         tmem_ld32_nowait(my_o + c, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       }
       if (ok && !*failed && rvalid) {
-        uint4* dst = reinterpret_cast<uint4*>(p.out + row * D + c);
+        uint4* dst = reinterpret_cast<uint4*>(p.out + row * p.dv + c);
 #pragma unroll
         for (int j = 0; j < 32; j += 8) {
+          if (c + j >= p.dv) break;
           uint4 w;
           __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&w);
 #pragma unroll
@@ -859,7 +871,7 @@ EncodeTiled encode_fn() {
   return fn;
 }
 // a pool [pages, nkv, page_size, d] seen as rows of d elements; boxes of one page of one head, 64 columns wide
-bool make_pool_map(CUtensorMap* map, const void* base, long long rows, int page_size, int d = D) {
+bool make_pool_map(CUtensorMap* map, const void* base, long long rows, int page_size, int d) {
   EncodeTiled fn = encode_fn();
   if (!fn) return false;
   cuuint64_t dims[2] = {(cuuint64_t)d, (cuuint64_t)rows};
@@ -873,19 +885,35 @@ bool make_pool_map(CUtensorMap* map, const void* base, long long rows, int page_
 int* error_flag_device = nullptr;
 int* error_flag_host = nullptr;
 
+// the kernel with a thread per row
+template <int HD, int HV>
+int launch_tc2(const CUtensorMap& map_k, const CUtensorMap& map_v, const Params& p, int num_seqs, int max_q_len, cudaStream_t stream) {
+  using Cfg = T2Cfg<HD, HV>;
+  static OncePerDevice configured;
+  if (!configured.here()) {
+    cudaError_t e = cudaFuncSetAttribute(paged_prefill_tc2_kernel<HD, HV>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM);
+    if (e != cudaSuccess) return (int)e;
+    configured.here() = true;
+  }
+  const int tiles = (max_q_len + Cfg::QT * p.tokens_per_tile - 1) / (Cfg::QT * p.tokens_per_tile);
+  if (tiles > 65535 || num_seqs > 65535) return DLI_ERR_UNSUPPORTED;  // the grid's y and z
+  return (int)launch_pdl((paged_prefill_tc2_kernel<HD, HV>), dim3(p.nkv * p.head_chunks, num_seqs, tiles), dim3(Cfg::THREADS), (size_t)Cfg::SMEM, stream, 1,
+                         map_k, map_v, p);
+}
+
 }  // namespace
 
 // Sequences [seq0, seq0 + num_seqs) of a batch, each bringing at most max_q_len tokens.
-// Head size 64 or 128; page_size must be 8, 16, 32, 64 or 128; num_pages is the pools' first extent.
-// query_tiles (head size 64): 1 or 2 tiles of 128 rows per CTA, 0 to let the launcher choose.
+// Key and value rows of up to 128 numbers, multiples of 8; page_size must be 8, 16, 32, 64 or 128; num_pages is the pools' first extent.
+// query_tiles (rows of 64): 1 or 2 tiles of 128 rows per CTA, 0 to let the launcher choose.
 DLI_EXPORT int dli_paged_prefill_tc(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long num_pages, const int* block_tables, int max_blocks, const int* q_start,
-                                    const int* kv_len, int seq0, int num_seqs, int max_q_len, int nh, int nkv, int head_dim,
+                                    const int* kv_len, int seq0, int num_seqs, int max_q_len, int nh, int nkv, int head_dim, int value_dim,
                                     int page_size, int window, float scale, float sink, const float* sink_heads, float softcap, const float* slopes,
                                     int query_tiles, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   if (!BENT_SCORES && (softcap != 0.f || slopes)) return DLI_ERR_UNSUPPORTED;
-  if (head_dim != 64 && head_dim != 128) return DLI_ERR_UNSUPPORTED;
+  if (head_dim < 8 || head_dim > 128 || head_dim % 8 || value_dim < 8 || value_dim > 128 || value_dim % 8) return DLI_ERR_UNSUPPORTED;
   if (nkv < 1 || nh % nkv || page_size < 8 || page_size > 128 || (KEYS % page_size) != 0) return DLI_ERR_UNSUPPORTED;
   if (((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)q) & 15) return DLI_ERR_UNSUPPORTED;
   if (!error_flag_host) {
@@ -901,7 +929,7 @@ DLI_EXPORT int dli_paged_prefill_tc(void* out, const void* q, long long q_stride
   }
   CUtensorMap map_k, map_v;
   const long long rows = num_pages * nkv * page_size;
-  if (!make_pool_map(&map_k, k_pool, rows, page_size, head_dim) || !make_pool_map(&map_v, v_pool, rows, page_size, head_dim)) return DLI_ERR_UNSUPPORTED;
+  if (!make_pool_map(&map_k, k_pool, rows, page_size, head_dim) || !make_pool_map(&map_v, v_pool, rows, page_size, value_dim)) return DLI_ERR_UNSUPPORTED;
   Params p;
   p.out = (bf16*)out; p.q = (const bf16*)q; p.q_stride = q_stride;
   p.block_tables = block_tables; p.max_blocks = max_blocks; p.q_start = q_start; p.kv_len = kv_len; p.seq0 = seq0;
@@ -915,37 +943,18 @@ DLI_EXPORT int dli_paged_prefill_tc(void* out, const void* q, long long q_stride
   p.head_chunks = (G + p.heads_per_chunk - 1) / p.heads_per_chunk;
   p.tokens_per_tile = ROWS / p.heads_per_chunk;
   p.error_flag = error_flag_device;
-  if (head_dim == 128) {  // one query tile per CTA, a thread per row
-    static OncePerDevice configured128;
-    if (!configured128.here()) {
-      cudaError_t e = cudaFuncSetAttribute(paged_prefill_tc2_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, T2Cfg<128>::SMEM);
-      if (e != cudaSuccess) return (int)e;
-      configured128.here() = true;
-    }
+  p.d = head_dim; p.dv = value_dim;
+  // rows of 64: one query tile per CTA, two threads a row, while a sequence brings no more tokens than one tile holds (or the caller asks)
+  if (head_dim == D && value_dim == D && (query_tiles == 1 || (query_tiles != 2 && max_q_len <= p.tokens_per_tile))) {
     const int tiles = (max_q_len + p.tokens_per_tile - 1) / p.tokens_per_tile;
     if (tiles > 65535 || num_seqs > 65535) return DLI_ERR_UNSUPPORTED;  // the grid's y and z
-    return (int)launch_pdl(paged_prefill_tc2_kernel<128>, dim3(nkv * p.head_chunks, num_seqs, tiles), dim3(T2Cfg<128>::THREADS),
-                           (size_t)T2Cfg<128>::SMEM, stream, 1, map_k, map_v, p);
+    return (int)launch_pdl(paged_prefill_tc_kernel, dim3(nkv * p.head_chunks, num_seqs, tiles), dim3(THREADS), (size_t)SMEM_BYTES, stream, 1, map_k,
+                           map_v, p);
   }
-  // two query tiles per CTA when a sequence brings more tokens than one tile holds, unless the caller chose
-  const bool two = query_tiles == 2 || (query_tiles != 1 && max_q_len > p.tokens_per_tile);
-  if (two) {
-    static OncePerDevice configured2;
-    if (!configured2.here()) {
-      cudaError_t e = cudaFuncSetAttribute(paged_prefill_tc2_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, T2Cfg<64>::SMEM);
-      if (e != cudaSuccess) return (int)e;
-      configured2.here() = true;
-    }
-    const int tiles = (max_q_len + 2 * p.tokens_per_tile - 1) / (2 * p.tokens_per_tile);
-    if (tiles > 65535 || num_seqs > 65535) return DLI_ERR_UNSUPPORTED;
-    return (int)launch_pdl(paged_prefill_tc2_kernel<64>, dim3(nkv * p.head_chunks, num_seqs, tiles), dim3(T2Cfg<64>::THREADS),
-                           (size_t)T2Cfg<64>::SMEM, stream, 1, map_k, map_v, p);
-  }
-  const int tiles = (max_q_len + p.tokens_per_tile - 1) / p.tokens_per_tile;
-  if (tiles > 65535 || num_seqs > 65535) return DLI_ERR_UNSUPPORTED;
-  cudaError_t e = launch_pdl(paged_prefill_tc_kernel, dim3(nkv * p.head_chunks, num_seqs, tiles), dim3(THREADS), (size_t)SMEM_BYTES, stream, 1,
-                             map_k, map_v, p);
-  return (int)e;
+  if (head_dim <= 64) return value_dim <= 64 ? launch_tc2<64, 64>(map_k, map_v, p, num_seqs, max_q_len, stream)
+                                             : launch_tc2<64, 128>(map_k, map_v, p, num_seqs, max_q_len, stream);
+  return value_dim <= 64 ? launch_tc2<128, 64>(map_k, map_v, p, num_seqs, max_q_len, stream)
+                         : launch_tc2<128, 128>(map_k, map_v, p, num_seqs, max_q_len, stream);
 }
 
 
@@ -956,31 +965,32 @@ constexpr int DN = 16;                 // keys per tile of one warp
 constexpr int CLUSTER_SPLITS_MAX = 16;  // the largest cluster of this GPU (more than 8 is the kernel's opt-in)
 constexpr int CLUSTER_ROWS_MAX = 23;    // rows of partial results that may arrive at one CTA
 
-// Sizes that depend on the head size HD (64 or 128).  A row of keys or values is HD * 2 bytes; the
-// 128-byte swizzle covers 64 elements, so a tile of 16 rows lies in shared memory as HD / 64 slabs of
-// [16 rows x 128 bytes], each filled by its own TMA box (the columns 64 s .. 64 s + 63 of the rows).
-// DWARPS: warps of a CTA, each with its own tiles and stages.  Four, so that four CTAs (two at head size 128) share an
+// Sizes that depend on the columns of keys (HD) and values (HV) in shared memory, 64 or 128 each.  The 128-byte swizzle covers 64
+// elements, so a tile of 16 rows lies there as HD / 64 (HV / 64) slabs of [16 rows x 128 bytes], each filled by its own TMA
+// box (the columns 64 s .. 64 s + 63 of the rows; what the pool's rows do not have is filled with zeros).
+// DWARPS: warps of a CTA, each with its own tiles and stages.  Four, so that four CTAs (two with rows of 128) share an
 // SM when the grid is large; eight when the grid has fewer CTAs than two per SM (one or two long sequences), where
 // nothing else would hide a warp's latencies.
-template <int HD, int DWARPS>
+template <int HD, int HV, int DWARPS>
 struct DecodeCfg {
-  static_assert(HD == 64 || HD == 128, "head sizes with whole 128-byte slabs");
+  static_assert((HD == 64 || HD == 128) && (HV == 64 || HV == 128), "head sizes with whole 128-byte slabs");
   static_assert(DWARPS == 4 || DWARPS == 8, "four or eight warps");
-  static constexpr int SLABS = HD / 64;
+  static constexpr int SLABS = HD / 64, VSLABS = HV / 64;
   static constexpr int SLAB = DN * 128;                 // bytes of one slab
-  static constexpr int TILE = SLABS * SLAB;             // one K or V tile
-  static constexpr int STAGES = HD == 64 ? 3 : 2;
+  static constexpr int KTILE = SLABS * SLAB;            // one tile of keys
+  static constexpr int STAGE = KTILE + VSLABS * SLAB;   // and the values behind it
+  static constexpr int STAGES = HD + HV < 256 ? 3 : 2;
   static constexpr int QROW = HD * 2 + 16;              // padded query rows (read once)
   // Splits merged inside a cluster: row r of the 16 belongs to CTA (r mod splits); every CTA pushes its
-  // partial (sums[HD], maximum, denominator) of a row into the owner's memory: splits * ceil(rows / splits)
+  // partial (sums[HV], maximum, denominator) of a row into the owner's memory: splits * ceil(rows / splits)
   // rows arrive at one CTA, and the launcher merges in the cluster only if that is at most
   // CLUSTER_ROWS_MAX.  The region starts where the query rows lay: they are in registers by then.
-  static constexpr int RECV_ROW = HD + 2;
+  static constexpr int RECV_ROW = HV + 2;
   static constexpr int RECV_BYTES = CLUSTER_ROWS_MAX * RECV_ROW * 4;
-  static constexpr int SMEM = 1024 + DWARPS * STAGES * 2 * TILE + RECV_BYTES + DWARPS * STAGES * 8 + 64;
+  static constexpr int SMEM = 1024 + DWARPS * STAGES * STAGE + RECV_BYTES + DWARPS * STAGES * 8 + 64;
   static_assert(RECV_BYTES >= 16 * QROW, "the received partial results lie over the query rows");
-  static_assert(DWARPS * 16 * (HD + 2) * 4 <= DWARPS * STAGES * 2 * TILE, "the merge buffer reuses the key/value stages");
-  static_assert((DWARPS == 8 ? 1 : HD == 64 ? 4 : 2) * (SMEM + 1024) <= 227 * 1024, "four CTAs per SM at head size 64, two at 128 (four warps)");
+  static_assert(DWARPS * 16 * (HV + 2) * 4 <= DWARPS * STAGES * STAGE, "the merge buffer reuses the key/value stages");
+  static_assert((DWARPS == 8 ? 1 : HD + HV == 128 ? 4 : 2) * (SMEM + 1024) <= 227 * 1024, "four CTAs per SM with rows of 64, two with rows of 128 (four warps)");
 };
 
 struct DecodeParams {
@@ -992,6 +1002,7 @@ struct DecodeParams {
   const int* q_start;
   const int* kv_len;
   int seq0, nh, nkv, page_size, window, splits;
+  int d, dv;          // columns of the pools' key and value rows (and of queries and output)
   int cluster_merge;  // the splits of a (sequence, head group) are one cluster and merge through shared memory
   float scale_log2;   // as in Params
   ScoreBend bend;     // as in Params
@@ -1046,17 +1057,17 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
 // are the query heads of one KV head; each warp walks its own share of the 16-key tiles.  A tile's
 // keys and values arrive by TMA (one box per page piece, 128-byte swizzle), four tiles ahead, on the
 // warp's own mbarriers: no thread spends instructions on addresses of individual 16-byte copies.
-template <int HD, int DWARPS>
+template <int HD, int HV, int DWARPS>
 __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                        const __grid_constant__ CUtensorMap map_v, const DecodeParams p) {
-  using Cfg = DecodeCfg<HD, DWARPS>;
-  constexpr int DSTAGES = Cfg::STAGES, DTILE = Cfg::TILE, QROW = Cfg::QROW, RECV_BYTES = Cfg::RECV_BYTES, RECV_ROW = Cfg::RECV_ROW;
+  using Cfg = DecodeCfg<HD, HV, DWARPS>;
+  constexpr int DSTAGES = Cfg::STAGES, KTILE = Cfg::KTILE, STAGE = Cfg::STAGE, QROW = Cfg::QROW, RECV_BYTES = Cfg::RECV_BYTES, RECV_ROW = Cfg::RECV_ROW;
   constexpr int D = HD;  // shadows the prefill kernel's head size within this kernel
   pdl_launch_dependents();
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* sKV = smem;                                   // [warp][stage][K | V]
-  unsigned char* sQ = sKV + DWARPS * DSTAGES * 2 * DTILE;      // 16 padded rows
+  unsigned char* sQ = sKV + DWARPS * DSTAGES * STAGE;      // 16 padded rows
   uint64_t* bars = (uint64_t*)(sQ + RECV_BYTES);               // [warp][stage]
   volatile int* failed = (volatile int*)(bars + DWARPS * DSTAGES);
 
@@ -1095,7 +1106,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   }
   __syncwarp();  // this warp's barriers are set up
 
-  unsigned char* wbuf = sKV + warp * DSTAGES * 2 * DTILE;
+  unsigned char* wbuf = sKV + warp * DSTAGES * STAGE;
   const uint32_t wbar = smem_u32(bars + warp * DSTAGES);
   const int my_tiles = (t_end - t_begin - warp + DWARPS - 1) / DWARPS;
   const int box_rows = p.page_size < DN ? p.page_size : DN;  // a tile is one piece of a page, or two whole pages of 8
@@ -1114,7 +1125,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   // every lane calls this (the shuffles need them all); lane 0 issues the copies of the warp's i-th tile into stage st
   auto issue = [&](int i, int st) {
     const uint32_t bar = wbar + 8 * st;
-    if (lane == 0) mbar_expect_tx(bar, 2 * DTILE);
+    if (lane == 0) mbar_expect_tx(bar, STAGE);
     for (int b = 0; b < boxes; ++b) {
       const int e = i * boxes + b;
       if (e >= cached_first + 32) {
@@ -1124,9 +1135,9 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
       const int row = __shfl_sync(0xffffffffu, cached, e - cached_first);
       if (lane == 0) {
 #pragma unroll
-        for (int sl = 0; sl < Cfg::SLABS; ++sl) {
-          tma_load_2d(smem_u32(wbuf + st * 2 * DTILE + sl * Cfg::SLAB + b * box_rows * 128), &map_k, sl * 64, row, bar);
-          tma_load_2d(smem_u32(wbuf + st * 2 * DTILE + DTILE + sl * Cfg::SLAB + b * box_rows * 128), &map_v, sl * 64, row, bar);
+        for (int sl = 0; sl < (HD > HV ? Cfg::SLABS : Cfg::VSLABS); ++sl) {
+          if (sl < Cfg::SLABS) tma_load_2d(smem_u32(wbuf + st * STAGE + sl * Cfg::SLAB + b * box_rows * 128), &map_k, sl * 64, row, bar);
+          if (sl < Cfg::VSLABS) tma_load_2d(smem_u32(wbuf + st * STAGE + KTILE + sl * Cfg::SLAB + b * box_rows * 128), &map_v, sl * 64, row, bar);
         }
       }
     }
@@ -1135,9 +1146,9 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   const int r0 = lane >> 2, r1 = r0 + 8;
   float m[2] = {-CUDART_INF_F, -CUDART_INF_F};
   float l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[HV / 8][4];
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+  for (int j = 0; j < HV / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
 
   // Keys and values of earlier steps do not depend on the kernel before this one (it wrote this
   // step's token only), nor do the tables and lengths: the first tiles are requested before the wait
@@ -1154,7 +1165,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   for (int idx = tid; idx < 16 * (D / 8); idx += DWARPS * 32) {
     const int r = idx / (D / 8), c = idx - r * (D / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < nheads) v = *reinterpret_cast<const uint4*>(p.q + (size_t)token * p.q_stride + (size_t)(head0 + r) * D + c * 8);
+    if (r < nheads && c * 8 < p.d) v = *reinterpret_cast<const uint4*>(p.q + (size_t)token * p.q_stride + (size_t)(head0 + r) * p.d + c * 8);
     *reinterpret_cast<uint4*>(sQ + r * QROW + c * 16) = v;
   }
   __syncthreads();
@@ -1181,7 +1192,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
     if (ok && !wait_or_fail(wbar + 8 * st, phase, failed, 21, p.error_flag)) ok = false;
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
-      const uint32_t tK = smem_u32(wbuf + st * 2 * DTILE), tV = tK + DTILE;
+      const uint32_t tK = smem_u32(wbuf + st * STAGE), tV = tK + KTILE;
       const int base = (t_begin + warp + i * DWARPS) * DN;
       // ---- S = Q K^T for 16 keys: two 8-key column tiles
       float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
@@ -1227,7 +1238,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
         l[0] *= c0;
         l[1] *= c1;
 #pragma unroll
-        for (int j = 0; j < D / 8; ++j) {
+        for (int j = 0; j < HV / 8; ++j) {
           o[j][0] *= c0; o[j][1] *= c0;
           o[j][2] *= c1; o[j][3] *= c1;
         }
@@ -1244,7 +1255,7 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
       // ---- O += P V (16 keys = one k step)
       uint32_t a[4] = {pack2(sc[0][0], sc[0][1]), pack2(sc[0][2], sc[0][3]), pack2(sc[1][0], sc[1][1]), pack2(sc[1][2], sc[1][3])};
 #pragma unroll
-      for (int jp = 0; jp < D / 16; ++jp) {
+      for (int jp = 0; jp < HV / 16; ++jp) {
         uint32_t b[4];
         const int key = (lane & 7) + ((lane >> 3) & 1) * 8;
         const int chunk = (jp & 3) * 2 + (lane >> 4);
@@ -1264,15 +1275,15 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
 
   // ---- merge the four warps' partial results in shared memory (the key/value stages are free)
   __syncthreads();
-  float* mo = reinterpret_cast<float*>(sKV);   // [DWARPS][16][D]
-  float* mm = mo + DWARPS * 16 * D;            // [DWARPS][16]
+  float* mo = reinterpret_cast<float*>(sKV);   // [DWARPS][16][HV]
+  float* mm = mo + DWARPS * 16 * HV;            // [DWARPS][16]
   float* ml = mm + DWARPS * 16;
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
     const int row = rr ? r1 : r0;
-    float* dst = mo + (warp * 16 + row) * D;
+    float* dst = mo + (warp * 16 + row) * HV;
 #pragma unroll
-    for (int j = 0; j < D / 8; ++j) *reinterpret_cast<float2*>(dst + j * 8 + (lane & 3) * 2) = make_float2(o[j][2 * rr], o[j][2 * rr + 1]);
+    for (int j = 0; j < HV / 8; ++j) *reinterpret_cast<float2*>(dst + j * 8 + (lane & 3) * 2) = make_float2(o[j][2 * rr], o[j][2 * rr + 1]);
     if ((lane & 3) == 0) {
       mm[warp * 16 + row] = m[rr];
       ml[warp * 16 + row] = l[rr];
@@ -1284,8 +1295,9 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   float* recv = reinterpret_cast<float*>(sQ);  // [split][owned row][sums | maximum | denominator]
   const int owned_max = (nheads + p.splits - 1) / p.splits;
   if (p.cluster_merge) cluster_wait();  // every CTA of the cluster has its query in registers: the region may be written
-  for (int idx = tid; idx < nheads * D; idx += DWARPS * 32) {
-    const int r = idx / D, dcol = idx - r * D;
+  for (int idx = tid; idx < nheads * HV; idx += DWARPS * 32) {
+    const int r = idx / HV, dcol = idx - r * HV;
+    if (dcol >= p.dv && !p.cluster_merge) continue;  // a cluster's receivers count every column
     float mx = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < DWARPS; ++w) mx = fmaxf(mx, mm[w * 16 + r]);
@@ -1295,21 +1307,21 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
       const float mw = mm[w * 16 + r];
       const float f = (mw == -CUDART_INF_F) ? 0.f : ex2(mw - mx);
       L += ml[w * 16 + r] * f;
-      acc += mo[(w * 16 + r) * D + dcol] * f;
+      acc += mo[(w * 16 + r) * HV + dcol] * f;
     }
     const size_t row = (size_t)token * p.nh + head0 + r;
     if (p.splits == 1) {
-      p.out[row * D + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
+      p.out[row * p.dv + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
     } else if (p.cluster_merge) {
       const uint32_t dst = smem_u32(recv + (split * owned_max + r / p.splits) * RECV_ROW);
       const int owner = r % p.splits;
       st_async_peer(dst + dcol * 4, merged, owner, acc);
       if (dcol == 0) {
-        st_async_peer(dst + D * 4, merged, owner, mx);
-        st_async_peer(dst + (D + 1) * 4, merged, owner, L);
+        st_async_peer(dst + HV * 4, merged, owner, mx);
+        st_async_peer(dst + (HV + 1) * 4, merged, owner, L);
       }
     } else {
-      p.part_acc[(row * p.splits + split) * D + dcol] = acc;
+      p.part_acc[(row * p.splits + split) * p.dv + dcol] = acc;
       if (dcol == 0) {
         p.part_ml[(row * p.splits + split) * 2] = mx;
         p.part_ml[(row * p.splits + split) * 2 + 1] = L;
@@ -1321,22 +1333,23 @@ __global__ void __launch_bounds__(DWARPS * 32) paged_decode_tma_kernel(const __g
   // cluster barrier, which would also hold the CTAs that merge nothing); nobody reads a peer's memory, and a CTA
   // leaves only after what was sent to it has landed
   if (!wait_cluster_or_fail(merged, 0, failed, 22, p.error_flag) || bad) return;
-  for (int idx = tid; idx < mine * D; idx += DWARPS * 32) {
-    const int ri = idx / D, dcol = idx - ri * D;
+  for (int idx = tid; idx < mine * HV; idx += DWARPS * 32) {
+    const int ri = idx / HV, dcol = idx - ri * HV;
+    if (dcol >= p.dv) continue;
     const int r = split + ri * p.splits;
     float mx = -CUDART_INF_F;
-    for (int i = 0; i < p.splits; ++i) mx = fmaxf(mx, recv[(i * owned_max + ri) * RECV_ROW + D]);
+    for (int i = 0; i < p.splits; ++i) mx = fmaxf(mx, recv[(i * owned_max + ri) * RECV_ROW + HV]);
     float L = 0.f, acc = 0.f;
     for (int i = 0; i < p.splits; ++i) {  // split 0 first: a fixed order
       const float* part = recv + (i * owned_max + ri) * RECV_ROW;
-      const float mi = part[D];
+      const float mi = part[HV];
       if (mi != -CUDART_INF_F) {
         const float f = ex2(mi - mx);
-        L += part[D + 1] * f;
+        L += part[HV + 1] * f;
         acc += part[dcol] * f;
       }
     }
-    p.out[((size_t)token * p.nh + head0 + r) * D + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
+    p.out[((size_t)token * p.nh + head0 + r) * p.dv + dcol] = __float2bfloat16_rn(acc / (L + sink_term(sink_of(p.sink_heads, p.sink_log2, head0 + r), mx)));
   }
 }
 
@@ -1385,51 +1398,52 @@ bool merges_in_cluster(int nh, int nkv, int splits) {
   return splits > 1 && (splits <= 8 || splits == CLUSTER_SPLITS_MAX) && splits * ((rows + splits - 1) / splits) <= CLUSTER_ROWS_MAX;
 }
 
-template <int HD, int DWARPS>
+template <int HD, int HV, int DWARPS>
 int launch_decode_warps(const CUtensorMap& map_k, const CUtensorMap& map_v, const DecodeParams& p, int num_seqs, int first_row, cudaStream_t stream) {
   static OncePerDevice configured;
   if (!configured.here()) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_tma_kernel<HD, DWARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecodeCfg<HD, DWARPS>::SMEM);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(paged_decode_tma_kernel<HD, DWARPS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    cudaError_t e = cudaFuncSetAttribute((paged_decode_tma_kernel<HD, HV, DWARPS>), cudaFuncAttributeMaxDynamicSharedMemorySize, (DecodeCfg<HD, HV, DWARPS>::SMEM));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute((paged_decode_tma_kernel<HD, HV, DWARPS>), cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (e != cudaSuccess) return (int)e;
     configured.here() = true;
   }
   const int G = p.nh / p.nkv;
-  cudaError_t e = launch_pdl(paged_decode_tma_kernel<HD, DWARPS>, dim3(num_seqs, p.splits, p.nkv * ((G + 15) / 16)), dim3(DWARPS * 32),
-                             (size_t)DecodeCfg<HD, DWARPS>::SMEM, stream, p.cluster_merge ? p.splits : 1, map_k, map_v, p);
+  cudaError_t e = launch_pdl((paged_decode_tma_kernel<HD, HV, DWARPS>), dim3(num_seqs, p.splits, p.nkv * ((G + 15) / 16)), dim3(DWARPS * 32),
+                             (size_t)DecodeCfg<HD, HV, DWARPS>::SMEM, stream, p.cluster_merge ? p.splits : 1, map_k, map_v, p);
   if (e != cudaSuccess) return (int)e;
   if (p.splits > 1 && !p.cluster_merge)
     e = launch_pdl(merge_decode_splits_kernel, dim3(num_seqs * p.nh), dim3(64), 0, stream, 1, p.out, (const float*)p.part_acc,
-                   (const float*)p.part_ml, first_row * p.nh, p.splits, HD, p.sink_log2, p.sink_heads, p.nh);
+                   (const float*)p.part_ml, first_row * p.nh, p.splits, p.dv, p.sink_log2, p.sink_heads, p.nh);
   return (int)e;
 }
 
 
-// Eight warps a CTA at head size 64 when the grid leaves SMs with one CTA at most and every warp still gets four tiles
+// Eight warps a CTA with rows of 64 when the grid leaves SMs with one CTA at most and every warp still gets four tiles
 // or more: one sequence of 32 K keys in 16 splits takes 33 us with four warps and 27 with eight.  (Measured slower
-// with eight: two CTAs on an SM, 39 -> 48 us for two such sequences, and head size 128, 44 -> 58 us.)
-template <int HD>
+// with eight: two CTAs on an SM, 39 -> 48 us for two such sequences, and rows of 128, 44 -> 58 us.)
+template <int HD, int HV>
 int launch_decode(const CUtensorMap& map_k, const CUtensorMap& map_v, const DecodeParams& p, int num_seqs, int first_row, int max_kv_len,
                   cudaStream_t stream) {
   const int G = p.nh / p.nkv;
   const long long ctas = (long long)num_seqs * p.splits * p.nkv * ((G + 15) / 16);
   const int tiles_per_split = (max_kv_len + DN - 1) / DN / p.splits;
-  if (HD == 64 && ctas <= sm_count() && tiles_per_split >= 32) return launch_decode_warps<HD, 8>(map_k, map_v, p, num_seqs, first_row, stream);
-  return launch_decode_warps<HD, 4>(map_k, map_v, p, num_seqs, first_row, stream);
+  if constexpr (HD == 64 && HV == 64)
+    if (ctas <= sm_count() && tiles_per_split >= 32) return launch_decode_warps<HD, HV, 8>(map_k, map_v, p, num_seqs, first_row, stream);
+  return launch_decode_warps<HD, HV, 4>(map_k, map_v, p, num_seqs, first_row, stream);
 }
 }  // namespace
 
-// Attention of num_seqs single-token sequences (head size 64 or 128; page size a multiple of 8, and
+// Attention of num_seqs single-token sequences (key and value rows of up to 128 numbers, multiples of 8; page size a multiple of 8, and
 // of 16 if larger than 8).  Up to 16 splits are one cluster and merge on the chip; more go through
 // part_acc / part_ml (scratch, as for dli_paged_attention_mma) and a second kernel.
 DLI_EXPORT int dli_paged_decode_tma(void* out, const void* q, long long q_stride, const void* k_pool, const void* v_pool,
                                     long long num_pages, const int* block_tables, int max_blocks, const int* q_start,
-                                    const int* kv_len, int seq0, int num_seqs, int first_row, int nh, int nkv, int head_dim,
+                                    const int* kv_len, int seq0, int num_seqs, int first_row, int nh, int nkv, int head_dim, int value_dim,
                                     int page_size, int window, float scale, float sink, const float* sink_heads, float softcap, const float* slopes,
                                     int splits, float* part_acc, float* part_ml, int max_kv_len, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   if (!BENT_SCORES && (softcap != 0.f || slopes)) return DLI_ERR_UNSUPPORTED;
-  if (head_dim != 64 && head_dim != 128) return DLI_ERR_UNSUPPORTED;
+  if (head_dim < 8 || head_dim > 128 || head_dim % 8 || value_dim < 8 || value_dim > 128 || value_dim % 8) return DLI_ERR_UNSUPPORTED;
   if (nkv < 1 || nh % nkv || splits < 1 || (splits > 1 && (!part_acc || !part_ml))) return DLI_ERR_UNSUPPORTED;
   if (page_size < 8 || (page_size % 8) || (page_size > 8 && (page_size % 16)) || page_size > 256) return DLI_ERR_UNSUPPORTED;
   if (((uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)q) & 15) return DLI_ERR_UNSUPPORTED;
@@ -1441,7 +1455,7 @@ DLI_EXPORT int dli_paged_decode_tma(void* out, const void* q, long long q_stride
   CUtensorMap map_k, map_v;
   const long long rows = num_pages * nkv * page_size;
   const int box_rows = page_size < DN ? page_size : DN;
-  if (!make_decode_map(&map_k, k_pool, rows, box_rows, head_dim) || !make_decode_map(&map_v, v_pool, rows, box_rows, head_dim))
+  if (!make_decode_map(&map_k, k_pool, rows, box_rows, head_dim) || !make_decode_map(&map_v, v_pool, rows, box_rows, value_dim))
     return DLI_ERR_UNSUPPORTED;
   DecodeParams p;
   p.out = (bf16*)out; p.q = (const bf16*)q; p.q_stride = q_stride;
@@ -1452,9 +1466,12 @@ DLI_EXPORT int dli_paged_decode_tma(void* out, const void* q, long long q_stride
   p.sink_log2 = sink * 1.4426950408889634f;  // -inf (no sink) stays -inf
   p.sink_heads = sink_heads;
   p.part_acc = part_acc; p.part_ml = part_ml; p.error_flag = error_flag_device;
+  p.d = head_dim; p.dv = value_dim;
   p.cluster_merge = merges_in_cluster(nh, nkv, splits);
-  return head_dim == 64 ? launch_decode<64>(map_k, map_v, p, num_seqs, first_row, max_kv_len, stream)
-                        : launch_decode<128>(map_k, map_v, p, num_seqs, first_row, max_kv_len, stream);
+#define DLI_DECODE(HD, HV) launch_decode<HD, HV>(map_k, map_v, p, num_seqs, first_row, max_kv_len, stream)
+  if (head_dim <= 64) return value_dim <= 64 ? DLI_DECODE(64, 64) : DLI_DECODE(64, 128);
+  return value_dim <= 64 ? DLI_DECODE(128, 64) : DLI_DECODE(128, 128);
+#undef DLI_DECODE
 }
 
 DLI_EXPORT int dli_decode_tma_merges_in_cluster(int nh, int nkv, int splits) { return merges_in_cluster(nh, nkv, splits) ? 1 : 0; }

@@ -1,12 +1,15 @@
 // The experts' products of a routed feed-forward for steps of many tokens (bfloat16): the (token, expert) pairs are
 // sorted by expert on the device (a counting sort; no shape depends on the data), and two grouped products run over the
 // sorted rows on the tensor cores (mma.sync m16n8k16 fed by ldmatrix, float32 sums), a tile of 64 rows belonging to one expert:
-//   hidden[row] = act(gate_e x) * (up_e x)        (both sums rounded to bfloat16 first, as a stored product would be)
+//   hidden[row] = act(gate_e x) * (up_e x), or act(up_e x) for experts without a gate
+//                                                 (the sums rounded to bfloat16 first, as a stored product would be)
 //   partial[row] = down_e hidden[row]             (float32)
-//   out[t] = sum_k weights[t][k] * partial[row of pair (t, k)], in the order of k, float32, one rounding.
+//   out[t] = sum_k weights[t][k] * partial[row of pair (t, k)] (+ shared[t]), in the order of k, float32, one rounding.
+// Experts numbered E and above are identities: their pairs have no row, and x[t] takes the place of partial in the sum.
 #include <math_constants.h>
 
 #include "common.cuh"
+#include "expert_act.cuh"
 
 using namespace dli;
 typedef __nv_bfloat16 bf16;
@@ -16,6 +19,7 @@ namespace {
 constexpr int BM = 64, BN = 64, BK = 64, PAD = 8, THREADS = 128;
 constexpr int LDS = BK + PAD;  // elements of a staged row: 144 bytes, so the eight rows of an 8 x 8 fragment lie in different banks
 constexpr int TILE_ELEMS = BM * LDS;  // one staged tile of 64 rows (A, or one of B's)
+enum { EPI_F32 = 0, EPI_GLU = 1, EPI_ACT = 2 };  // what a grouped product does with its sums
 constexpr int SORT_SMALL_MAX_PAIRS = 2048;  // up to here one block sorts the pairs in one launch
 
 // counts <- 0, and -1 into the tile and row maps (what no expert claims stays -1)
@@ -28,11 +32,11 @@ __global__ void moe_init_kernel(int* __restrict__ counts, int n_counts, int* __r
   }
 }
 
-__global__ void moe_count_kernel(const int* __restrict__ ids, int pairs, int* __restrict__ counts, int* __restrict__ rank) {
+__global__ void moe_count_kernel(const int* __restrict__ ids, int pairs, int E, int* __restrict__ counts, int* __restrict__ rank) {
   pdl_launch_dependents();
   pdl_wait();
   const int p = blockIdx.x * blockDim.x + threadIdx.x;
-  if (p < pairs) rank[p] = atomicAdd(&counts[ids[p]], 1);
+  if (p < pairs && ids[p] < E) rank[p] = atomicAdd(&counts[ids[p]], 1);
 }
 
 // offsets[e]: first sorted row of expert e, every expert's run padded to whole tiles; tile_expert[tile]: the tile's expert
@@ -54,12 +58,12 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts, int E, int* __re
 }
 
 // pos[p]: the sorted row of pair p; row_pair[row]: the pair of a sorted row (-1 for padding: set by the caller beforehand)
-__global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __restrict__ rank, const int* __restrict__ offsets, int pairs,
+__global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __restrict__ rank, const int* __restrict__ offsets, int pairs, int E,
                                    int* __restrict__ pos, int* __restrict__ row_pair) {
   pdl_launch_dependents();
   pdl_wait();
   const int p = blockIdx.x * blockDim.x + threadIdx.x;
-  if (p >= pairs) return;
+  if (p >= pairs || ids[p] >= E) return;
   const int row = offsets[ids[p]] + rank[p];
   pos[p] = row;
   row_pair[row] = p;
@@ -78,7 +82,8 @@ __global__ void moe_sort_small_kernel(const int* __restrict__ ids, int pairs, in
   for (int i = threadIdx.x; i < tiles; i += blockDim.x) tile_expert[i] = -1;
   for (int i = threadIdx.x; i < tiles * BM; i += blockDim.x) row_pair[i] = -1;
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += blockDim.x) pos[p] = atomicAdd(&cnt[ids[p]], 1);  // the pair's rank for now
+  for (int p = threadIdx.x; p < pairs; p += blockDim.x)
+    if (ids[p] < E) pos[p] = atomicAdd(&cnt[ids[p]], 1);  // the pair's rank for now
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0;
@@ -95,6 +100,7 @@ __global__ void moe_sort_small_kernel(const int* __restrict__ ids, int pairs, in
       for (int tile = off[e] / BM; tile < off[e + 1] / BM; ++tile) tile_expert[tile] = e;
   }
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+    if (ids[p] >= E) continue;
     const int row = off[ids[p]] + pos[p];
     pos[p] = row;
     row_pair[row] = p;
@@ -114,12 +120,6 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
 
-__device__ __forceinline__ float glu_act(float g, int act) {
-  if (act == 1) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-  if (act == 2) return g / (1.f + expf(-1.702f * g));
-  return g / (1.f + expf(-g));
-}
-
 __device__ __forceinline__ float round_bf16(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const bf16* p) {
@@ -127,12 +127,14 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const bf16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
 
-// C[row][n] = sum_k A[src(row)][k] * B_e[n][k] over one tile of 64 sorted rows of expert e = tile_expert[tile] and 64 columns.
-// GLU: two B tiles (rows n and half + n of the expert's matrix) and C = act(first) * second, bfloat16; else C float32.
-// row_pair (GLU): the sorted row's pair, whose token pair / top is the row of A (-1: zeros); without it the row of A is the sorted row.
+// C[row][n] = sum_k A[src(row)][k] * B_e[n][k] over one tile of 64 sorted rows of expert e = tile_expert[tile] and 64 NB columns.
+// EPI_GLU: two B tiles (rows n and half + n of the expert's matrix) and C = act(first) * second, bfloat16 (64 columns a tile).
+// EPI_ACT: C = act(sum), bfloat16; EPI_F32: C float32; with NB = 2 their second B tile is the next 64 columns, so that a tile of A
+// is read once for 128.
+// row_pair (the up products): the sorted row's pair, whose token pair / top is the row of A (-1: zeros); without it the row of A is the sorted row.
 // k-tiles of 64 arrive by asynchronous copies STAGES deep: three for a step of few tokens, which only streams the experts' matrices
 // and is bound by the bytes in flight; two for many tokens, where more CTAs an SM hide more latency.  Fragments are read with ldmatrix.
-template <bool GLU, int STAGES>
+template <int EPI, int NB, int STAGES>
 __global__ void __launch_bounds__(THREADS) moe_grouped_gemm_kernel(const bf16* __restrict__ A, long long a_stride, const int* __restrict__ row_pair,
                                                                    int top, const bf16* __restrict__ B, long long b_expert_stride, int half,
                                                                    void* __restrict__ C, long long c_stride, int N, int K,
@@ -142,14 +144,14 @@ __global__ void __launch_bounds__(THREADS) moe_grouped_gemm_kernel(const bf16* _
   const int tile_m = blockIdx.y;
   const int e = tile_expert[tile_m];
   if (e < 0) return;
-  constexpr int NB = GLU ? 2 : 1;
+  static_assert(EPI != EPI_GLU || NB == 2, "a gated product has two tiles of B");
   constexpr int STAGE_ELEMS = (1 + NB) * TILE_ELEMS;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* smem = reinterpret_cast<bf16*>(smem_raw);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int wm = warp >> 1, wn = warp & 1;
   const int g = lane >> 2, t = lane & 3;
-  const int n0 = blockIdx.x * BN;
+  const int n0 = blockIdx.x * (EPI == EPI_GLU ? BN : NB * BN);
   const bf16* Be = B + (size_t)e * b_expert_stride;
 
   // the four 16-byte chunks of A (and of each B tile) this thread copies per k-tile: rows r0 + 16 i, one column of chunks
@@ -167,7 +169,10 @@ __global__ void __launch_bounds__(THREADS) moe_grouped_gemm_kernel(const bf16* _
       a_src[i] = A + (size_t)row * a_stride;
     }
 #pragma unroll
-    for (int j = 0; j < NB; ++j) b_src[j][i] = n0 + r < N ? Be + (size_t)(j * half + n0 + r) * K : nullptr;
+    for (int j = 0; j < NB; ++j) {
+      const int col = EPI == EPI_GLU ? n0 + r : n0 + j * BN + r;
+      b_src[j][i] = col < N ? Be + (size_t)(EPI == EPI_GLU ? j * half + col : col) * K : nullptr;
+    }
   }
 
   auto load = [&](int stage, int k0) {
@@ -238,32 +243,67 @@ __global__ void __launch_bounds__(THREADS) moe_grouped_gemm_kernel(const bf16* _
 #pragma unroll
       for (int hrow = 0; hrow < 2; ++hrow) {
         const size_t row = (size_t)tile_m * BM + wm * 32 + mi * 16 + g + hrow * 8;
-        const int col = n0 + wn * 32 + ni * 8 + 2 * t;
-        if (col >= N) continue;
-        const float v0 = acc[0][mi][ni][2 * hrow], v1 = acc[0][mi][ni][2 * hrow + 1];
-        if (GLU) {
-          const float u0 = acc[NB - 1][mi][ni][2 * hrow], u1 = acc[NB - 1][mi][ni][2 * hrow + 1];
-          bf16* dst = reinterpret_cast<bf16*>(C) + row * c_stride + col;
-          dst[0] = __float2bfloat16_rn(glu_act(round_bf16(v0), act) * round_bf16(u0));
-          if (col + 1 < N) dst[1] = __float2bfloat16_rn(glu_act(round_bf16(v1), act) * round_bf16(u1));
-        } else {
-          float* dst = reinterpret_cast<float*>(C) + row * c_stride + col;
-          dst[0] = v0;
-          if (col + 1 < N) dst[1] = v1;
+#pragma unroll
+        for (int j = 0; j < (EPI == EPI_GLU ? 1 : NB); ++j) {
+          const int col = n0 + j * BN + wn * 32 + ni * 8 + 2 * t;  // N is a multiple of 8: a pair of columns lies inside or outside
+          if (col >= N) continue;
+          const float v0 = acc[j][mi][ni][2 * hrow], v1 = acc[j][mi][ni][2 * hrow + 1];
+          if (EPI == EPI_F32) {
+            *reinterpret_cast<float2*>(reinterpret_cast<float*>(C) + row * c_stride + col) = make_float2(v0, v1);
+          } else {
+            float o0, o1;
+            if (EPI == EPI_GLU) {
+              o0 = glu_act(round_bf16(v0), act) * round_bf16(acc[NB - 1][mi][ni][2 * hrow]);
+              o1 = glu_act(round_bf16(v1), act) * round_bf16(acc[NB - 1][mi][ni][2 * hrow + 1]);
+            } else {
+              o0 = plain_act(round_bf16(v0), act);
+              o1 = plain_act(round_bf16(v1), act);
+            }
+            *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf16*>(C) + row * c_stride + col) = __floats2bfloat162_rn(o0, o1);
+          }
         }
       }
 }
 
-__global__ void moe_combine_kernel(bf16* __restrict__ out, const float* __restrict__ partial, const int* __restrict__ pos,
-                                   const float* __restrict__ weights, int W, int top) {
+// eight columns a thread (W is a multiple of 8)
+__global__ void moe_combine_kernel(bf16* __restrict__ out, const float* __restrict__ partial, const int* __restrict__ pos, const int* __restrict__ ids,
+                                   const float* __restrict__ weights, const bf16* __restrict__ x, const bf16* __restrict__ shared, int W, int E, int top) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
-  for (int c = threadIdx.x; c < W; c += blockDim.x) {
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k) acc = fmaf(weights[t * top + k], partial[(size_t)pos[t * top + k] * W + c], acc);
-    out[t * W + c] = __float2bfloat16_rn(acc);
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    for (int k = 0; k < top; ++k) {
+      const float w = weights[t * top + k];
+      float v[8];
+      if (ids[t * top + k] < E) load8(partial + (size_t)pos[t * top + k] * W + c, v);
+      else load8(x + t * W + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] = fmaf(w, v[i], acc[i]);
+    }
+    if (shared) {
+      float v[8];
+      load8(shared + t * W + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] += v[i];
+    }
+    store8(out + t * W + c, acc);
   }
+}
+
+template <int EPI, int NB, int STAGES>
+cudaError_t launch_grouped(const bf16* A, long long a_stride, const int* row_pair, int top, const bf16* B, long long b_expert_stride, int half, void* C,
+                           int N, int K, const int* tile_expert, int tiles, int act, cudaStream_t stream) {
+  constexpr int SMEM = STAGES * (1 + NB) * TILE_ELEMS * (int)sizeof(bf16);
+  static OncePerDevice configured;
+  if (!configured.here()) {
+    cudaError_t e = cudaFuncSetAttribute(moe_grouped_gemm_kernel<EPI, NB, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    if (e != cudaSuccess) return e;
+    configured.here() = true;
+  }
+  constexpr int COLS = EPI == EPI_GLU ? BN : NB * BN;
+  return launch_pdl((moe_grouped_gemm_kernel<EPI, NB, STAGES>), dim3((N + COLS - 1) / COLS, tiles), dim3(THREADS), SMEM, stream, 1, A, a_stride, row_pair, top, B,
+                    b_expert_stride, half, C, (long long)N, N, K, tile_expert, act);
 }
 
 }  // namespace
@@ -274,10 +314,11 @@ DLI_EXPORT int dli_moe_grouped_tile_rows() { return BM; }
 
 // ints: scratch of E + 1 (counts) + E + 1 (offsets) + 2 pairs (rank, pos) + tiles (tile_expert) + tiles * BM (row_pair) ints;
 // hidden: [tiles * BM][ff] bfloat16; partial: [tiles * BM][W] float32.  stages: 2 or 3 deep copies, or 0: chosen here.
-DLI_EXPORT int dli_moe_grouped(void* out, const void* x, const int* ids, const float* weights, const void* w_gate_up, const void* w_down, int* ints,
-                               void* hidden, float* partial, int n, int W, int ff, int E, int top, int act, int stages, cudaStream_t stream) {
+// gated: w_up holds an expert's gate rows, then its up rows; else its up rows alone.  ids from E on are identities; shared [n][W] or null.
+DLI_EXPORT int dli_moe_grouped(void* out, const void* x, const int* ids, const float* weights, const void* w_up, const void* w_down, const void* shared,
+                               int* ints, void* hidden, float* partial, int n, int W, int ff, int E, int top, int act, int gated, int stages, cudaStream_t stream) {
   if (n == 0) return 0;
-  if (W < 8 || ff < 8 || (W % 8) || (ff % 8) || E < 1 || top < 1 || ((((uintptr_t)x) | ((uintptr_t)w_gate_up) | ((uintptr_t)w_down) | ((uintptr_t)hidden)) & 15))
+  if (W < 8 || ff < 8 || (W % 8) || (ff % 8) || E < 1 || top < 1 || ((((uintptr_t)x) | ((uintptr_t)w_up) | ((uintptr_t)w_down) | ((uintptr_t)hidden) | ((uintptr_t)out) | ((uintptr_t)shared) | ((uintptr_t)partial)) & 15))
     return DLI_ERR_UNSUPPORTED;
   const int pairs = n * top;
   const int tiles = dli_moe_grouped_tiles(pairs, E);
@@ -298,42 +339,27 @@ DLI_EXPORT int dli_moe_grouped(void* out, const void* x, const int* ids, const f
     e = launch_pdl((moe_init_kernel), dim3((E + 1 + n_maps + 255) / 256 < 1024 ? (E + 1 + n_maps + 255) / 256 : 1024), dim3(256), 0, stream, 1, counts, E + 1,
                    tile_expert, n_maps);
     if (e != cudaSuccess) return (int)e;
-    e = launch_pdl((moe_count_kernel), dim3((pairs + 255) / 256), dim3(256), 0, stream, 1, ids, pairs, counts, rank);
+    e = launch_pdl((moe_count_kernel), dim3((pairs + 255) / 256), dim3(256), 0, stream, 1, ids, pairs, E, counts, rank);
     if (e != cudaSuccess) return (int)e;
     e = launch_pdl((moe_plan_kernel), dim3(1), dim3(256), 0, stream, 1, (const int*)counts, E, offsets, tile_expert);
     if (e != cudaSuccess) return (int)e;
-    e = launch_pdl((moe_scatter_kernel), dim3((pairs + 255) / 256), dim3(256), 0, stream, 1, ids, (const int*)rank, (const int*)offsets, pairs, pos, row_pair);
+    e = launch_pdl((moe_scatter_kernel), dim3((pairs + 255) / 256), dim3(256), 0, stream, 1, ids, (const int*)rank, (const int*)offsets, pairs, E, pos, row_pair);
     if (e != cudaSuccess) return (int)e;
   }
-  constexpr int TILE_BYTES = TILE_ELEMS * (int)sizeof(bf16);
-  static OncePerDevice configured;
-  if (!configured.here()) {
-    e = cudaFuncSetAttribute(moe_grouped_gemm_kernel<true, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * 3 * TILE_BYTES);
-    if (e != cudaSuccess) return (int)e;
-    e = cudaFuncSetAttribute(moe_grouped_gemm_kernel<false, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * 2 * TILE_BYTES);
-    if (e != cudaSuccess) return (int)e;
-    e = cudaFuncSetAttribute(moe_grouped_gemm_kernel<true, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * 3 * TILE_BYTES);
-    if (e != cudaSuccess) return (int)e;
-    e = cudaFuncSetAttribute(moe_grouped_gemm_kernel<false, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * 2 * TILE_BYTES);
-    if (e != cudaSuccess) return (int)e;
-    configured.here() = true;
-  }
-  const int deep = stages == 2 || stages == 3 ? stages : (pairs > 16 * E ? 2 : 3);  // many rows an expert: the products bound the time, not the stream
-  const dim3 grid_up((ff + BN - 1) / BN, tiles), grid_down((W + BN - 1) / BN, tiles);
-  if (deep == 3) {
-    e = launch_pdl((moe_grouped_gemm_kernel<true, 3>), grid_up, dim3(THREADS), 3 * 3 * TILE_BYTES, stream, 1, (const bf16*)x, (long long)W, (const int*)row_pair, top,
-                   (const bf16*)w_gate_up, (long long)2 * ff * W, ff, hidden, (long long)ff, ff, W, (const int*)tile_expert, act);
-    if (e != cudaSuccess) return (int)e;
-    e = launch_pdl((moe_grouped_gemm_kernel<false, 3>), grid_down, dim3(THREADS), 3 * 2 * TILE_BYTES, stream, 1, (const bf16*)hidden, (long long)ff,
-                   (const int*)nullptr, top, (const bf16*)w_down, (long long)W * ff, 0, (void*)partial, (long long)W, W, ff, (const int*)tile_expert, 0);
-  } else {
-    e = launch_pdl((moe_grouped_gemm_kernel<true, 2>), grid_up, dim3(THREADS), 2 * 3 * TILE_BYTES, stream, 1, (const bf16*)x, (long long)W, (const int*)row_pair, top,
-                   (const bf16*)w_gate_up, (long long)2 * ff * W, ff, hidden, (long long)ff, ff, W, (const int*)tile_expert, act);
-    if (e != cudaSuccess) return (int)e;
-    e = launch_pdl((moe_grouped_gemm_kernel<false, 2>), grid_down, dim3(THREADS), 2 * 2 * TILE_BYTES, stream, 1, (const bf16*)hidden, (long long)ff,
-                   (const int*)nullptr, top, (const bf16*)w_down, (long long)W * ff, 0, (void*)partial, (long long)W, W, ff, (const int*)tile_expert, 0);
-  }
+  const bool many = stages == 2 || (stages != 3 && pairs > 16 * E);  // many rows an expert: the products bound the time, not the stream of the matrices
+  const bf16 *bx = (const bf16*)x, *up = (const bf16*)w_up, *down = (const bf16*)w_down;
+#define DLI_UP(EPI, NB, ST) \
+  launch_grouped<EPI, NB, ST>(bx, W, row_pair, top, up, (long long)(gated ? 2 : 1) * ff * W, ff, hidden, ff, W, tile_expert, tiles, act, stream)
+#define DLI_DOWN(NB, ST) \
+  launch_grouped<EPI_F32, NB, ST>((const bf16*)hidden, ff, nullptr, top, down, (long long)W * ff, 0, partial, W, ff, tile_expert, tiles, 0, stream)
+  if (gated) e = many ? DLI_UP(EPI_GLU, 2, 2) : DLI_UP(EPI_GLU, 2, 3);
+  else e = !many ? DLI_UP(EPI_ACT, 1, 3) : ff > BN ? DLI_UP(EPI_ACT, 2, 2) : DLI_UP(EPI_ACT, 1, 2);
   if (e != cudaSuccess) return (int)e;
-  e = launch_pdl((moe_combine_kernel), dim3(n), dim3(W >= 1024 ? 256 : 128), 0, stream, 1, (bf16*)out, (const float*)partial, (const int*)pos, weights, W, top);
+  e = !many ? DLI_DOWN(1, 3) : W > BN ? DLI_DOWN(2, 2) : DLI_DOWN(1, 2);
+  if (e != cudaSuccess) return (int)e;
+#undef DLI_UP
+#undef DLI_DOWN
+  e = launch_pdl((moe_combine_kernel), dim3(n), dim3(W >= 2048 ? 256 : W >= 1024 ? 128 : 64), 0, stream, 1, (bf16*)out, (const float*)partial, (const int*)pos, ids, weights, bx,
+                 (const bf16*)shared, W, E, top);
   return (int)e;
 }

@@ -1,7 +1,7 @@
 """Chooses the attention kernels of a step.
 
 float32: the CUDA-core kernel for every token (true 32-bit).  bfloat16: tensor-core kernels
-where the head size is a multiple of 16 — one launch for the sequences that bring one token
+where the sizes of keys and values are multiples of 16 — one launch for the sequences that bring one token
 (keys split across CTAs when there are few sequences and long contexts) and one for the longer
 portions, which takes the tcgen05 + TMA kernel when head and page size allow it and the
 mma.sync kernel otherwise — and the CUDA-core kernel for any other head size.
@@ -67,11 +67,20 @@ def choose_splits(num_seqs: int, ctas_per_seq: int, max_kv_len: int, wave: int |
     return max(range(1, min(4, most) + 1), key=score)
 
 
-def decode_splits(num_seqs: int, num_heads: int, nkv: int, head_dim: int, page_size: int, max_kv_len: int) -> int:
-    """Key splits of the decode kernel that will serve these sizes."""
+def _slab_kernels(head_dim: int, one_pool: bool) -> bool:
+    """Whether the TMA-fed kernels may serve these rows (``ops.decode_tma_supported`` and its sister also look at the page size).
+    They copy keys and values separately: where the values lie in the keys' rows (``one_pool``) they are only taken at the sizes
+    that fill their slabs, and the mma.sync kernels, which then copy a row once, serve the rest."""
+    return not one_pool or head_dim in (64, 128)
+
+
+def decode_splits(num_seqs: int, num_heads: int, nkv: int, head_dim: int, page_size: int, max_kv_len: int, value_dim: int | None = None,
+                  one_pool: bool = False) -> int:
+    """Key splits of the decode kernel that will serve these sizes (``value_dim`` None: values as long as keys)."""
     ctas_per_seq = nkv * -(-(num_heads // nkv) // 16)
-    tma = ops.decode_tma_supported(head_dim, page_size)
-    wave = one_wave(4 if head_dim <= 64 else 2) if tma else one_wave(2)
+    value_dim = value_dim or head_dim
+    tma = ops.decode_tma_supported(head_dim, page_size, value_dim) and _slab_kernels(head_dim, one_pool)
+    wave = one_wave(4 if max(head_dim, value_dim) <= 64 else 2) if tma else one_wave(2)
     splits = choose_splits(num_seqs, ctas_per_seq, max_kv_len, wave, fill_last_wave=not tma)
     if tma and splits > 8:  # a cluster merges its splits on the chip: 16 of them for one or two sequences' head groups, else 8
         pairs = num_seqs * ctas_per_seq
@@ -95,24 +104,26 @@ def paged_attention(out: torch.Tensor, qkv: torch.Tensor, cache, batch, num_head
     query head): then slopes[h] * (position - key position) is taken off (None: neither)."""
     group = batch.group(cache.group)
     _, nkv, _, d = cache.k.shape
+    dv = cache.v.shape[3]  # a value's size may differ from a key's
+    one_pool = cache.v.data_ptr() == cache.k.data_ptr()
     bend = {"softcap": softcap, "slopes": slopes} if softcap or slopes is not None else {}
-    if out.dtype != torch.bfloat16 or not ops.mma_head_dim_supported(d):
+    if out.dtype != torch.bfloat16 or not (ops.mma_head_dim_supported(d) and ops.mma_head_dim_supported(dv)):
         ops.paged_attention_simt(out, qkv, cache.k, cache.v, group.block_tables, batch.seq_of_token, batch.positions,
                                  num_heads, scale, window, sink, **bend)
         return
     singles, total = batch.num_single, batch.num_seqs
     if singles:
-        tma = ops.decode_tma_supported(d, cache.page_size)
-        splits = splits or decode_splits(singles, num_heads, nkv, d, cache.page_size, batch.max_kv_len_single)
+        tma = ops.decode_tma_supported(d, cache.page_size, dv) and _slab_kernels(d, one_pool)
+        splits = splits or decode_splits(singles, num_heads, nkv, d, cache.page_size, batch.max_kv_len_single, dv, one_pool)
         scratch = None
         if splits > 1:
             rows = singles * num_heads
-            scratch = (torch.empty(rows * splits * d, dtype=torch.float32, device=out.device),
+            scratch = (torch.empty(rows * splits * dv, dtype=torch.float32, device=out.device),
                        torch.empty(rows * splits * 2, dtype=torch.float32, device=out.device))
         kernel = ops.paged_decode_tma if tma else ops.paged_attention_mma
         args = (out, qkv, cache.k, cache.v, group.block_tables, batch.q_start, batch.kv_len, 0, singles) + (() if tma else (1,))
         kernel(*args, 0, num_heads, scale, window, splits, scratch, *((batch.max_kv_len_single,) if tma else ()), sink=sink, **bend)
-    if total > singles and ops.prefill_tc_supported(d, cache.page_size):
+    if total > singles and ops.prefill_tc_supported(d, cache.page_size, dv) and _slab_kernels(d, one_pool):
         ops.paged_prefill_tc(out, qkv, cache.k, cache.v, group.block_tables, batch.q_start, batch.kv_len, singles, total - singles,
                              batch.max_q_len, num_heads, scale, window, sink=sink, **bend)
     elif total > singles:

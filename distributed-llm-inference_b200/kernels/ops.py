@@ -342,33 +342,42 @@ def paged_attention_simt(
     """Causal attention of every token over its sequence's pages, on CUDA cores.  ``sink``: see ``_sink``.  ``softcap`` c: a score s
     (after the scale) becomes c tanh(s / c); ``slopes``: then slopes[h] * (position - key position) is taken off.
 
-    out [n, nh * d]; queries are the first nh * d columns of qkv; pools [pages, nkv, page_size, d];
-    block_tables [seqs, max_blocks]; a token at position p reads keys max(0, p - window + 1) .. p.
+    out [n, nh * dv]; queries are the first nh * d columns of qkv; pools [pages, nkv, page_size, d] and [.., dv] (the values' size may
+    differ from the keys'); block_tables [seqs, max_blocks]; a token at position p reads keys max(0, p - window + 1) .. p.
     """
     _need(out, "out"), _need(qkv, "qkv", out.dtype), _need(k_pool, "k_pool", out.dtype), _need(v_pool, "v_pool", out.dtype)
     _need(block_tables, "block_tables", torch.int32), _need(seq_of_token, "seq_of_token", torch.int32)
     _need(positions, "positions", torch.int32)
     n = out.shape[0]
     _, nkv, page_size, d = k_pool.shape
-    if out.dtype not in DT_CODE or out.shape[1] != num_heads * d or qkv.shape[0] != n or qkv.shape[1] < num_heads * d:
+    dv = v_pool.shape[3]
+    if (out.dtype not in DT_CODE or out.shape[1] != num_heads * dv or qkv.shape[0] != n or qkv.shape[1] < num_heads * d
+            or v_pool.shape[:3] != k_pool.shape[:3]):
         raise KernelError("paged_attention_simt: shapes or dtype do not agree")
-    if d > SIMT_MAX_HEAD_DIM or num_heads % nkv:
+    if d > SIMT_MAX_HEAD_DIM or dv > SIMT_MAX_HEAD_DIM or num_heads % nkv:
         raise KernelError(f"paged_attention_simt: head_dim {d} (<= {SIMT_MAX_HEAD_DIM}) / heads {num_heads} per kv head {nkv} not supported")
     f = _fn(
         "attention_simt.cu", "dli_paged_attention_simt",
-        [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 6
+        [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 7
         + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p],
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), block_tables.shape[1],
-          _ptr(seq_of_token), _ptr(positions), n, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
+          _ptr(seq_of_token), _ptr(positions), n, num_heads, nkv, d, dv, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
           *_bend(softcap, slopes, num_heads), DT_CODE[out.dtype], _stream()),
         "paged_attention_simt",
     )
 
 
-def prefill_tc_supported(head_dim: int, page_size: int) -> bool:
-    return head_dim in (64, 128) and page_size in (8, 16, 32, 64, 128)
+def _tma_rows(head_dim: int, value_dim: int | None) -> bool:
+    """Whether the TMA-fed attention kernels take keys and values of these sizes: multiples of 8 up to 128.  They work on slabs of 64
+    columns, so rows much shorter than that are left to the kernels built for their size."""
+    value_dim = value_dim or head_dim
+    return head_dim % 8 == 0 and value_dim % 8 == 0 and 32 < max(head_dim, value_dim) <= 128
+
+
+def prefill_tc_supported(head_dim: int, page_size: int, value_dim: int | None = None) -> bool:
+    return _tma_rows(head_dim, value_dim) and page_size in (8, 16, 32, 64, 128)
 
 
 def paged_prefill_tc(
@@ -391,22 +400,23 @@ def paged_prefill_tc(
     slopes: torch.Tensor | None = None,
 ) -> None:
     """bfloat16 attention for prompt portions on tcgen05 tensor cores with TMA-fed pages
-    (head size 64 or 128; page sizes 8, 16, 32, 64, 128).  Arguments as paged_attention_mma.
-    ``query_tiles`` (head size 64): 1 or 2 tiles of 128 (token, head) rows per CTA; 0 lets the launcher choose (two
+    (key and value rows of up to 128 numbers, multiples of 8; page sizes 8, 16, 32, 64, 128).  Arguments as paged_attention_mma.
+    ``query_tiles`` (rows of 64): 1 or 2 tiles of 128 (token, head) rows per CTA; 0 lets the launcher choose (two
     when a sequence brings more tokens than one tile holds)."""
     for t, name in ((out, "out"), (qkv, "qkv"), (k_pool, "k_pool"), (v_pool, "v_pool")):
         _need(t, name, torch.bfloat16)
     _need(block_tables, "block_tables", torch.int32), _need(q_start, "q_start", torch.int32), _need(kv_len, "kv_len", torch.int32)
     pages, nkv, page_size, d = k_pool.shape
-    if not prefill_tc_supported(d, page_size):
-        raise KernelError(f"paged_prefill_tc: head_dim {d} (64 or 128) or page size {page_size} (8..128, dividing 128) not supported")
-    if out.shape[1] != num_heads * d or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv or k_pool.shape != v_pool.shape:
+    dv = v_pool.shape[3]
+    if not prefill_tc_supported(d, page_size, dv):
+        raise KernelError(f"paged_prefill_tc: rows of {d} and {dv} numbers (multiples of 8 up to 128) or page size {page_size} (8..128, dividing 128) not supported")
+    if out.shape[1] != num_heads * dv or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv or k_pool.shape[:3] != v_pool.shape[:3]:
         raise KernelError("paged_prefill_tc: shapes do not agree")
     if seq0 + num_seqs > kv_len.numel() or q_start.numel() != kv_len.numel() + 1:
         raise KernelError("paged_prefill_tc: sequence range outside the batch")
     f = _fn(
         "attention_tc.cu", "dli_paged_prefill_tc",
-        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8
+        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 9
         + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p],
         _bent_defines(softcap, slopes),
     )
@@ -414,14 +424,14 @@ def paged_prefill_tc(
         raise KernelError("paged_prefill_tc: query_tiles is 0 (choose), 1 or 2")
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), pages, _ptr(block_tables), block_tables.shape[1],
-          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, max_q_len, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
+          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, max_q_len, num_heads, nkv, d, dv, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
           *_bend(softcap, slopes, num_heads), query_tiles, _stream()),
         "paged_prefill_tc",
     )
 
 
-def decode_tma_supported(head_dim: int, page_size: int) -> bool:
-    return head_dim in (64, 128) and page_size % 8 == 0 and (page_size == 8 or page_size % 16 == 0) and page_size <= 256
+def decode_tma_supported(head_dim: int, page_size: int, value_dim: int | None = None) -> bool:
+    return _tma_rows(head_dim, value_dim) and page_size % 8 == 0 and (page_size == 8 or page_size % 16 == 0) and page_size <= 256
 
 
 def paged_decode_tma(
@@ -445,17 +455,18 @@ def paged_decode_tma(
     softcap: float | None = None,
     slopes: torch.Tensor | None = None,
 ) -> None:
-    """bfloat16 attention of single-token sequences whose keys and values arrive by TMA (head size
-    64 or 128; page sizes 8, 16, 32, ...).  Arguments as paged_attention_mma with max_q_len = 1.
+    """bfloat16 attention of single-token sequences whose keys and values arrive by TMA (rows of
+    up to 128 numbers, multiples of 8, the values' size may differ from the keys'; page sizes 8, 16, 32, ...).  Arguments as paged_attention_mma with max_q_len = 1.
     ``max_kv_len``: the longest sequence, if the host knows it (a hint: with few CTAs and long runs of keys
     the launcher gives a CTA eight warps instead of four); 0 if not."""
     for t, name in ((out, "out"), (qkv, "qkv"), (k_pool, "k_pool"), (v_pool, "v_pool")):
         _need(t, name, torch.bfloat16)
     _need(block_tables, "block_tables", torch.int32), _need(q_start, "q_start", torch.int32), _need(kv_len, "kv_len", torch.int32)
     pages, nkv, page_size, d = k_pool.shape
-    if not decode_tma_supported(d, page_size):
-        raise KernelError(f"paged_decode_tma: head_dim {d} (64 or 128) or page size {page_size} not supported")
-    if out.shape[1] != num_heads * d or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv or k_pool.shape != v_pool.shape:
+    dv = v_pool.shape[3]
+    if not decode_tma_supported(d, page_size, dv):
+        raise KernelError(f"paged_decode_tma: rows of {d} and {dv} numbers (multiples of 8 up to 128) or page size {page_size} not supported")
+    if out.shape[1] != num_heads * dv or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv or k_pool.shape[:3] != v_pool.shape[:3]:
         raise KernelError("paged_decode_tma: shapes do not agree")
     if seq0 + num_seqs > kv_len.numel() or q_start.numel() != kv_len.numel() + 1:
         raise KernelError("paged_decode_tma: sequence range outside the batch")
@@ -466,17 +477,17 @@ def paged_decode_tma(
         acc, ml = scratch
         _need(acc, "scratch[0]", torch.float32), _need(ml, "scratch[1]", torch.float32)
         rows = (first_row + num_seqs) * num_heads
-        if acc.numel() < rows * splits * d or ml.numel() < rows * splits * 2:
+        if acc.numel() < rows * splits * dv or ml.numel() < rows * splits * 2:
             raise KernelError("paged_decode_tma: scratch too small")
     f = _fn(
         "attention_tc.cu", "dli_paged_decode_tma",
-        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8
+        [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 9
         + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p],
         _bent_defines(softcap, slopes),
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), pages, _ptr(block_tables), block_tables.shape[1],
-          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, first_row, num_heads, nkv, d, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
+          _ptr(q_start), _ptr(kv_len), seq0, num_seqs, first_row, num_heads, nkv, d, dv, page_size, int(window or 0), scale, _sink(sink), _sink_heads(sink, num_heads),
           *_bend(softcap, slopes, num_heads), splits, _ptr(acc), _ptr(ml), int(max_kv_len), _stream()),
         "paged_decode_tma",
     )
@@ -597,16 +608,17 @@ def paged_attention_mma(
     Queries are the first nh * d columns of qkv; a sequence's tokens sit in rows
     q_start[s] .. q_start[s + 1] at positions kv_len[s] - q_len .. kv_len[s] - 1.  With
     ``splits`` > 1 (single-token sequences only) the keys are cut into that many runs;
-    ``scratch`` = (float32 [rows * splits * d], float32 [rows * splits * 2]) with
-    rows = (first_row + num_seqs) * nh holds the partial results.
+    ``scratch`` = (float32 [rows * splits * dv], float32 [rows * splits * 2]) with
+    rows = (first_row + num_seqs) * nh holds the partial results; dv is the size of a value row, which may differ from d.
     """
     for t, name in ((out, "out"), (qkv, "qkv"), (k_pool, "k_pool"), (v_pool, "v_pool")):
         _need(t, name, torch.bfloat16)
     _need(block_tables, "block_tables", torch.int32), _need(q_start, "q_start", torch.int32), _need(kv_len, "kv_len", torch.int32)
     _, nkv, page_size, d = k_pool.shape
-    if not mma_head_dim_supported(d):
-        raise KernelError(f"paged_attention_mma: head_dim {d} is not a multiple of 16 in [16, 256]")
-    if out.shape[1] != num_heads * d or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv:
+    dv = v_pool.shape[3]
+    if not (mma_head_dim_supported(d) and mma_head_dim_supported(dv)):
+        raise KernelError(f"paged_attention_mma: a row of {d} or {dv} numbers is not a multiple of 16 in [16, 256]")
+    if out.shape[1] != num_heads * dv or qkv.shape[0] != out.shape[0] or qkv.shape[1] < num_heads * d or num_heads % nkv or v_pool.shape[:3] != k_pool.shape[:3]:
         raise KernelError("paged_attention_mma: shapes do not agree")
     if seq0 + num_seqs > kv_len.numel() or q_start.numel() != kv_len.numel() + 1:
         raise KernelError("paged_attention_mma: sequence range outside the batch")
@@ -617,13 +629,13 @@ def paged_attention_mma(
         acc, ml = scratch
         _need(acc, "scratch[0]", torch.float32), _need(ml, "scratch[1]", torch.float32)
         rows = (first_row + num_seqs) * num_heads
-        if acc.numel() < rows * splits * d or ml.numel() < rows * splits * 2:
+        if acc.numel() < rows * splits * dv or ml.numel() < rows * splits * 2:
             raise KernelError("paged_attention_mma: scratch too small")
     f = _fn(
         "attention_mma.cu", "dli_paged_attention_mma",
         [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]
         + [c_int] * 8 + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
-        _bent_defines(softcap, slopes, {"HEAD_DIM": d}),
+        _bent_defines(softcap, slopes, {"HEAD_DIM": d} if dv == d else {"HEAD_DIM": d, "VALUE_DIM": dv}),
     )
     _check(
         f(_ptr(out), _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_tables), block_tables.shape[1],
@@ -1010,38 +1022,47 @@ ELEMENTWISE_ACTIVATIONS = {**ACTIVATIONS, "tanh": 3}  # what the kernel of its o
 def qk_norm_rotary_store(proj: torch.Tensor, wq: torch.Tensor | None, wk: torch.Tensor | None, eps: float, positions: torch.Tensor,
                          inv_freq: torch.Tensor | None, slots: torch.Tensor | None, k_pool: torch.Tensor | None,
                          v_pool: torch.Tensor | None, num_heads: int, num_kv_heads: int, head_dim: int, rotary_dim: int,
-                         page_size: int, write_kv: bool = True, values_from_keys: bool = True) -> torch.Tensor:
-    """proj [n, >= (nh + nkv) d]: q | k (| v, when the values are not the keys) as projected.  With ``wq`` and ``wk``
-    q and k are each divided by the RMS of the whole projection (all heads together, ``eps`` inside the root) and
-    multiplied by these weights [nh d], [nkv d]; then rotary (rotate-half pairing) on the first ``rotary_dim``
-    dimensions of every head.  Returns q [n, nh d]; k goes to ``k_pool`` and the values — the keys as projected
-    (``values_from_keys``) or the columns behind k — to ``v_pool`` [pages, nkv, page_size, d] at ``slots``."""
+                         page_size: int, write_kv: bool = True, values_from_keys: bool = True, value_dim: int | None = None,
+                         per_head: bool = False, row: int | None = None) -> torch.Tensor:
+    """proj [n, >= (nh + nkv) d]: q | k (| v, when the values are not the keys) as projected; without ``write_kv`` only q is read.
+    With ``wq`` (and ``wk``) q and k are each divided by the RMS of the whole projection (all heads together, ``eps`` inside the
+    root) and multiplied by these weights [nh d], [nkv d] — or, with ``per_head``, head by head, the weights [d] shared by all heads;
+    then rotary (rotate-half pairing) on the first ``rotary_dim`` dimensions of every head.  Returns q [n, nh row]; k goes to
+    ``k_pool`` [pages, nkv, page_size, row] and the values — the keys as projected (``values_from_keys``) or the nkv ``value_dim``
+    columns behind k — to ``v_pool`` [pages, nkv, page_size, >= value_dim] at ``slots``.  ``row`` (default head_dim): how many numbers a
+    head's row has as it leaves; what lies beyond head_dim (value_dim) is zero."""
     _need(positions, "positions", torch.int32)
     if proj.dtype not in DT_CODE or proj.dim() != 2 or proj.stride(1) != 1 or not proj.is_cuda:
         raise KernelError("qk_norm_rotary_store: proj must be a CUDA matrix with unit column stride")
     n = proj.shape[0]
-    need_cols = (num_heads + (1 if values_from_keys else 2) * num_kv_heads) * head_dim
-    if proj.shape[1] < need_cols or positions.numel() != n:
+    dv, row = value_dim or head_dim, row or head_dim
+    need_cols = num_heads * head_dim + (num_kv_heads * (head_dim + (0 if values_from_keys else dv)) if write_kv else 0)
+    if proj.shape[1] < need_cols or positions.numel() != n or row < head_dim or (values_from_keys and dv != head_dim):
         raise KernelError("qk_norm_rotary_store: shapes do not agree")
     normed = wq is not None
     if normed:
-        _need(wq, "wq", torch.float32), _need(wk, "wk", torch.float32)
-        if wq.numel() != num_heads * head_dim or wk.numel() != num_kv_heads * head_dim:
-            raise KernelError("qk_norm_rotary_store: norm weights must cover the whole projections")
+        _need(wq, "wq", torch.float32)
+        if write_kv:
+            _need(wk, "wk", torch.float32)
+        if wq.numel() != (1 if per_head else num_heads) * head_dim or (write_kv and wk.numel() != (1 if per_head else num_kv_heads) * head_dim):
+            raise KernelError("qk_norm_rotary_store: norm weights must cover the whole projections, or one head with per_head")
     if rotary_dim:
         _need(inv_freq, "inv_freq", torch.float32)
         if inv_freq.numel() != rotary_dim // 2:
             raise KernelError("qk_norm_rotary_store: inv_freq must have rotary_dim / 2 entries")
+    vrow = dv
     if write_kv:
         _need(slots, "slots", torch.int32), _need(k_pool, "k_pool", proj.dtype), _need(v_pool, "v_pool", proj.dtype)
-        if tuple(k_pool.shape[1:]) != (num_kv_heads, page_size, head_dim) or k_pool.shape != v_pool.shape or slots.numel() != n:
-            raise KernelError("qk_norm_rotary_store: pool layout must be [pages, kv_heads, page_size, head_dim]")
-    q = torch.empty((n, num_heads * head_dim), dtype=proj.dtype, device=proj.device)
+        vrow = v_pool.shape[3]
+        if tuple(k_pool.shape[1:]) != (num_kv_heads, page_size, row) or k_pool.shape[:3] != v_pool.shape[:3] or vrow < dv or slots.numel() != n:
+            raise KernelError("qk_norm_rotary_store: pool layout must be [pages, kv_heads, page_size, row]")
+    q = torch.empty((n, num_heads * row), dtype=proj.dtype, device=proj.device)
     f = _fn("attention_prep.cu", "dli_qk_norm_rotary_store",
-            [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 10 + [c_void_p])
-    _check(f(_ptr(q), _ptr(proj), proj.stride(0), _ptr(wq), _ptr(wk), eps, _ptr(positions), _ptr(inv_freq if rotary_dim else None),
+            [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 13 + [c_void_p])
+    norm = 0 if not normed else (2 if per_head else 1)
+    _check(f(_ptr(q), _ptr(proj), proj.stride(0), _ptr(wq), _ptr(wk if write_kv else None), eps, _ptr(positions), _ptr(inv_freq if rotary_dim else None),
              _ptr(slots if write_kv else None), _ptr(k_pool if write_kv else None), _ptr(v_pool if write_kv else None), n, num_heads,
-             num_kv_heads, head_dim, rotary_dim, page_size, int(write_kv), int(normed), int(values_from_keys), DT_CODE[proj.dtype], _stream()),
+             num_kv_heads, head_dim, dv, row, vrow, rotary_dim, page_size, int(write_kv), norm, int(values_from_keys), DT_CODE[proj.dtype], _stream()),
            "qk_norm_rotary_store")
     return q
 
@@ -1719,7 +1740,7 @@ def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, 
         raise KernelError("matrix_memory_scan: form is walk or chunk")
 
 
-# ------------------------------------------------------------------ routed mixture of gated feed-forwards
+# ------------------------------------------------------------------ routed mixture of small feed-forwards
 
 MOE_MAX_TOP = 32
 MOE_GROUPED_TILE_ROWS = 64  # BM of csrc/moe_grouped.cu
@@ -1733,7 +1754,7 @@ def moe_grouped_supported(tokens: int, W: int, ff: int, dtype: torch.dtype) -> b
 MOE_PAIR_CHUNK = 8192  # tokens a launch of the pair kernels takes (their grids count (token, expert) pairs along y)
 
 
-MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1}
+MOE_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
 
 
 def moe_route(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, group_count: int,
@@ -1742,7 +1763,8 @@ def moe_route(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router:
     With ``group_count`` > 1 the experts form equal groups of neighbours, a group's mark is the sum of its two largest choice scores,
     and only experts of the ``group_keep`` best groups are eligible.  ids [n, top] int32: the eligible experts with the largest choice
     scores, best first (ties: the lower index); weights [n, top] float32 = s[ids] / (their sum + 1e-20) * scale.
-    ``score`` = ``"softmax_chosen"``: choice = z + correction, and the weights are softmax(choice[ids]) * scale."""
+    ``score`` = ``"softmax_chosen"``: choice = z + correction, and the weights are softmax(choice[ids]) * scale.
+    ``score`` = ``"softmax"``: s = softmax(z) over all experts, choice = s + correction, and the weights are s[ids] * scale."""
     _need(ids, "ids", torch.int32), _need(weights, "weights", torch.float32), _need(x, "x"), _need(router, "router", torch.float32)
     _need(correction, "correction", torch.float32)
     n, W = x.shape
@@ -1755,21 +1777,27 @@ def moe_route(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router:
              _stream()), "moe_route")
 
 
-def moe_experts(out: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                activation: str = "silu", stages: int = 0) -> None:
-    """out[t] = sum_k weights[t, k] * down_e(act(gate_e x[t]) * (up_e x[t])), e = ids[t, k], added in the order of k in float32.
-    w_gate_up [E, 2 ff, W] (an expert's gate rows, then its up rows), w_down [E, W, ff].  The two inner sums are rounded to the
-    activation dtype before the activation, and so is their product.  ``stages`` (2, 3; 0: chosen from the step's shape): how deep
-    the grouped products' asynchronous copies run."""
+def moe_experts(out: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
+                activation: str = "silu", stages: int = 0, gated: bool = True, shared: torch.Tensor | None = None) -> None:
+    """out[t] = sum_k weights[t, k] * y_k (+ shared[t]), added in the order of k in float32.  With e = ids[t, k] below E = len(w_down):
+    y_k = down_e(act(gate_e x[t]) * (up_e x[t])), or down_e(act(up_e x[t])) without ``gated``; from E on the expert is the identity,
+    y_k = x[t].  w_up [E, 2 ff, W] (an expert's gate rows, then its up rows) or [E, ff, W], w_down [E, W, ff].  The inner sums are
+    rounded to the activation dtype before the activation, and so is what goes down.  ``activation``: one of GLU_ACTIVATIONS, or of
+    ACTIVATIONS without a gate.  ``stages`` (2, 3; 0: chosen from the step's shape): how deep the grouped products' asynchronous
+    copies run."""
     _need(out, "out"), _need(x, "x", out.dtype), _need(ids, "ids", torch.int32), _need(weights, "weights", torch.float32)
-    _need(w_gate_up, "w_gate_up", out.dtype), _need(w_down, "w_down", out.dtype)
+    _need(w_up, "w_up", out.dtype), _need(w_down, "w_down", out.dtype)
     n, W = x.shape
     top = ids.shape[1]
-    E, ff2, _ = w_gate_up.shape
-    ff = ff2 // 2
-    if (out.dtype not in DT_CODE or tuple(out.shape) != (n, W) or w_gate_up.shape[2] != W or tuple(w_down.shape) != (E, W, ff) or tuple(ids.shape) != (n, top)
-            or tuple(weights.shape) != (n, top) or activation not in GLU_ACTIVATIONS):
+    E, _, ff = w_down.shape
+    known = GLU_ACTIVATIONS if gated else ACTIVATIONS
+    if (out.dtype not in DT_CODE or tuple(out.shape) != (n, W) or tuple(w_up.shape) != (E, (2 if gated else 1) * ff, W) or w_down.shape[1] != W
+            or tuple(ids.shape) != (n, top) or tuple(weights.shape) != (n, top) or activation not in known):
         raise KernelError("moe_experts: shapes, dtype or activation do not agree")
+    if shared is not None:
+        _need(shared, "shared", out.dtype)
+        if tuple(shared.shape) != (n, W):
+            raise KernelError("moe_experts: the shared expert's output must be [n, W]")
     global launch_count
     if moe_grouped_supported(n, W, ff, out.dtype):
         # many tokens: the pairs sorted by expert, two grouped products on the tensor cores (csrc/moe_grouped.cu)
@@ -1778,16 +1806,16 @@ def moe_experts(out: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: 
         ints = torch.empty(2 * (E + 1) + 2 * n * top + tiles + rows, dtype=torch.int32, device=out.device)
         hidden = torch.empty((rows, ff), dtype=out.dtype, device=out.device)
         partial = torch.empty((rows, W), dtype=torch.float32, device=out.device)
-        g = _fn("moe_grouped.cu", "dli_moe_grouped", [c_void_p] * 9 + [c_int] * 7 + [c_void_p])
-        _check(g(_ptr(out), _ptr(x), _ptr(ids), _ptr(weights), _ptr(w_gate_up), _ptr(w_down), _ptr(ints), _ptr(hidden), _ptr(partial), n, W, ff, E, top,
-                 GLU_ACTIVATIONS[activation], int(stages), _stream()), "moe_experts")
+        g = _fn("moe_grouped.cu", "dli_moe_grouped", [c_void_p] * 10 + [c_int] * 8 + [c_void_p])
+        _check(g(_ptr(out), _ptr(x), _ptr(ids), _ptr(weights), _ptr(w_up), _ptr(w_down), _ptr(shared), _ptr(ints), _ptr(hidden), _ptr(partial), n, W, ff, E,
+                 top, known[activation], int(gated), int(stages), _stream()), "moe_experts")
         launch_count += 3 if n * top <= 2048 else 6  # four kernels a call (one block sorts up to 2,048 pairs), else seven
         return
-    f = _fn("moe.cu", "dli_moe_pairs", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p] + [c_int] * 6 + [c_void_p])
+    f = _fn("moe.cu", "dli_moe_pairs", [c_void_p] * 8 + [c_int] * 8 + [c_void_p])
     step = max(1, min(MOE_PAIR_CHUNK, 65535 // top))
     hidden = torch.empty((min(n, step) * top, ff), dtype=out.dtype, device=out.device)
     for t0 in range(0, n, step):
         m = min(step, n - t0)
-        _check(f(_ptr(out[t0:]), _ptr(hidden), _ptr(x[t0:]), _ptr(ids[t0:]), _ptr(weights[t0:]), _ptr(w_gate_up), _ptr(w_down), m, W, ff, top,
-                 GLU_ACTIVATIONS[activation], DT_CODE[out.dtype], _stream()), "moe_experts")
+        _check(f(_ptr(out[t0:]), _ptr(hidden), _ptr(x[t0:]), _ptr(ids[t0:]), _ptr(weights[t0:]), _ptr(w_up), _ptr(w_down),
+                 _ptr(None if shared is None else shared[t0:]), m, W, ff, E, top, known[activation], int(gated), DT_CODE[out.dtype], _stream()), "moe_experts")
         launch_count += 1  # two kernels a call

@@ -84,17 +84,21 @@ class SinkAttention(Part):
 
     * ``sink`` (a score, or None): exp(sink) is added to every softmax denominator and carries no value,
       p_j = exp(s_j) / (exp(sink) + sum_j exp(s_j)), so a token may attend to nothing;
-    * ``qk_norm_eps`` (or None): q and k are each divided by the RMS of their whole projection (all heads
-      together, before they are cut into heads) and multiplied by a weight of that size, before the position
-      encoding;
+    * ``qk_norm_eps`` (or None): before the position encoding q and k are divided by a root mean square and multiplied by a weight
+      — ``qk_norm``: ``"projection"``, the whole projection's (all heads together, before they are cut into heads; a weight of that
+      size), or ``"head"``, every head's own (one weight of the head's size for all);
     * ``values``: ``"keys"`` — the values are the keys as projected (before norm and rotation; no value matrix)
-      — or ``"projected"`` (a value matrix of its own);
-    * ``gate``: the concatenated heads are multiplied by sigmoid(Wg x) before the output projection.
+      — or ``"projected"`` (a value matrix of its own), whose heads may have a size of their own (``value_dim``);
+    * ``gate``: the concatenated heads are multiplied by sigmoid(Wg x) before the output projection;
+    * ``own_kv`` false: no key and value tensors; the layer's run step reads another step's cache (keys as that layer wrote them,
+      normed and rotated) with its own queries, mask and everything else.
 
+    A cached token is one key row and one value row per KV head; in bfloat16 both are padded with zeros to a multiple of 16, for the
+    tensor-core kernels (and the output projection's matrix with zero columns to match, once, at load).
     One product yields q | k (| v) (| g); one kernel norms, rotates and writes the cache (the position part's
     ``norm_rotate_and_store``); the framework's attention kernels run with their sink argument.
-    params: hidden_size, num_heads, num_kv_heads, head_dim, scale, window, position (PartSpec), sink,
-    qk_norm_eps, values, gate, tensors (names of q, k, v, g, o, q_norm, k_norm)."""
+    params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window, position (PartSpec), sink,
+    qk_norm_eps, qk_norm, values, gate, own_kv, tensors (names of q, k, v, g, o, q_norm, k_norm)."""
 
     graph_capturable = True
     takes_scaled_rows = False
@@ -104,69 +108,83 @@ class SinkAttention(Part):
         p = spec.params
         self.hidden = int(p["hidden_size"])
         self.nh, self.nkv, self.d = int(p["num_heads"]), int(p["num_kv_heads"]), int(p["head_dim"])
+        self.dv = int(p.get("value_dim") or self.d)
+        self.row, self.vrow = self.d, self.dv  # what a page keeps per token and KV head: of keys, of values
+        if env.dtype == torch.bfloat16:
+            self.row, self.vrow = -(-self.d // 16) * 16, -(-self.dv // 16) * 16
         self.scale = float(p["scale"])
         self.window = p.get("window")
         self.sink = None if p.get("sink") is None else float(p["sink"])
         self.qk_norm_eps = None if p.get("qk_norm_eps") is None else float(p["qk_norm_eps"])
+        self.per_head = p.get("qk_norm", "projection") == "head"
         self.values_from_keys = p.get("values", "projected") == "keys"
         self.gated = bool(p.get("gate", False))
-        if p.get("values", "projected") not in ("keys", "projected"):
-            raise ValueError(f"values={p['values']!r} (keys, projected)")
+        self.own_kv = bool(p.get("own_kv", True))
+        if p.get("values", "projected") not in ("keys", "projected") or p.get("qk_norm", "projection") not in ("projection", "head"):
+            raise ValueError(f"values={p.get('values')!r} (keys, projected), qk_norm={p.get('qk_norm')!r} (projection, head)")
         if self.nh % self.nkv:
             raise ValueError(f"num_heads={self.nh} is not a multiple of num_kv_heads={self.nkv}")
+        if self.values_from_keys and self.dv != self.d:
+            raise ValueError(f"values that are the keys have their size: value_dim={self.dv}, head_dim={self.d}")
         self.position = build_part("position", p["position"], env)
         if not hasattr(self.position, "norm_rotate_and_store"):
-            raise ValueError(f"position part {p['position'].kind!r} cannot follow a norm over the whole projection")
+            raise ValueError(f"position part {p['position'].kind!r} cannot follow a norm of queries and keys")
         self.names = {role: tensor_name(spec, role, default) for role, default in (
             ("q", "q_proj.weight"), ("k", "k_proj.weight"), ("v", "v_proj.weight"), ("g", "g_proj.weight"), ("o", "o_proj.weight"),
             ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"))}
+        # the rows of the one product, in order
+        self.sizes = {"q": self.nh * self.d}
+        if self.own_kv:
+            self.sizes["k"] = self.nkv * self.d
+            if not self.values_from_keys:
+                self.sizes["v"] = self.nkv * self.dv
+        self.gate_col = sum(self.sizes.values())
+        if self.gated:
+            self.sizes["g"] = self.nh * self.dv
         self.w_in: torch.Tensor | None = None
         self.wo: torch.Tensor | None = None
         self.wq_norm = self.wk_norm = None
-        self.gate_col = (self.nh + (1 if self.values_from_keys else 2) * self.nkv) * self.d
 
     def children(self):
         return [self.position]
 
     def declare(self):
-        H, d, nm = self.hidden, self.d, self.names
-        out = {nm["q"]: TensorDecl((self.nh * d, H)), nm["k"]: TensorDecl((self.nkv * d, H)), nm["o"]: TensorDecl((H, self.nh * d))}
-        if not self.values_from_keys:
-            out[nm["v"]] = TensorDecl((self.nkv * d, H))
-        if self.gated:
-            out[nm["g"]] = TensorDecl((self.nh * d, H))
+        nm = self.names
+        out = {nm[role]: TensorDecl((rows, self.hidden)) for role, rows in self.sizes.items()}
+        out[nm["o"]] = TensorDecl((self.hidden, self.nh * self.dv))
         if self.qk_norm_eps is not None:
-            out[nm["q_norm"]] = TensorDecl((self.nh * d,), "vector32")
-            out[nm["k_norm"]] = TensorDecl((self.nkv * d,), "vector32")
+            out[nm["q_norm"]] = TensorDecl(((1 if self.per_head else self.nh) * self.d,), "vector32")
+            if self.own_kv:
+                out[nm["k_norm"]] = TensorDecl(((1 if self.per_head else self.nkv) * self.d,), "vector32")
         return out
 
     def load(self, tensors):
         nm = self.names
-        rows = [tensors[nm["q"]], tensors[nm["k"]]]
-        if not self.values_from_keys:
-            rows.append(tensors[nm["v"]])
-        if self.gated:
-            rows.append(tensors[nm["g"]])
-        self.w_in = torch.cat(rows, 0).contiguous()
-        self.wo = tensors[nm["o"]]
+        self.w_in = torch.cat([tensors[nm[role]] for role in self.sizes], 0).contiguous()
+        self.wo = zero_padded_heads(tensors[nm["o"]], self.nh, self.dv, self.vrow)
         if self.qk_norm_eps is not None:
-            self.wq_norm, self.wk_norm = tensors[nm["q_norm"]], tensors[nm["k_norm"]]
+            self.wq_norm, self.wk_norm = tensors[nm["q_norm"]], tensors[nm["k_norm"]] if self.own_kv else None
 
     def cache_need(self):
-        return PagedKVNeed(self.nkv, self.d, self.window)
+        return PagedKVNeed(self.nkv, self.row, self.window, value_dim=None if self.vrow == self.row else self.vrow)
 
     def decode_launch_key(self, num_seqs: int, max_kv_len: int, page_size: int):
-        return attn_kernels.decode_splits(num_seqs, self.nh, self.nkv, self.d, page_size, max_kv_len)
+        return attn_kernels.decode_splits(num_seqs, self.nh, self.nkv, self.row, page_size, max_kv_len, self.vrow)
 
     def forward(self, x: torch.Tensor, batch, cache) -> torch.Tensor:
+        if cache.writes and not self.own_kv:
+            raise RuntimeError("sink_attention: a layer without keys and values of its own reads another step's cache")
         proj = project(x, self.w_in)
         q = self.position.norm_rotate_and_store(proj, self.wq_norm, self.wk_norm, self.qk_norm_eps or 0.0, batch, cache, self.nh, self.nkv,
-                                                cache.writes, self.values_from_keys)
-        out = torch.empty((x.shape[0], self.nh * self.d), dtype=x.dtype, device=x.device)
+                                                cache.writes, self.values_from_keys, value_dim=self.dv, per_head=self.per_head, row=self.row)
+        out = torch.empty((x.shape[0], self.nh * self.vrow), dtype=x.dtype, device=x.device)
         attn_kernels.paged_attention(out, q, cache, batch, self.nh, self.scale, self.window, splits=batch.launch_keys.get(id(self)),
                                      sink=self.sink)
         if self.gated:
-            ops.sigmoid_gate(out, proj[:, self.gate_col : self.gate_col + self.nh * self.d])
+            gate = proj[:, self.gate_col : self.gate_col + self.nh * self.dv]
+            if self.vrow != self.dv:  # the padding's gates are of no consequence: what they multiply is zero
+                gate = torch.nn.functional.pad(gate.reshape(-1, self.nh, self.dv), (0, self.vrow - self.dv)).view(-1, self.nh * self.vrow)
+            ops.sigmoid_gate(out, gate)
         return project(out, self.wo)
 
 
@@ -497,7 +515,7 @@ class LatentAttention(Part):
         return PagedKVNeed(1, self.row, self.window, values_in_keys=True)
 
     def decode_launch_key(self, num_seqs: int, max_kv_len: int, page_size: int):
-        return attn_kernels.decode_splits(num_seqs, self.nh, 1, self.row, page_size, max_kv_len)
+        return attn_kernels.decode_splits(num_seqs, self.nh, 1, self.row, page_size, max_kv_len, one_pool=True)
 
     def forward(self, x: torch.Tensor, batch, cache) -> torch.Tensor:
         n = x.shape[0]

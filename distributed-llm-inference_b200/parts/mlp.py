@@ -7,7 +7,7 @@ import torch
 from ..kernels import ops
 from ..kernels.gemm import dense_product, fused_epilogue, last_product, project
 from ..weights.loader import TensorDecl
-from .base import Part, register_part, tensor_name
+from .base import Part, build_part, register_part, tensor_name
 
 
 @register_part("feed_forward", "glu")
@@ -102,26 +102,33 @@ class DenseActMLP(Part):
         return project(ops.activation(project(x, self.w_up), self.activation), self.w_down)
 
 
+@register_part("feed_forward", "routed_mlp")
 @register_part("feed_forward", "routed_glu")
-class RoutedGLU(Part):
-    """A mixture of ``num_experts`` small gated feed-forwards down_e(act(gate_e(x)) * up_e(x)), of which each token uses ``top``.
+class RoutedMLP(Part):
+    """A mixture of ``num_experts`` small feed-forwards, of which each token uses ``top``: gated ones, down_e(act(gate_e(x)) * up_e(x)), or
+    (``gated`` false) plain ones, down_e(act(up_e(x))).  The router has ``identity`` outputs more than there are experts; these last
+    ones are experts without tensors whose output is the input itself.
 
     The router's logits z = W_r x and everything that follows them are float32.  ``score``:
 
     * ``"sigmoid"``: scores are sigmoid(z).  The experts are CHOSEN by score + correction (a learned number per expert that steers
       the choice and nothing else); they are WEIGHTED by their scores without it, divided by their sum (+ 1e-20) and multiplied
       by ``route_scale``;
+    * ``"softmax"``: scores are softmax(z) over all router outputs; chosen by score + correction, weighted by the scores without
+      it as they are (their sum is below one), times ``route_scale``;
     * ``"softmax_chosen"``: the tensor ``correction`` is a bias of the logits, z = W_r x + b.  The experts with the largest logits
       are chosen, their weights are the softmax over the chosen experts' logits alone, times ``route_scale``.
 
     With ``group_count`` > 1 the experts form that many equal groups of neighbours; a group's mark is the sum of its two
     largest choice scores (or logits), and only experts of the ``group_keep`` best groups can be chosen.  The output is the weighted
-    sum of the chosen experts' outputs, added up in float32 in the order of the choice.
+    sum of the chosen experts' outputs, added up in float32 in the order of the choice, and, if there is one, of the ``shared``
+    feed-forward (a PartSpec; its weight is one), which runs for every token.
 
     One kernel routes; the tokens of every expert are then gathered by a counting sort on the device (no shape depends on
-    the data, so a step with this part can be recorded in a CUDA graph), and two grouped products run over the sorted rows.
-    params: hidden_size, intermediate_size, num_experts, top, route_scale, group_count, group_keep, activation, score, tensors
-    (names of router, correction and, with ``{}`` for the expert's number, gate, up, down)."""
+    the data, so a step with this part can be recorded in a CUDA graph), and two grouped products run over the sorted rows; the
+    kernel that adds the outputs up reads the identities' input and the shared feed-forward's output in place.
+    params: hidden_size, intermediate_size, num_experts, identity, top, route_scale, group_count, group_keep, activation, gated, score,
+    shared, tensors (names of router, correction and, with ``{}`` for the expert's number, gate, up, down)."""
 
     graph_capturable = True
     takes_scaled_rows = False
@@ -131,27 +138,35 @@ class RoutedGLU(Part):
         p = spec.params
         self.hidden, self.inter = int(p["hidden_size"]), int(p["intermediate_size"])
         self.experts, self.top = int(p["num_experts"]), int(p["top"])
+        self.outputs = self.experts + int(p.get("identity") or 0)  # of the router
         self.route_scale = float(p.get("route_scale", 1.0))
         self.group_count, self.group_keep = int(p.get("group_count") or 1), int(p.get("group_keep") or 1)
+        self.gated = bool(p.get("gated", True))
         self.activation = p.get("activation", "silu")
         self.score = p.get("score", "sigmoid")
         if self.score not in ops.MOE_SCORES:
-            raise ValueError(f"routed_glu: score={self.score!r} (known: {', '.join(ops.MOE_SCORES)})")
-        if self.activation not in ops.GLU_ACTIVATIONS:
-            raise ValueError(f"activation {self.activation!r} is not supported (known: {sorted(ops.GLU_ACTIVATIONS)})")
-        per = self.experts // self.group_count
-        if self.experts % self.group_count or self.group_keep > self.group_count or self.top > self.group_keep * per or self.top > ops.MOE_MAX_TOP:
-            raise ValueError("routed_glu: experts must divide into the groups, and the kept groups must hold at least ``top`` experts")
+            raise ValueError(f"routed_mlp: score={self.score!r} (known: {', '.join(ops.MOE_SCORES)})")
+        known = ops.GLU_ACTIVATIONS if self.gated else ops.ACTIVATIONS
+        if self.activation not in known:
+            raise ValueError(f"activation {self.activation!r} is not supported (known: {sorted(known)})")
+        per = self.outputs // self.group_count
+        if self.outputs % self.group_count or self.group_keep > self.group_count or self.top > self.group_keep * per or self.top > ops.MOE_MAX_TOP:
+            raise ValueError("routed_mlp: experts must divide into the groups, and the kept groups must hold at least ``top`` experts")
+        self.shared = build_part("feed_forward", p["shared"], env) if p.get("shared") is not None else None
         defaults = {"router": "router.weight", "correction": "router.correction", "gate": "experts.{}.gate_proj.weight",
                     "up": "experts.{}.up_proj.weight", "down": "experts.{}.down_proj.weight"}
         self.names = {role: tensor_name(spec, role, default) for role, default in defaults.items()}
-        self.w_router = self.correction = self.w_gate_up = self.w_down = None
+        self.w_router = self.correction = self.w_up = self.w_down = None
+
+    def children(self):
+        return [self.shared] if self.shared is not None else []
 
     def declare(self):
         nm = self.names
-        out = {nm["router"]: TensorDecl((self.experts, self.hidden), "vector32"), nm["correction"]: TensorDecl((self.experts,), "vector32")}
+        out = {nm["router"]: TensorDecl((self.outputs, self.hidden), "vector32"), nm["correction"]: TensorDecl((self.outputs,), "vector32")}
         for e in range(self.experts):
-            out[nm["gate"].format(e)] = TensorDecl((self.inter, self.hidden))
+            if self.gated:
+                out[nm["gate"].format(e)] = TensorDecl((self.inter, self.hidden))
             out[nm["up"].format(e)] = TensorDecl((self.inter, self.hidden))
             out[nm["down"].format(e)] = TensorDecl((self.hidden, self.inter))
         return out
@@ -159,8 +174,9 @@ class RoutedGLU(Part):
     def load(self, tensors):
         nm = self.names
         self.w_router, self.correction = tensors[nm["router"]], tensors[nm["correction"]]
-        # [experts, 2 ff, H]: an expert's gate rows, then its up rows; [experts, H, ff]
-        self.w_gate_up = torch.stack([torch.cat([tensors[nm["gate"].format(e)], tensors[nm["up"].format(e)]], 0) for e in range(self.experts)], 0).contiguous()
+        # [experts, (2) ff, H]: an expert's gate rows, if it has any, then its up rows; [experts, H, ff]
+        roles = ("gate", "up") if self.gated else ("up",)
+        self.w_up = torch.stack([torch.cat([tensors[nm[r].format(e)] for r in roles], 0) for e in range(self.experts)], 0).contiguous()
         self.w_down = torch.stack([tensors[nm["down"].format(e)] for e in range(self.experts)], 0).contiguous()
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
@@ -169,5 +185,6 @@ class RoutedGLU(Part):
         weights = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
         ops.moe_route(ids, weights, x, self.w_router, self.correction, self.group_count, self.group_keep, self.route_scale, self.score)
         out = torch.empty((n, self.hidden), dtype=x.dtype, device=x.device)
-        ops.moe_experts(out, x, ids, weights, self.w_gate_up, self.w_down, self.activation)
+        shared = self.shared.forward(x) if self.shared is not None else None
+        ops.moe_experts(out, x, ids, weights, self.w_up, self.w_down, self.activation, gated=self.gated, shared=shared)
         return out

@@ -16,15 +16,16 @@ def inverse_frequencies(params) -> torch.Tensor:
     (src/dli/model/rope.py:21-47): exponents 2j/d, 1 / theta**e; ``linear`` divides every
     frequency by ``factor`` (positions are interpolated); for ``llama3`` wavelengths
     beyond original_max / low_freq_factor are divided by ``factor``, those under
-    original_max / high_freq_factor kept, and the band between interpolated."""
+    original_max / high_freq_factor kept, and the band between interpolated.  With ``exact`` every
+    step is taken in float64 and the result rounded once."""
     d = int(params["rotary_dim"])
-    exponents = torch.arange(0, d, 2, dtype=torch.int64).to(torch.float32) / d
+    exponents = torch.arange(0, d, 2, dtype=torch.int64).to(torch.float64 if params.get("exact") else torch.float32) / d
     inv = 1.0 / (float(params["theta"]) ** exponents)
     scaling = params.get("scaling", "default")
     if scaling == "default":
-        return inv
+        return inv.to(torch.float32)
     if scaling == "linear":
-        return inv / float(params["factor"])
+        return (inv / float(params["factor"])).to(torch.float32)
     if scaling != "llama3":
         raise ValueError(f"rotary scaling {scaling!r} is not supported (default, linear, llama3)")
     old = params["original_max_position_embeddings"]
@@ -34,7 +35,7 @@ def inverse_frequencies(params) -> torch.Tensor:
     smooth = (old / wavelen - low) / (high - low)
     smoothed = (1 - smooth) * scaled / factor + smooth * scaled
     medium = ~(wavelen < old / high) & ~(wavelen > old / low)
-    return torch.where(medium, smoothed, scaled)
+    return torch.where(medium, smoothed, scaled).to(torch.float32)
 
 
 def _step_table(batch, inv_freq, table_key):
@@ -74,17 +75,17 @@ def _project_and_encode(x, wqkv, batch, cache, num_heads, num_kv_heads, write_kv
     return _rotate_and_store(project(x, wqkv), batch, cache, num_heads, num_kv_heads, write_kv, head_dim, rotary_dim, inv_freq, table_key)
 
 
-def _norm_rotate_and_store(proj, wq, wk, eps, batch, cache, num_heads, num_kv_heads, write_kv, values_from_keys, head_dim, rotary_dim, inv_freq):
+def _norm_rotate_and_store(proj, wq, wk, eps, batch, cache, num_heads, num_kv_heads, write_kv, values_from_keys, head_dim, rotary_dim, inv_freq, **form):
     group = batch.group(cache.group)
     return ops.qk_norm_rotary_store(proj, wq, wk, eps, batch.positions, inv_freq, group.slots if write_kv else None,
                                     cache.k if write_kv else None, cache.v if write_kv else None, num_heads, num_kv_heads, head_dim,
-                                    rotary_dim, cache.page_size, write_kv, values_from_keys)
+                                    rotary_dim, cache.page_size, write_kv, values_from_keys, **form)
 
 
 @register_part("position", "rotary")
 class Rotary(Part):
     """params: head_dim, rotary_dim (<= head_dim; elements beyond it pass through), theta,
-    scaling and its constants.  The angle float32(position) * inv_freq and its sine and cosine
+    scaling and its constants, exact (see ``inverse_frequencies``).  The angle float32(position) * inv_freq and its sine and cosine
     are computed in float32 inside the kernel that also writes k and v to the cache."""
 
     graph_capturable = True
@@ -107,11 +108,11 @@ class Rotary(Part):
         return _project_and_encode(x, wqkv, batch, cache, num_heads, num_kv_heads, write_kv, self.head_dim, self.rotary_dim, self.inv_freq, self.table_key)
 
     def norm_rotate_and_store(self, proj, wq, wk, eps: float, batch, cache, num_heads: int, num_kv_heads: int, write_kv: bool,
-                              values_from_keys: bool):
-        """For a mixer that norms q and k over their whole projection before the encoding: norm (if ``wq``), rotation
-        and cache write in one kernel; returns the encoded queries [n, num_heads * head_dim]."""
+                              values_from_keys: bool, **form):
+        """For a mixer that norms q and k before the encoding: norm (if ``wq``), rotation and cache write in one kernel; returns the
+        encoded queries [n, num_heads * row].  ``form``: value_dim, per_head, row of ``ops.qk_norm_rotary_store``."""
         return _norm_rotate_and_store(proj, wq, wk, eps, batch, cache, num_heads, num_kv_heads, write_kv, values_from_keys,
-                                      self.head_dim, self.rotary_dim, self.inv_freq)
+                                      self.head_dim, self.rotary_dim, self.inv_freq, **form)
 
 
 @register_part("position", "none")
@@ -131,6 +132,6 @@ class NoPosition(Part):
         return _project_and_encode(x, wqkv, batch, cache, num_heads, num_kv_heads, write_kv, self.head_dim, 0, None)
 
     def norm_rotate_and_store(self, proj, wq, wk, eps: float, batch, cache, num_heads: int, num_kv_heads: int, write_kv: bool,
-                              values_from_keys: bool):
+                              values_from_keys: bool, **form):
         return _norm_rotate_and_store(proj, wq, wk, eps, batch, cache, num_heads, num_kv_heads, write_kv, values_from_keys,
-                                      self.head_dim, 0, None)
+                                      self.head_dim, 0, None, **form)

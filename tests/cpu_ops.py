@@ -116,6 +116,7 @@ def paged_attention_simt(out, qkv, k_pool, v_pool, block_tables, seq_of_token, p
     n = out.shape[0]
     _, nkv, page_size, d = k_pool.shape
     fan = num_heads // nkv
+    assert out.shape[1] == num_heads * v_pool.shape[3]
     q = qkv[:, : num_heads * d].view(n, num_heads, d).float()
     for t in range(n):
         p = int(positions[t])
@@ -219,15 +220,19 @@ def activation(x, kind):
 
 
 def qk_norm_rotary_store(proj, wq, wk, eps, positions, inv_freq, slots, k_pool, v_pool, num_heads, num_kv_heads, head_dim, rotary_dim,
-                         page_size, write_kv=True, values_from_keys=True):
+                         page_size, write_kv=True, values_from_keys=True, value_dim=None, per_head=False, row=None):
     n = proj.shape[0]
-    nq, nk = num_heads * head_dim, num_kv_heads * head_dim
+    nq, nk, dv, row = num_heads * head_dim, num_kv_heads * head_dim if write_kv else 0, value_dim or head_dim, row or head_dim
     q, k = proj[:, :nq].float(), proj[:, nq : nq + nk].float()
-    v = proj[:, nq : nq + nk] if values_from_keys else proj[:, nq + nk : nq + 2 * nk]
+    v = proj[:, nq : nq + nk] if values_from_keys else proj[:, nq + nk : nq + nk + num_kv_heads * dv]
+
+    def normed(y, w):
+        z = y.reshape(n, -1, head_dim) if per_head else y
+        return (z * torch.rsqrt((z * z).mean(-1, keepdim=True) + eps) * w).reshape(y.shape)
+
     if wq is not None:
-        q = q * torch.rsqrt((q * q).mean(-1, keepdim=True) + eps) * wq
-        k = k * torch.rsqrt((k * k).mean(-1, keepdim=True) + eps) * wk
-    qk = torch.cat([q, k], -1).view(n, num_heads + num_kv_heads, head_dim).clone()
+        q, k = normed(q, wq), normed(k, wk) if write_kv else k
+    qk = torch.cat([q, k], -1).view(n, -1, head_dim).clone()
     if rotary_dim:
         half = rotary_dim // 2
         ang = positions.float()[:, None] * inv_freq[None, :]
@@ -237,9 +242,13 @@ def qk_norm_rotary_store(proj, wq, wk, eps, positions, inv_freq, slots, k_pool, 
         qk[..., half:rotary_dim] = hi * cos + lo * sin
     if write_kv:
         page, off = (slots // page_size).long(), (slots % page_size).long()
-        k_pool[page, :, off, :] = qk[:, num_heads:].to(k_pool.dtype)
-        v_pool[page, :, off, :] = v.reshape(n, num_kv_heads, head_dim).to(v_pool.dtype)
-    return qk[:, :num_heads].reshape(n, nq).to(proj.dtype)
+        k_pool[page, :, off, :] = _padded(qk[:, num_heads:], k_pool.shape[3]).to(k_pool.dtype)
+        v_pool[page, :, off, :] = _padded(v.reshape(n, num_kv_heads, dv), v_pool.shape[3]).to(v_pool.dtype)
+    return _padded(qk[:, :num_heads], row).reshape(n, num_heads * row).to(proj.dtype)
+
+
+def _padded(x, row):
+    return torch.nn.functional.pad(x, (0, row - x.shape[-1]))
 
 
 def qk_norm_mix_store(q_out, qkv, bias, wq, wk, eps, positions, temp, source, lam, slots, k_pool, v_pool, num_heads, num_kv_heads, head_dim, value_dim,
@@ -770,6 +779,8 @@ def moe_route(ids, weights, x, router, correction, group_count, group_keep, scal
     s = x.float() @ router.t()
     if score == "sigmoid":
         s = torch.sigmoid(s)
+    elif score == "softmax":
+        s = torch.softmax(s, -1)
     choice = s + correction
     logits = choice
     if group_count > 1:
@@ -785,6 +796,9 @@ def moe_route(ids, weights, x, router, correction, group_count, group_keep, scal
     if score == "softmax_chosen":
         weights.copy_(torch.softmax(logits.gather(1, picked), -1) * scale)
         return
+    if score == "softmax":
+        weights.copy_(w * scale)
+        return
     weights.copy_(w / (w.sum(-1, keepdim=True) + 1e-20) * scale)
 
 
@@ -796,16 +810,27 @@ def _glu_act(g, activation):
     return _silu(g)
 
 
-def moe_experts(out, x, ids, weights, w_gate_up, w_down, activation="silu", stages=0):
+_plain_act = activation  # the stand-in of that name, which a parameter hides below
+
+
+def moe_experts(out, x, ids, weights, w_up, w_down, activation="silu", stages=0, gated=True, shared=None):
     n, top = ids.shape
-    ff = w_gate_up.shape[1] // 2
+    E, _, ff = w_down.shape
     acc = torch.zeros((n, x.shape[1]))
     for k in range(top):
         for e in ids[:, k].unique().tolist():
             rows = (ids[:, k] == e).nonzero().flatten()
-            gu = _sums(x[rows], w_gate_up[e]).to(x.dtype).float()
-            hidden = (_glu_act(gu[:, :ff], activation) * gu[:, ff:]).to(x.dtype)
+            if e >= E:  # the identity
+                acc[rows] += weights[rows, k, None] * x[rows].float()
+                continue
+            inner = _sums(x[rows], w_up[e]).to(x.dtype).float()
+            if gated:
+                hidden = (_glu_act(inner[:, :ff], activation) * inner[:, ff:]).to(x.dtype)
+            else:
+                hidden = _plain_act(inner, activation).to(x.dtype)
             acc[rows] += weights[rows, k, None] * _sums(hidden, w_down[e])
+    if shared is not None:
+        acc += shared.float()
     out.copy_(acc.to(out.dtype))
 
 

@@ -256,6 +256,6 @@ def test_plain_libraries_refuse_bent_scores():
     from ctypes import c_float, c_int, c_longlong, c_void_p
 
     f = ops._fn("attention_tc.cu", "dli_paged_decode_tma", [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p]
-                + [c_int] * 8 + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p])
+                + [c_int] * 9 + [c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p])
     none = c_void_p(0)
-    assert f(none, none, 0, none, none, 0, none, 0, none, none, 0, 1, 0, 1, 1, 64, 16, 0, 1.0, 0.0, none, 5.0, none, 1, none, none, 0, none) == 1001
+    assert f(none, none, 0, none, none, 0, none, 0, none, none, 0, 1, 0, 1, 1, 64, 64, 16, 0, 1.0, 0.0, none, 5.0, none, 1, none, none, 0, none) == 1001

@@ -12,7 +12,7 @@ from dli_b200.config import gedunex as config_mod
 from dli_b200.config import registry as registry_mod
 from dli_b200.parts import block as block_mod
 from dli_b200.parts.attention import CappedAttention
-from dli_b200.parts.mlp import RoutedGLU
+from dli_b200.parts.mlp import RoutedMLP
 from dli_b200.parts.model import SinusoidEmbedding
 from dli_b200.parts.ssm import MatrixMemory
 from tests import cpu_ops, gedunex_suite as suite
@@ -53,7 +53,7 @@ MUTANTS = {
     "the divisor has no floor": (cpu_ops, "matrix_memory_scan", "torch.maximum(out[:, dv].abs(), torch.exp(-m)) + 1e-6", "out[:, dv].abs() + 1e-6"),
     "the router's weights are taken over all experts": (cpu_ops, "moe_route", "torch.softmax(logits.gather(1, picked), -1) * scale",
                                                         "torch.softmax(logits, -1).gather(1, picked) * scale"),
-    "the router scores by the logistic function": (RoutedGLU, "forward", "self.route_scale, self.score)", 'self.route_scale, "sigmoid")'),
+    "the router scores by the logistic function": (RoutedMLP, "forward", "self.route_scale, self.score)", 'self.route_scale, "sigmoid")'),
     "the embedding's scale is left out": (SinusoidEmbedding, "forward_step", "self.weight, self.scale,", "self.weight, 1.0,"),
     "sines and cosines change places": (cpu_ops, "sinusoid_embedding", "torch.stack([ang.sin(), ang.cos()], -1)", "torch.stack([ang.cos(), ang.sin()], -1)"),
     "the window is read one token too wide": (config_mod, "_parse_attention", 'window = _positive(m["mask"]["size"], where + ".mask.size")',

@@ -13,7 +13,7 @@ from dli_b200.parts import base as base_mod
 from dli_b200.parts import block as block_mod
 from dli_b200.parts import entry as entry_mod
 from dli_b200.parts.attention import ConvAttention, LatentAttention
-from dli_b200.parts.mlp import RoutedGLU
+from dli_b200.parts.mlp import RoutedMLP
 from dli_b200.parts.pair import WeightedPairMixer
 from dli_b200.parts.ssm import ChannelDeltaRule, ShiftDecayRecurrence
 from tests import cpu_ops, lokolorn_suite as suite
@@ -52,7 +52,7 @@ MUTANTS = {
     "neighbouring pairs are read as distant ones": (LatentAttention, "load", 'if self.pairing == "neighbours" and self.rotary_dim:', "if False:"),
     "the correction enters the weights": (cpu_ops, "moe_route", "w = s.gather(1, picked)", "w = choice.gather(1, picked)"),
     "a group is marked by its best expert alone": (cpu_ops, "moe_route", "topk(min(2, per), -1)", "topk(1, -1)"),
-    "the router's scale is left out": (RoutedGLU, "forward", "self.group_keep, self.route_scale, self.score)", "self.group_keep, 1.0, self.score)"),
+    "the router's scale is left out": (RoutedMLP, "forward", "self.group_keep, self.route_scale, self.score)", "self.group_keep, 1.0, self.score)"),
     "the loop entry forgets the embedding": (entry_mod.ConcatProject, "apply", "ops.concat_stream_rows(both, h, self.table, batch.token_ids)",
                                              "ops.concat_stream_rows(both, h, self.table, batch.token_ids * 0)"),
     "the window is read one token too wide": (config_mod, "_parse_latent", 'window = _positive(m["mask"]["size"], where + ".mask.size")',
