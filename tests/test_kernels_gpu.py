@@ -386,7 +386,7 @@ def test_prefill_tc_when_row_maxima_keep_rising(ramp):
 def test_prefill_tc_refuses_other_sizes():
     t = attention_case(2, 1, 32, 16, [(0, 4)], torch.bfloat16)
     out = torch.empty((4, 64), dtype=torch.bfloat16, device=DEV)
-    with pytest.raises(ops.KernelError, match="head_dim"):
+    with pytest.raises(ops.KernelError, match="multiples of 8"):
         ops.paged_prefill_tc(out, t["qkv"], t["kp"], t["vp"], t["tables"], t["q_start"], t["kv_len"], 0, 1, 4, 2, 1.0)
     assert not ops.prefill_tc_supported(64, 4) and not ops.prefill_tc_supported(64, 48)
 
