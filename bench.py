@@ -1125,6 +1125,141 @@ def gedunex_kernels(size, pk, tokens=4096, seqs=64):
     return out
 
 
+def novunex_sizes(width, heads, kv_heads, dim, vdim, dim_2, vdim_2, ff, experts, identity, top, vocab=32000):
+    """A Novunex model of eight layers (scaled rotation with a norm over the projections, twice the other kind, then one that reads the
+    first one's keys and values; twice over) whose routed feed-forward chooses ``top`` of ``experts`` + ``identity`` outputs, an
+    expert having ff / top numbers, and the Gedunex configuration of the same width and heads (rows of max(dim, vdim) numbers),
+    experts and number of layers, attention in every one."""
+    def mlp():
+        return {"kind": "moe", "expert": {"ff": ff // top}, "router": {"experts": experts, "identity": identity, "top": top}, "shared": {"ff": ff // top}}
+
+    def second(kv_from=None):
+        m = {"heads": heads, "kv_heads": kv_heads, "dim": dim_2, "vdim": vdim_2, "scale": dim_2**-0.5,
+             "rot": {"base": 500000.0, "dims": dim_2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+        return {"type": "attention_2", "mlp": mlp(), "mixer": m if kv_from is None else {**m, "kv_from": kv_from}}
+
+    one = {"type": "attention", "mlp": mlp(), "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim**-0.5,
+                                                        "rot": {"base": 10000.0, "dims": dim // 2}}}
+    nv = {"architecture": "Novunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": [second(), one, one, second(0), second(), one, one, second(4)]}
+    row = max(dim, vdim, dim_2, vdim_2)
+    att = {"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": ff // top}, "router": {"experts": experts + identity, "top": top}},
+           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": row, "vdim": row, "scale": row**-0.5, "softcap": 30.0, "q_temp": {"coef": 0.1, "every": 4096},
+                     "v_mix": True}}
+    gd = {"architecture": "Gedunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "layers": [att] * 8}
+    return nv, gd
+
+
+NOVUNEX_SIZES = {
+    name: dict(width=s["width"], heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"] * 3 // 4, vdim=s["dim"] // 2, dim_2=s["dim"] // 2, vdim_2=s["dim"] * 3 // 4,
+               ff=s["ff"], experts=s["experts"] - 4, identity=4, top=s["top"])
+    for name, s in LOKOLORN_SIZES.items()
+}
+
+
+def novunex_kernels(size, pk, tokens=4096, seqs=64):
+    """Every kernel of the Novunex parts beside its like, at one size: a prompt portion of ``tokens`` tokens and a decode step of ``seqs``
+    sequences.  us, the bytes (or operations) the kernel has to move, and the share of the measured HBM peak (of the measured bf16 rate
+    for attention and the experts' products)."""
+    import torch
+
+    from dli_b200.kernels import attention as attn
+    from dli_b200.kernels import ops
+
+    dev, bf = "cuda", torch.bfloat16
+    W, nh, nkv = size["width"], size["heads"], size["kv_heads"]
+    E, identity, top = size["experts"], size["identity"], size["top"]
+    eff = size["ff"] // top
+    rows = max(size["dim"], size["vdim"], size["dim_2"], size["vdim_2"])
+    out = {}
+
+    def record(name, us, nbytes, like=None, flops=None):
+        rec = {"us": round(us, 1), "gb_s": round(nbytes / us / 1e3, 1), "hbm_frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)}
+        if flops is not None:
+            rec["tflops_bf16"] = round(flops / us / 1e6, 1)
+            rec["bf16_frac"] = round(flops / us / 1e6 / pk["bf16_tflops"], 3)
+        if like:
+            rec["like"] = like
+        out[name] = rec
+
+    for label, n, S in (("portion", tokens, 1), ("decode", seqs, seqs)):
+        q_len, context = n // S, (n if S == 1 else 2048)
+        q_start = torch.arange(S + 1, dtype=torch.int32, device=dev) * q_len
+        seq_of = torch.repeat_interleave(torch.arange(S, dtype=torch.int32), q_len).to(dev)
+        positions = (torch.arange(n, dtype=torch.int32) % q_len + (0 if S == 1 else context - 1)).to(dev)
+        pages = -(-context // 16) * S + 1
+        tables = (torch.randperm(pages - 1, device=dev)[: -(-context // 16) * S].view(S, -1)).to(torch.int32)
+        slots = torch.arange(n, dtype=torch.int32, device=dev)
+
+        class Group:
+            block_tables = tables
+
+        class Batch:
+            num_single, num_seqs, max_q_len, max_kv_len = (S if q_len == 1 else 0), S, q_len, context
+            max_kv_len_single = context if q_len == 1 else 0
+
+            def group(self, i):
+                return Group
+
+        Batch.q_start, Batch.kv_len, Batch.seq_of_token, Batch.positions = q_start, torch.full((S,), context, dtype=torch.int32, device=dev), seq_of, positions
+        pairs = sum(p + 1 for p in range(n)) if S == 1 else S * context
+
+        def pools(d, dv):
+            class Cache:
+                k, v = torch.randn(pages, nkv, 16, d, device=dev).to(bf), torch.randn(pages, nkv, 16, dv, device=dev).to(bf)
+                page_size, group = 16, 0
+
+            return Cache
+
+        def attention(name, d, dv, like=None, **more):
+            cache, q, o = pools(d, dv), torch.randn(n, nh * d, device=dev).to(bf), torch.empty(n, nh * dv, dtype=bf, device=dev)
+            us = time_kernel(lambda: attn.paged_attention(o, q, cache, Batch(), nh, d**-0.5, None, sink=0.0, **more))
+            moved = (n if S == 1 else S * context) * nkv * (d + dv) * 2 + n * nh * (d + dv) * 2
+            record(f"{label}.{name}", us, moved, like, flops=2.0 * pairs * nh * (d + dv))
+
+        slopes = torch.tensor([2.0 ** (-8.0 * (i + 1) / nh) for i in range(nh)], device=dev)
+        attention("attention_like", rows, rows, softcap=30.0, slopes=slopes)  # as the other model runs it
+        attention("attention_equal_rows", rows, rows)
+        attention("attention_equal_rows_128", 128, 128)
+        for kind, (d, dv) in (("attention", (size["dim"], size["vdim"])), ("attention_2", (size["dim_2"], size["vdim_2"]))):
+            attention(kind, d, dv, "attention_like")
+            cache, C = pools(d, dv), (nh + nkv) * d + nkv * dv
+            proj = torch.randn(n, C, device=dev).to(bf)
+            per_head = kind == "attention"
+            rot = d // 2 if per_head else d
+            wq, wk = torch.ones((1 if per_head else nh) * d, device=dev), torch.ones((1 if per_head else nkv) * d, device=dev)
+            inv = (1.0 / (10000.0 ** (torch.arange(0, rot, 2).float() / rot))).to(dev)
+            us = time_kernel(lambda: ops.qk_norm_rotary_store(proj, wq, wk, 1e-6, positions, inv, slots, cache.k, cache.v, nh, nkv, d, rot, 16, True, False,
+                                                              value_dim=dv, per_head=per_head))
+            record(f"{label}.{kind}_prep", us, n * C * 4, "qk_norm_mix_store")
+        cache, C = pools(rows, rows), (nh + 2 * nkv) * rows
+        proj, src, q = torch.randn(n, C, device=dev).to(bf), torch.randn(n, nkv * rows, device=dev), torch.empty(n, nh * rows, dtype=bf, device=dev)
+        wq, wk = torch.ones(nh * rows, device=dev), torch.ones(nkv * rows, device=dev)
+        us = time_kernel(lambda: ops.qk_norm_mix_store(q, proj, None, wq, wk, 1e-6, positions, (0.1, 4096.0), src, 0.5, slots, cache.k, cache.v, nh, nkv, rows, rows, 16))
+        record(f"{label}.qk_norm_mix_store", us, n * (C * 4 + nkv * rows * 4))
+        # router
+        x = torch.randn(n, W, device=dev).to(bf)
+        router, rb = torch.randn(E + identity, W, device=dev) * 0.05, torch.randn(E + identity, device=dev) * 0.1
+        ids, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        for score, like in (("softmax_chosen", None), ("softmax", "route_softmax_chosen")):
+            record(f"{label}.route_{score}", time_kernel(lambda: ops.moe_route(ids, wts, x, router, rb, 1, 1, 1.0, score)), n * W * 2 + (E + identity) * W * 4, like)
+        # experts: without a gate, identities among the choices, a shared output added; with a gate, every choice an expert
+        o, sh = torch.empty(n, W, dtype=bf, device=dev), torch.randn(n, W, device=dev).to(bf)
+        down = torch.randn(E + identity, W, eff, device=dev).to(bf) * 0.02
+        for gated in (True, False):
+            count = E + identity if gated else E
+            up = torch.randn(count, (2 if gated else 1) * eff, W, device=dev).to(bf) * 0.02
+            real = int((ids < count).sum())
+            moved = real * 2 * W * 2 + min(real, count) * (3 if gated else 2) * eff * W * 2
+            us = time_kernel(lambda: ops.moe_experts(o, x, ids, wts, up, down[:count], "silu" if gated else "relu2", gated=gated, shared=None if gated else sh))
+            record(f"{label}.experts_{'gated' if gated else 'plain'}", us, moved, None if gated else "experts_gated", flops=(6.0 if gated else 4.0) * real * W * eff)
+        # behind a sublayer
+        h, w = torch.randn(n, W, device=dev), torch.ones(W, device=dev)
+        y, y2 = torch.empty(n, W, dtype=bf, device=dev), torch.empty(n, W, dtype=bf, device=dev)
+        record(f"{label}.output_norm_add", time_kernel(lambda: ops.group_norm_add(h, o, w, 1, 1e-6, 1.0, y)), n * W * 12, "add_norm")
+        record(f"{label}.add_norm", time_kernel(lambda: ops.add_rmsnorm_pair(y2, None, h, o, y, w, None, 1e-6, None)), n * W * 14)
+    return out
+
+
 SIMT_FP32_TFLOPS = 148 * 128 * 2 * 1.9e9 / 1e12  # CUDA-core multiply-adds of a B200 at 1.9 GHz: the scan's ceiling (no float32 tensor-core path)
 
 
@@ -1135,6 +1270,7 @@ DESIGNS = {
     "pokadra": (POKADRA_SIZES, pokadra_sizes, "pazenex", pokadra_kernels),
     "lokolorn": (LOKOLORN_SIZES, lokolorn_sizes, "sugonex", lokolorn_kernels),
     "gedunex": (GEDUNEX_SIZES, gedunex_sizes, "lokolorn", gedunex_kernels),
+    "novunex": (NOVUNEX_SIZES, novunex_sizes, "gedunex", novunex_kernels),
 }
 
 
@@ -1376,7 +1512,7 @@ def main() -> int:
     ap.add_argument("--phase", default="all", choices=["all", "decode", "prefill", "sample"],
                     help="profiling runs: only the device-timed decode steps, only the prefill step, or only the sampling kernel (prints a short line)")
     ap.add_argument("--no-graphs", action="store_true", help="profiling runs: launch the step's kernels one by one")
-    ap.add_argument("--design", default=None, choices=["pazenex", "sugonex", "pokadra", "lokolorn", "gedunex"],
+    ap.add_argument("--design", default=None, choices=["pazenex", "sugonex", "pokadra", "lokolorn", "gedunex", "novunex"],
                     help="another measurement: this architecture beside Llama at equal sizes, and its kernels beside their likes (prints its own line)")
     ap.add_argument("--size", default=None, choices=list(DESIGN_SIZES), help="--design: one size only (every design has these names)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN,

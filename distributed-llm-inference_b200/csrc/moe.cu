@@ -10,7 +10,8 @@ using namespace dli;
 
 namespace {
 
-constexpr int ROUTE_THREADS = 512;  // at most: sixteen warps, an expert's row each, for a step of few tokens (a handful of blocks); four warps a token for many
+constexpr int ROUTE_THREADS = 512;  // at most: sixteen warps, an expert's row each, for a step of few tokens (a handful of blocks); four warps for more
+constexpr int ROUTE_MANY_TOKENS = 256;  // from here on a block takes several tokens
 constexpr int MAX_TOP = 32;
 enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_CHOSEN = 1, ROUTE_SOFTMAX_ALL = 2 };
 
@@ -31,39 +32,15 @@ __device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* 
   return warp_sum(acc);
 }
 
-// One block per token.  z = W_r x (float32 sums of float32 products); s = sigmoid(z); choice = s + correction.
+// What a token chooses.  z = W_r x (float32 sums of float32 products); s = sigmoid(z); choice = s + correction.
 // Groups: `groups` equal runs of neighbouring experts; a group's mark is the sum of its two largest choice scores (its
 // one score if it has one expert); only the `keep` groups with the largest marks stay eligible.  The `top` eligible experts
 // with the largest choice scores are chosen (ties: the lower index), in that order; weights = s[chosen] / (sum + 1e-20) * scale.
 // mode ROUTE_SOFTMAX_CHOSEN: choice = z + correction instead, and weights = softmax over the chosen experts' choices * scale.
 // mode ROUTE_SOFTMAX_ALL: s = softmax(z) over all experts, choice = s + correction, and weights = s[chosen] * scale as they are.
-template <typename T>
-__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x,
-                                                                  const float* __restrict__ router, const float* __restrict__ correction,
-                                                                  int W, int E, int top, int groups, int keep, float scale, int mode) {
-  pdl_launch_dependents();
-  pdl_wait();
-  extern __shared__ float sm[];  // x [W] | score [E] | choice [E] | mark [groups]
-  float* xs = sm;
-  float* score = xs + W;
-  float* choice = score + E;
-  float* mark = choice + E;
-  __shared__ int picked[MAX_TOP];
-  const size_t t = blockIdx.x;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  for (int i = threadIdx.x; i < W; i += blockDim.x) xs[i] = to_float(x[t * W + i]);
-  __syncthreads();
-  const bool vec = (W % 8) == 0 && (((uintptr_t)router) & 15) == 0;
-  for (int e = warp; e < E; e += blockDim.x >> 5) {
-    const float z = warp_dot<float>(router + (size_t)e * W, xs, W, lane, vec);
-    if (lane == 0) {
-      const float s = mode == ROUTE_SIGMOID ? 1.f / (1.f + expf(-z)) : mode == ROUTE_SOFTMAX_CHOSEN ? z + correction[e] : z;
-      score[e] = s;
-      choice[e] = mode == ROUTE_SIGMOID ? s + correction[e] : s;
-    }
-  }
-  __syncthreads();
-  if (warp != 0) return;
+// Done by one warp, from the token's scores (ROUTE_SOFTMAX_ALL: its logits) and choice scores in shared memory.
+__device__ __forceinline__ void choose_experts(int* __restrict__ ids, float* __restrict__ weights, float* score, float* choice, float* mark, int* picked,
+                                               const float* __restrict__ correction, int E, int top, int groups, int keep, float scale, int mode, int lane) {
   if (mode == ROUTE_SOFTMAX_ALL) {  // the logits become their softmax
     float high = -CUDART_INF_F, sum = 0.f;
     for (int e = lane; e < E; e += 32) high = fmaxf(high, score[e]);
@@ -138,8 +115,96 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restric
   }
   const float f = mode == ROUTE_SOFTMAX_ALL ? scale : scale / (mode == ROUTE_SOFTMAX_CHOSEN ? total : total + 1e-20f);
   for (int k = lane; k < top; k += 32) {
-    ids[t * top + k] = picked[k];
-    weights[t * top + k] = (mode == ROUTE_SOFTMAX_CHOSEN ? expf(score[picked[k]] - largest) : score[picked[k]]) * f;
+    ids[k] = picked[k];
+    weights[k] = (mode == ROUTE_SOFTMAX_CHOSEN ? expf(score[picked[k]] - largest) : score[picked[k]]) * f;
+  }
+}
+
+__device__ __forceinline__ void put_score(float* score, float* choice, int e, float z, const float* __restrict__ correction, int mode) {
+  const float s = mode == ROUTE_SIGMOID ? 1.f / (1.f + expf(-z)) : mode == ROUTE_SOFTMAX_CHOSEN ? z + correction[e] : z;
+  score[e] = s;
+  choice[e] = mode == ROUTE_SIGMOID ? s + correction[e] : s;
+}
+
+// A step of few tokens: a block per token, a warp per expert's row in turn.
+template <typename T>
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x,
+                                                                  const float* __restrict__ router, const float* __restrict__ correction,
+                                                                  int W, int E, int top, int groups, int keep, float scale, int mode) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float sm[];  // x [W] | score [E] | choice [E] | mark [groups]
+  float* xs = sm;
+  float* score = xs + W;
+  float* choice = score + E;
+  float* mark = choice + E;
+  __shared__ int picked[MAX_TOP];
+  const size_t t = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) xs[i] = to_float(x[t * W + i]);
+  __syncthreads();
+  const bool vec = (W % 8) == 0 && (((uintptr_t)router) & 15) == 0;
+  for (int e = warp; e < E; e += blockDim.x >> 5) {
+    const float z = warp_dot<float>(router + (size_t)e * W, xs, W, lane, vec);
+    if (lane == 0) put_score(score, choice, e, z, correction, mode);
+  }
+  __syncthreads();
+  if (warp == 0) choose_experts(ids + t * top, weights + t * top, score, choice, mark, picked, correction, E, top, groups, keep, scale, mode, lane);
+}
+
+// A portion of many tokens: a block takes four of them and a warp four experts' rows at a time, so that a number of either, once read,
+// serves four products.  Every sum is added up in the order of the kernel above.  W a multiple of 8, 16-byte aligned rows.
+constexpr int ROUTE_TOKENS = 4, ROUTE_ROWS = 4;
+template <typename T>
+__global__ void __launch_bounds__(ROUTE_TOKENS * 32) moe_route_many_kernel(int* __restrict__ ids, float* __restrict__ weights, const T* __restrict__ x,
+                                                                           const float* __restrict__ router, const float* __restrict__ correction, int n,
+                                                                           int W, int E, int top, int groups, int keep, float scale, int mode) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float sm[];  // per token: score [E] | choice [E] | mark [groups]
+  __shared__ int picked[ROUTE_TOKENS][MAX_TOP];
+  const int per_token = 2 * E + groups;
+  const size_t t0 = (size_t)blockIdx.x * ROUTE_TOKENS;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const T* rows[ROUTE_TOKENS];
+#pragma unroll
+  for (int j = 0; j < ROUTE_TOKENS; ++j) rows[j] = x + (t0 + j < (size_t)n ? t0 + j : (size_t)n - 1) * W;
+  for (int e0 = warp * ROUTE_ROWS; e0 < E; e0 += ROUTE_TOKENS * ROUTE_ROWS) {
+    float acc[ROUTE_ROWS][ROUTE_TOKENS];
+#pragma unroll
+    for (int r = 0; r < ROUTE_ROWS; ++r)
+#pragma unroll
+      for (int j = 0; j < ROUTE_TOKENS; ++j) acc[r][j] = 0.f;
+    const float* w[ROUTE_ROWS];
+#pragma unroll
+    for (int r = 0; r < ROUTE_ROWS; ++r) w[r] = router + (size_t)min(e0 + r, E - 1) * W;
+    for (int i = lane * 8; i < W; i += 256) {
+      float xv[ROUTE_TOKENS][8];
+#pragma unroll
+      for (int j = 0; j < ROUTE_TOKENS; ++j) load8(rows[j] + i, xv[j]);
+#pragma unroll
+      for (int r = 0; r < ROUTE_ROWS; ++r) {
+        float wv[8];
+        load8(w[r] + i, wv);
+#pragma unroll
+        for (int j = 0; j < ROUTE_TOKENS; ++j)
+#pragma unroll
+          for (int k = 0; k < 8; ++k) acc[r][j] = fmaf(wv[k], xv[j][k], acc[r][j]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < ROUTE_ROWS; ++r)
+#pragma unroll
+      for (int j = 0; j < ROUTE_TOKENS; ++j) {
+        const float z = warp_sum(acc[r][j]);
+        if (lane == 0 && e0 + r < E) put_score(sm + j * per_token, sm + j * per_token + E, e0 + r, z, correction, mode);
+      }
+  }
+  __syncthreads();
+  const size_t t = t0 + warp;  // a warp chooses for one token
+  if (t < (size_t)n) {
+    float* score = sm + warp * per_token;
+    choose_experts(ids + t * top, weights + t * top, score, score + E, score + 2 * E, picked[warp], correction, E, top, groups, keep, scale, mode, lane);
   }
 }
 
@@ -224,8 +289,17 @@ DLI_EXPORT int dli_moe_route(int* ids, float* weights, const void* x, const floa
     return DLI_ERR_UNSUPPORTED;
   const size_t smem = ((size_t)W + 2 * E + groups) * sizeof(float);
   if (smem > 200 * 1024) return DLI_ERR_UNSUPPORTED;
-  const int threads = n <= 256 ? ROUTE_THREADS : 128;
+  const int threads = n <= ROUTE_MANY_TOKENS ? ROUTE_THREADS : 128;
   cudaError_t e;
+  const size_t many_smem = (size_t)ROUTE_TOKENS * (2 * E + groups) * sizeof(float);
+  if (n > ROUTE_MANY_TOKENS && (W % 8) == 0 && ((((uintptr_t)x) | ((uintptr_t)router)) & 15) == 0 && many_smem <= 48 * 1024 - ROUTE_TOKENS * MAX_TOP * sizeof(int)) {
+    const dim3 grid((n + ROUTE_TOKENS - 1) / ROUTE_TOKENS), block(ROUTE_TOKENS * 32);
+    if (dtype == DLI_F32)
+      return (int)launch_pdl((moe_route_many_kernel<float>), grid, block, many_smem, stream, 1, ids, weights, (const float*)x, router, correction, n, W, E, top,
+                             groups, keep, scale, mode);
+    return (int)launch_pdl((moe_route_many_kernel<__nv_bfloat16>), grid, block, many_smem, stream, 1, ids, weights, (const __nv_bfloat16*)x, router, correction,
+                           n, W, E, top, groups, keep, scale, mode);
+  }
   if (dtype == DLI_F32) {
     static MaxPerDevice set;
     if ((e = allow_smem(moe_route_kernel<float>, smem, set)) != cudaSuccess) return (int)e;

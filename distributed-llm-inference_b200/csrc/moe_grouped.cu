@@ -4,8 +4,7 @@
 //   hidden[row] = act(gate_e x) * (up_e x), or act(up_e x) for experts without a gate
 //                                                 (the sums rounded to bfloat16 first, as a stored product would be)
 //   partial[row] = down_e hidden[row]             (float32)
-//   out[t] = sum_k weights[t][k] * partial[row of pair (t, k)] (+ shared[t]), in the order of k, float32, one rounding.
-// Experts numbered E and above are identities: their pairs have no row, and x[t] takes the place of partial in the sum.
+// Experts numbered E and above are identities: their pairs have no row.  (moe_combine.cu adds the rows up, token by token.)
 #include <math_constants.h>
 
 #include "common.cuh"
@@ -265,32 +264,6 @@ __global__ void __launch_bounds__(THREADS) moe_grouped_gemm_kernel(const bf16* _
       }
 }
 
-// eight columns a thread (W is a multiple of 8)
-__global__ void moe_combine_kernel(bf16* __restrict__ out, const float* __restrict__ partial, const int* __restrict__ pos, const int* __restrict__ ids,
-                                   const float* __restrict__ weights, const bf16* __restrict__ x, const bf16* __restrict__ shared, int W, int E, int top) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const size_t t = blockIdx.x;
-  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
-    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    for (int k = 0; k < top; ++k) {
-      const float w = weights[t * top + k];
-      float v[8];
-      if (ids[t * top + k] < E) load8(partial + (size_t)pos[t * top + k] * W + c, v);
-      else load8(x + t * W + c, v);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) acc[i] = fmaf(w, v[i], acc[i]);
-    }
-    if (shared) {
-      float v[8];
-      load8(shared + t * W + c, v);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) acc[i] += v[i];
-    }
-    store8(out + t * W + c, acc);
-  }
-}
-
 template <int EPI, int NB, int STAGES>
 cudaError_t launch_grouped(const bf16* A, long long a_stride, const int* row_pair, int top, const bf16* B, long long b_expert_stride, int half, void* C,
                            int N, int K, const int* tile_expert, int tiles, int act, cudaStream_t stream) {
@@ -314,11 +287,11 @@ DLI_EXPORT int dli_moe_grouped_tile_rows() { return BM; }
 
 // ints: scratch of E + 1 (counts) + E + 1 (offsets) + 2 pairs (rank, pos) + tiles (tile_expert) + tiles * BM (row_pair) ints;
 // hidden: [tiles * BM][ff] bfloat16; partial: [tiles * BM][W] float32.  stages: 2 or 3 deep copies, or 0: chosen here.
-// gated: w_up holds an expert's gate rows, then its up rows; else its up rows alone.  ids from E on are identities; shared [n][W] or null.
-DLI_EXPORT int dli_moe_grouped(void* out, const void* x, const int* ids, const float* weights, const void* w_up, const void* w_down, const void* shared,
-                               int* ints, void* hidden, float* partial, int n, int W, int ff, int E, int top, int act, int gated, int stages, cudaStream_t stream) {
+// gated: w_up holds an expert's gate rows, then its up rows; else its up rows alone.  ids from E on are identities.  The rows of
+// the pairs are left behind the first 2 (E + 1) + pairs numbers of ints (those of identities undefined).
+DLI_EXPORT int dli_moe_grouped(const void* x, const int* ids, const void* w_up, const void* w_down, int* ints, void* hidden, float* partial, int n, int W, int ff, int E, int top, int act, int gated, int stages, cudaStream_t stream) {
   if (n == 0) return 0;
-  if (W < 8 || ff < 8 || (W % 8) || (ff % 8) || E < 1 || top < 1 || ((((uintptr_t)x) | ((uintptr_t)w_up) | ((uintptr_t)w_down) | ((uintptr_t)hidden) | ((uintptr_t)out) | ((uintptr_t)shared) | ((uintptr_t)partial)) & 15))
+  if (W < 8 || ff < 8 || (W % 8) || (ff % 8) || E < 1 || top < 1 || ((((uintptr_t)x) | ((uintptr_t)w_up) | ((uintptr_t)w_down) | ((uintptr_t)hidden) | ((uintptr_t)partial)) & 15))
     return DLI_ERR_UNSUPPORTED;
   const int pairs = n * top;
   const int tiles = dli_moe_grouped_tiles(pairs, E);
@@ -359,7 +332,5 @@ DLI_EXPORT int dli_moe_grouped(void* out, const void* x, const int* ids, const f
   if (e != cudaSuccess) return (int)e;
 #undef DLI_UP
 #undef DLI_DOWN
-  e = launch_pdl((moe_combine_kernel), dim3(n), dim3(W >= 2048 ? 256 : W >= 1024 ? 128 : 64), 0, stream, 1, (bf16*)out, (const float*)partial, (const int*)pos, ids, weights, bx,
-                 (const bf16*)shared, W, E, top);
-  return (int)e;
+  return 0;
 }

@@ -1744,13 +1744,13 @@ def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, 
 
 MOE_MAX_TOP = 32
 MOE_GROUPED_TILE_ROWS = 64  # BM of csrc/moe_grouped.cu
-MOE_GROUPED_MIN_TOKENS = 4  # fewer tokens rarely share an expert: every chosen expert is read once per pair, on the CUDA cores
+MOE_FEW_MAX_TOKENS = 64  # up to here a step's experts are found without sorting the pairs (csrc/moe_few.cu)
+MOE_NORM_ADD_MAX_SIZE = 12288
 
 
-def moe_grouped_supported(tokens: int, W: int, ff: int, dtype: torch.dtype) -> bool:
-    """Whether the experts' products of a step go to the grouped tensor-core kernels: bfloat16, more tokens than a decode step
-    brings, rows of whole 16-byte chunks."""
-    return dtype == torch.bfloat16 and tokens >= MOE_GROUPED_MIN_TOKENS and W % 8 == 0 and ff % 8 == 0
+def moe_products_supported(W: int, ff: int, dtype: torch.dtype) -> bool:
+    """Whether the experts' products of a step go to the tensor-core kernels: bfloat16, rows of whole 16-byte chunks."""
+    return dtype == torch.bfloat16 and W % 8 == 0 and ff % 8 == 0
 MOE_PAIR_CHUNK = 8192  # tokens a launch of the pair kernels takes (their grids count (token, expert) pairs along y)
 
 
@@ -1777,45 +1777,125 @@ def moe_route(ids: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router:
              _stream()), "moe_route")
 
 
+class MoeSums:
+    """The experts' outputs of a step as the products leave them: float32 rows, one per (token, choice) pair at ``pos`` (None: the pair's
+    own number), still to be weighted and added up (``moe_combine``, ``moe_combine_norm_add``).  ``shared`` [n, W]: what is added to
+    every token's sum (or None); ``shared_row``: the first of n float32 rows of ``partial`` that are (or None)."""
+
+    __slots__ = ("partial", "pos", "ids", "weights", "x", "experts", "shared", "shared_row")
+
+    def __init__(self, partial, pos, ids, weights, x, experts, shared, shared_row) -> None:
+        self.partial, self.pos, self.ids, self.weights, self.x = partial, pos, ids, weights, x
+        self.experts, self.shared, self.shared_row = experts, shared, shared_row
+
+    @property
+    def shared_rows(self) -> torch.Tensor | None:
+        return None if self.shared_row is None else self.partial[self.shared_row :]
+
+
+def _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared):
+    _need(x, "x"), _need(ids, "ids", torch.int32), _need(weights, "weights", torch.float32), _need(w_up, "w_up", x.dtype), _need(w_down, "w_down", x.dtype)
+    n, W = x.shape
+    top = ids.shape[1]
+    E, _, ff = w_down.shape
+    known = GLU_ACTIVATIONS if gated else ACTIVATIONS
+    if (x.dtype not in DT_CODE or tuple(w_up.shape) != (E, (2 if gated else 1) * ff, W) or w_down.shape[1] != W or tuple(ids.shape) != (n, top)
+            or tuple(weights.shape) != (n, top) or activation not in known):
+        raise KernelError("experts: shapes, dtype or activation do not agree")
+    if shared is not None:
+        _need(shared, "shared", x.dtype)
+        if tuple(shared.shape) != (n, W):
+            raise KernelError("experts: what is added to every token must be [n, W]")
+    return n, W, top, E, ff, known[activation]
+
+
+def moe_products(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, activation: str = "silu",
+                 gated: bool = True, shared: torch.Tensor | None = None, extra: tuple[torch.Tensor, torch.Tensor, str] | None = None,
+                 stages: int = 0, few: bool | None = None) -> MoeSums:
+    """The experts' products of ``moe_experts`` in bfloat16, not yet added up.  Up to MOE_FEW_MAX_TOKENS tokens every chosen expert's matrix
+    is streamed once and nothing is sorted (csrc/moe_few.cu); more tokens are sorted by expert and take two grouped products
+    (csrc/moe_grouped.cu; ``few`` False: so do few).  ``extra`` (up [f, W], down [W, f], activation): a feed-forward without a gate that runs
+    for every token and, with few tokens and beside experts without a gate, rides in the same launches."""
+    n, W, top, E, ff, act = _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared)
+    if not moe_products_supported(W, ff, x.dtype):
+        raise KernelError("moe_products: bfloat16 and sizes that are multiples of 8")
+    global launch_count
+    pairs = n * top
+    if n <= MOE_FEW_MAX_TOKENS if few is None else few:
+        extra_ff, extra_act, extra_up, extra_down = 0, 0, None, None
+        if extra is not None:
+            extra_up, extra_down, kind = extra
+            _need(extra_up, "extra[0]", x.dtype), _need(extra_down, "extra[1]", x.dtype)
+            extra_ff, extra_act = extra_up.shape[0], ACTIVATIONS[kind]
+            if gated or extra_up.shape[1] != W or tuple(extra_down.shape) != (W, extra_ff):
+                raise KernelError("moe_products: a feed-forward rides along beside experts without a gate, with matrices [f, W] and [W, f]")
+        hidden = torch.empty(pairs * ff + n * extra_ff, dtype=x.dtype, device=x.device)
+        partial = torch.empty((pairs + (n if extra is not None else 0), W), dtype=torch.float32, device=x.device)
+        f = _fn("moe_few.cu", "dli_moe_few", [c_void_p] * 8 + [c_int] * 9 + [c_void_p])
+        _check(f(_ptr(partial), _ptr(hidden), _ptr(x), _ptr(ids), _ptr(w_up), _ptr(w_down), _ptr(extra_up), _ptr(extra_down), n, W, ff, E, top, act, int(gated),
+                 extra_ff, extra_act, _stream()), "moe_products")
+        launch_count += 1  # two kernels
+        return MoeSums(partial, None, ids, weights, x, E, shared, pairs if extra is not None else None)
+    if extra is not None:
+        raise KernelError("moe_products: a feed-forward rides along with few tokens only")
+    tiles = min(pairs, E) + pairs // MOE_GROUPED_TILE_ROWS
+    rows = tiles * MOE_GROUPED_TILE_ROWS
+    ints = torch.empty(2 * (E + 1) + 2 * pairs + tiles + rows, dtype=torch.int32, device=x.device)
+    hidden = torch.empty((rows, ff), dtype=x.dtype, device=x.device)
+    partial = torch.empty((rows, W), dtype=torch.float32, device=x.device)
+    g = _fn("moe_grouped.cu", "dli_moe_grouped", [c_void_p] * 7 + [c_int] * 8 + [c_void_p])
+    _check(g(_ptr(x), _ptr(ids), _ptr(w_up), _ptr(w_down), _ptr(ints), _ptr(hidden), _ptr(partial), n, W, ff, E, top, act, int(gated), int(stages), _stream()),
+           "moe_products")
+    launch_count += 2 if pairs <= 2048 else 5  # three kernels a call (one block sorts up to 2,048 pairs), else six
+    return MoeSums(partial, ints[2 * (E + 1) + pairs : 2 * (E + 1) + 2 * pairs], ids, weights, x, E, shared, None)
+
+
+def _moe_combine(sums: MoeSums, out, h, y, norm_weight, eps, mult) -> None:
+    n, W = sums.x.shape
+    f = _fn("moe_combine.cu", "dli_moe_combine", [c_void_p] * 4 + [c_float] * 2 + [c_void_p] * 7 + [c_int] * 4 + [c_void_p])
+    _check(f(_ptr(out), _ptr(h), _ptr(y), _ptr(norm_weight), float(eps), float(mult), _ptr(sums.partial), _ptr(sums.pos), _ptr(sums.ids), _ptr(sums.weights),
+             _ptr(sums.x), _ptr(sums.shared), _ptr(sums.shared_rows), n, W, sums.experts, sums.ids.shape[1], _stream()), "moe_combine")
+
+
+def moe_combine(out: torch.Tensor, sums: MoeSums) -> None:
+    """out[t] = sum_k weights[t, k] * (the pair's row, or x[t] for an identity) (+ shared), in the order of k, float32, one rounding."""
+    _need(out, "out", torch.bfloat16)
+    if out.shape != sums.x.shape:
+        raise KernelError("moe_combine: out has the input's shape")
+    _moe_combine(sums, out, None, None, None, 0.0, 1.0)
+
+
+def moe_combine_norm_add(h: torch.Tensor, sums: MoeSums, weight: torch.Tensor, eps: float, mult: float, y: torch.Tensor | None = None) -> None:
+    """h += mult * v / sqrt(mean(v^2) + eps) * weight, v the sums of ``moe_combine`` (not rounded); with ``y`` the new h is also written there."""
+    _need(h, "h", torch.float32), _need(weight, "weight", torch.float32)
+    if h.shape != sums.x.shape or weight.numel() != h.shape[1] or h.shape[1] > MOE_NORM_ADD_MAX_SIZE:
+        raise KernelError(f"moe_combine_norm_add: h has the input's shape, a row at most {MOE_NORM_ADD_MAX_SIZE} numbers")
+    if y is not None:
+        _need(y, "y", torch.bfloat16)
+    _moe_combine(sums, None, h, y, weight, eps, mult)
+
+
 def moe_experts(out: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
                 activation: str = "silu", stages: int = 0, gated: bool = True, shared: torch.Tensor | None = None) -> None:
     """out[t] = sum_k weights[t, k] * y_k (+ shared[t]), added in the order of k in float32.  With e = ids[t, k] below E = len(w_down):
     y_k = down_e(act(gate_e x[t]) * (up_e x[t])), or down_e(act(up_e x[t])) without ``gated``; from E on the expert is the identity,
     y_k = x[t].  w_up [E, 2 ff, W] (an expert's gate rows, then its up rows) or [E, ff, W], w_down [E, W, ff].  The inner sums are
     rounded to the activation dtype before the activation, and so is what goes down.  ``activation``: one of GLU_ACTIVATIONS, or of
-    ACTIVATIONS without a gate.  ``stages`` (2, 3; 0: chosen from the step's shape): how deep the grouped products' asynchronous
-    copies run."""
-    _need(out, "out"), _need(x, "x", out.dtype), _need(ids, "ids", torch.int32), _need(weights, "weights", torch.float32)
-    _need(w_up, "w_up", out.dtype), _need(w_down, "w_down", out.dtype)
-    n, W = x.shape
-    top = ids.shape[1]
-    E, _, ff = w_down.shape
-    known = GLU_ACTIVATIONS if gated else ACTIVATIONS
-    if (out.dtype not in DT_CODE or tuple(out.shape) != (n, W) or tuple(w_up.shape) != (E, (2 if gated else 1) * ff, W) or w_down.shape[1] != W
-            or tuple(ids.shape) != (n, top) or tuple(weights.shape) != (n, top) or activation not in known):
-        raise KernelError("moe_experts: shapes, dtype or activation do not agree")
-    if shared is not None:
-        _need(shared, "shared", out.dtype)
-        if tuple(shared.shape) != (n, W):
-            raise KernelError("moe_experts: the shared expert's output must be [n, W]")
-    global launch_count
-    if moe_grouped_supported(n, W, ff, out.dtype):
-        # many tokens: the pairs sorted by expert, two grouped products on the tensor cores (csrc/moe_grouped.cu)
-        tiles = (min(n * top, E) + n * top // MOE_GROUPED_TILE_ROWS)
-        rows = tiles * MOE_GROUPED_TILE_ROWS
-        ints = torch.empty(2 * (E + 1) + 2 * n * top + tiles + rows, dtype=torch.int32, device=out.device)
-        hidden = torch.empty((rows, ff), dtype=out.dtype, device=out.device)
-        partial = torch.empty((rows, W), dtype=torch.float32, device=out.device)
-        g = _fn("moe_grouped.cu", "dli_moe_grouped", [c_void_p] * 10 + [c_int] * 8 + [c_void_p])
-        _check(g(_ptr(out), _ptr(x), _ptr(ids), _ptr(weights), _ptr(w_up), _ptr(w_down), _ptr(shared), _ptr(ints), _ptr(hidden), _ptr(partial), n, W, ff, E,
-                 top, known[activation], int(gated), int(stages), _stream()), "moe_experts")
-        launch_count += 3 if n * top <= 2048 else 6  # four kernels a call (one block sorts up to 2,048 pairs), else seven
+    ACTIVATIONS without a gate.  ``stages`` (2, 3; 0: chosen from the step's shape): the grouped products for many tokens, their
+    asynchronous copies that deep."""
+    n, W, top, E, ff, act = _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared)
+    _need(out, "out", x.dtype)
+    if tuple(out.shape) != (n, W):
+        raise KernelError("moe_experts: out has the input's shape")
+    if moe_products_supported(W, ff, x.dtype):
+        moe_combine(out, moe_products(x, ids, weights, w_up, w_down, activation, gated, shared, stages=stages, few=False if stages else None))
         return
+    global launch_count
     f = _fn("moe.cu", "dli_moe_pairs", [c_void_p] * 8 + [c_int] * 8 + [c_void_p])
     step = max(1, min(MOE_PAIR_CHUNK, 65535 // top))
     hidden = torch.empty((min(n, step) * top, ff), dtype=out.dtype, device=out.device)
     for t0 in range(0, n, step):
         m = min(step, n - t0)
         _check(f(_ptr(out[t0:]), _ptr(hidden), _ptr(x[t0:]), _ptr(ids[t0:]), _ptr(weights[t0:]), _ptr(w_up), _ptr(w_down),
-                 _ptr(None if shared is None else shared[t0:]), m, W, ff, E, top, known[activation], int(gated), DT_CODE[out.dtype], _stream()), "moe_experts")
+                 _ptr(None if shared is None else shared[t0:]), m, W, ff, E, top, act, int(gated), DT_CODE[out.dtype], _stream()), "moe_experts")
         launch_count += 1  # two kernels a call

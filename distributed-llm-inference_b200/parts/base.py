@@ -54,6 +54,9 @@ The outputs of two branches that run side by side stay pending as ``PendingSum(a
 A sublayer's output that is normed before the residual addition stays pending as ``PendingNormed(a, norm)``:
 a norm with ``post_add_norm(h, a, post, rows=None) -> y`` (h += post(a); y = norm(h), one kernel) takes it as
 it is; any other reader gets it settled first (``post.add_into(h, a)``).
+
+A feed-forward with an attribute ``defer_mixture`` (default False) may, when its owner set it, return a ``PendingMixture`` (experts'
+outputs not yet added up) for a norm with ``add_mixture_into``.
 """
 
 from __future__ import annotations
@@ -129,6 +132,23 @@ class PendingNormed:
 
     def __init__(self, a: torch.Tensor, norm) -> None:
         self.a, self.norm = a, norm
+
+
+class PendingMixture:
+    """The outputs of a mixture's experts that are still to be weighted and added up: a norm with ``add_mixture_into(h, mixture,
+    want_cast)`` does that, norms the sum and adds it to the stream in one kernel.  ``materialize()`` adds them up the plain way."""
+
+    __slots__ = ("sums",)
+
+    def __init__(self, sums) -> None:
+        self.sums = sums
+
+    def materialize(self) -> torch.Tensor:
+        from ..kernels import ops
+
+        out = torch.empty_like(self.sums.x)
+        ops.moe_combine(out, self.sums)
+        return out
 
 
 class PendingSum:

@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from ..weights.loader import TensorDecl
-from .base import BuildEnv, Part, PendingNormed, PendingScaled, PendingSum, ResidualStream, build_part, can_fuse, normed_input, register_part
+from .base import BuildEnv, Part, PendingMixture, PendingNormed, PendingScaled, PendingSum, ResidualStream, build_part, can_fuse, normed_input, register_part
 
 
 @register_part("arrangement", "prenorm")
@@ -204,6 +204,8 @@ class OutNormBlock(Part):
         for norm in (self.mixer_post_norm, *([self.ffn_post_norm] if self.has_ffn else [])):
             if not hasattr(norm, "add_scaled_into"):
                 raise ValueError("outnorm: the norm behind a sublayer must offer add_scaled_into(h, a, want_cast)")
+        if self.has_ffn and hasattr(self.ffn, "defer_mixture"):
+            self.ffn.defer_mixture = hasattr(self.ffn_post_norm, "add_mixture_into")
 
     def children(self):
         return [self.mixer, self.mixer_post_norm] + ([self.ffn, self.ffn_post_norm] if self.has_ffn else []) + self.after
@@ -219,9 +221,10 @@ class OutNormBlock(Part):
         h = stream.settle()
         dtype = self.env.dtype
         a = self.mixer.forward(stream.activation(dtype), batch, cache)
-        stream.cast = self.mixer_post_norm.add_scaled_into(h, a, want_cast=self.has_ffn or bool(self.after))
+        stream.cast = self.mixer_post_norm.add_scaled_into(h, a, want_cast=True)
         if self.has_ffn:
             f = self.ffn.forward(stream.activation(dtype))
-            stream.cast = self.ffn_post_norm.add_scaled_into(h, f, want_cast=bool(self.after))
+            add = self.ffn_post_norm.add_mixture_into if isinstance(f, PendingMixture) else self.ffn_post_norm.add_scaled_into
+            stream.cast = add(h, f, want_cast=True)
         for i, part in enumerate(self.after):
             part.apply(stream, batch, want_cast=True)

@@ -7,7 +7,7 @@ import torch
 from ..kernels import ops
 from ..kernels.gemm import dense_product, fused_epilogue, last_product, project
 from ..weights.loader import TensorDecl
-from .base import Part, build_part, register_part, tensor_name
+from .base import Part, PendingMixture, build_part, register_part, tensor_name
 
 
 @register_part("feed_forward", "glu")
@@ -125,13 +125,15 @@ class RoutedMLP(Part):
     feed-forward (a PartSpec; its weight is one), which runs for every token.
 
     One kernel routes; the tokens of every expert are then gathered by a counting sort on the device (no shape depends on
-    the data, so a step with this part can be recorded in a CUDA graph), and two grouped products run over the sorted rows; the
-    kernel that adds the outputs up reads the identities' input and the shared feed-forward's output in place.
+    the data, so a step with this part can be recorded in a CUDA graph), and two grouped products run over the sorted rows; a step of
+    few tokens is not sorted, and its shared feed-forward runs in the experts' launches.  The kernel that adds the outputs up reads
+    the identities' input and the shared feed-forward's output in place, and may also be the norm behind (``PendingMixture``).
     params: hidden_size, intermediate_size, num_experts, identity, top, route_scale, group_count, group_keep, activation, gated, score,
     shared, tensors (names of router, correction and, with ``{}`` for the expert's number, gate, up, down)."""
 
     graph_capturable = True
     takes_scaled_rows = False
+    defer_mixture = False  # set by an owner whose norm adds the outputs up itself (parts.base.PendingMixture)
 
     def __init__(self, spec, env) -> None:
         super().__init__(spec, env)
@@ -184,7 +186,16 @@ class RoutedMLP(Part):
         ids = torch.empty((n, self.top), dtype=torch.int32, device=x.device)
         weights = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
         ops.moe_route(ids, weights, x, self.w_router, self.correction, self.group_count, self.group_keep, self.route_scale, self.score)
-        out = torch.empty((n, self.hidden), dtype=x.dtype, device=x.device)
-        shared = self.shared.forward(x) if self.shared is not None else None
-        ops.moe_experts(out, x, ids, weights, self.w_up, self.w_down, self.activation, gated=self.gated, shared=shared)
-        return out
+        if not ops.moe_products_supported(self.hidden, self.inter, x.dtype):
+            out = torch.empty((n, self.hidden), dtype=x.dtype, device=x.device)
+            shared = self.shared.forward(x) if self.shared is not None else None
+            ops.moe_experts(out, x, ids, weights, self.w_up, self.w_down, self.activation, gated=self.gated, shared=shared)
+            return out
+        extra = shared = None
+        if self.shared is not None:
+            if n <= ops.MOE_FEW_MAX_TOKENS and not self.gated and isinstance(self.shared, DenseActMLP) and self.shared.inter % 8 == 0:
+                extra = (self.shared.w_up, self.shared.w_down, self.shared.activation)  # a few tokens: in the experts' launches
+            else:
+                shared = self.shared.forward(x)
+        mixture = PendingMixture(ops.moe_products(x, ids, weights, self.w_up, self.w_down, self.activation, self.gated, shared, extra))
+        return mixture if self.defer_mixture else mixture.materialize()

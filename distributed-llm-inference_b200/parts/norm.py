@@ -161,3 +161,11 @@ class GroupRMSNorm(Part):
         y = torch.empty_like(a) if want_cast and a.dtype != torch.float32 else None
         ops.group_norm_add(h, a, self.weight, self.groups, self.eps, self.mult, y)
         return y
+
+    def add_mixture_into(self, h: torch.Tensor, mixture, want_cast: bool = False) -> torch.Tensor | None:
+        """``add_scaled_into`` for a mixture whose experts' outputs are still to be added up: one kernel does both."""
+        if self.groups != 1 or self.size > ops.MOE_NORM_ADD_MAX_SIZE:
+            return self.add_scaled_into(h, mixture.materialize(), want_cast)
+        y = torch.empty_like(mixture.sums.x) if want_cast else None
+        ops.moe_combine_norm_add(h, mixture.sums, self.weight, self.eps, self.mult, y)
+        return y

@@ -857,7 +857,7 @@ OPS = {"embedding": embedding, "sinusoid_embedding": sinusoid_embedding, "qk_nor
        "depth_average": depth_average, "mingru_scan": mingru_scan, "diff_prep": diff_prep, "diff_attention_simt": diff_attention_simt,
        "diff_attention_tc": diff_attention_tc, "add_rmsnorm_scaled": add_rmsnorm_scaled, "concat_stream_rows": concat_stream_rows,
        "token_shift_blend": token_shift_blend, "rotary_unit_store": rotary_unit_store, "shift_decay_prep": shift_decay_prep,
-       "moe_grouped_supported": lambda tokens, W, ff, dtype: False, "channel_delta_prep": channel_delta_prep, "decay_recurrence": decay_recurrence, "moe_route": moe_route, "moe_experts": moe_experts}
+       "moe_products_supported": lambda W, ff, dtype: False, "channel_delta_prep": channel_delta_prep, "decay_recurrence": decay_recurrence, "moe_route": moe_route, "moe_experts": moe_experts}
 
 
 calls: dict[str, int] = {}  # how often each stand-in ran since patched() was entered

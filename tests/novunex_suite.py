@@ -197,7 +197,7 @@ def case_each_mechanism_alone(tmp_path, device, dtype):
         got = [s.step(("b", toks[:80], list(range(80))))] + [s.step(("b", [t], [0])) for t in toks[80:]]
         close(np.concatenate(got), want, dtype, name + ", the last ten decoded")
     for name, mlp in {"one_choice": moe(ff=24, experts=4, identity=2, top=1), "three": moe(ff=16, experts=7, identity=2, top=3), "all_chosen": moe(ff=8, experts=4, identity=2, top=6),
-                      "many": moe(ff=32, experts=40, identity=8, top=12, shared=64), "one_expert": moe(ff=24, experts=1, identity=0, top=1), "no_shared": moe(shared=0),
+                      "many": moe(ff=32, experts=26, identity=6, top=12, shared=64), "one_expert": moe(ff=24, experts=1, identity=0, top=1), "no_shared": moe(shared=0),
                       "more_identities": moe(ff=16, experts=2, identity=9, top=4), "wide_experts": moe(ff=136, experts=3, identity=1, top=2, shared=72),
                       "odd": moe(ff=21, experts=5, identity=2, top=2, shared=19)}.items():
         cfg = steady(config([first(heads=1, kv_heads=1, dim=8, vdim=8)], mlps=(mlp,)), dtype)

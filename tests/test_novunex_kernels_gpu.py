@@ -167,13 +167,14 @@ def test_router_by_softmax_over_all_outputs(dtype, tol):
 @pytest.mark.parametrize("dtype,tol", DTYPES)
 @pytest.mark.parametrize("sizes", [(48, 20, 5, 3, 3), (64, 64, 8, 0, 4), (40, 136, 3, 6, 5), (256, 72, 12, 4, 6), (200, 64, 1, 1, 2), (51, 11, 4, 2, 2), (320, 256, 4, 2, 3)])
 def test_experts(sizes, dtype, tol, gated):
-    """Experts with and without a gate beside identities, with and without a shared output, for one token, a few, and so many that the
-    sort takes several launches; expert counts that leave experts without tokens and tokens with identities alone."""
+    """Experts with and without a gate beside identities, with and without a shared output, for one token, as many as one, two and four
+    row tiles of the unsorted kernels hold and one more, and so many that the sort takes several launches; expert counts that leave
+    experts without tokens and tokens with identities alone."""
     W, ff, E, identity, top = sizes
     g = torch.Generator().manual_seed(3)
     w_up, w_down = _rand(E, (2 if gated else 1) * ff, W, seed=1, scale=1.0 / W**0.5).to(dtype), _rand(E, W, ff, seed=2, scale=1.0 / ff**0.5).to(dtype)
     act = "silu" if gated else "relu2"
-    for n in (1, 3, 17, 700):
+    for n in (1, 3, 16, 17, 33, 64, 65, 700):
         x, shared = _rand(n, W, seed=n).to(dtype), _rand(n, W, seed=n + 1).to(dtype)
         ids = torch.stack([torch.randperm(E + identity, generator=g)[:top] for _ in range(n)]).to(torch.int32)
         if identity >= top:
@@ -200,3 +201,66 @@ def test_plain_activations_of_experts():
             _close(got, want, tol, act)
     with pytest.raises(ops.KernelError):
         ops.moe_experts(got, args[0].cuda(), ids.cuda(), weights.cuda(), args[1].cuda(), args[2].cuda(), "quick_gelu", gated=False)
+
+
+@pytest.mark.parametrize("sizes", [(64, 64, 8, 2, 4, 128), (256, 72, 12, 4, 6, 40), (200, 136, 3, 1, 2, 264), (512, 128, 5, 0, 5, 8)])
+def test_a_feed_forward_rides_along(sizes):
+    """The shared feed-forward in the launches of few tokens' experts, wider and narrower than an expert; the sums added up, and added up,
+    normed and added to the stream in one kernel."""
+    W, ff, E, identity, top, shared_ff = sizes
+    bf = torch.bfloat16
+    g = torch.Generator().manual_seed(3)
+    w_up, w_down = _rand(E, ff, W, seed=1, scale=1.0 / W**0.5).to(bf), _rand(E, W, ff, seed=2, scale=1.0 / ff**0.5).to(bf)
+    s_up, s_down = _rand(shared_ff, W, seed=4, scale=1.0 / W**0.5).to(bf), _rand(W, shared_ff, seed=5, scale=1.0 / shared_ff**0.5).to(bf)
+    norm = 1 + 0.2 * _rand(W, seed=6)
+    for n in (1, 7, 16, 30, 64):
+        x = _rand(n, W, seed=n).to(bf)
+        ids = torch.stack([torch.randperm(E + identity, generator=g)[:top] for _ in range(n)]).to(torch.int32)
+        weights = torch.rand(n, top, generator=g)
+        hidden = torch.relu((x.float() @ s_up.float().t()).to(bf).float()) ** 2
+        shared = (hidden.to(bf).float() @ s_down.float().t())
+        want = torch.zeros(n, W)
+        ref.moe_experts(want, x.float(), ids, weights, w_up.float(), w_down.float(), "relu2", gated=False)
+        want += shared
+        d = [t.cuda() for t in (x, ids, weights, w_up, w_down)]
+        sums = ops.moe_products(*d, "relu2", gated=False, extra=(s_up.cuda(), s_down.cuda(), "relu2"))
+        out = torch.empty(n, W, dtype=bf, device="cuda")
+        ops.moe_combine(out, sums)
+        _close(out, want, 2e-2, f"{n} tokens")
+        h = _rand(n, W, seed=9)
+        h_dev, y = h.cuda(), torch.empty(n, W, dtype=bf, device="cuda")
+        ops.moe_combine_norm_add(h_dev, sums, norm.cuda(), 1e-3, 0.7, y)
+        h_want = h + 0.7 * want / torch.sqrt((want * want).mean(-1, keepdim=True) + 1e-3) * norm
+        _close(h_dev, h_want, 2e-2, f"{n} tokens, normed and added")
+        _close(y, h_want, 2e-2, f"{n} tokens, normed and added, rounded")
+        assert (y.float() - h_dev).abs().max() <= 0.01 * h_dev.abs().max()
+
+
+def test_sums_of_sorted_pairs_are_normed_and_added_too():
+    W, ff, E, top, n = 320, 64, 6, 3, 130
+    bf = torch.bfloat16
+    g = torch.Generator().manual_seed(5)
+    x, shared = _rand(n, W, seed=1).to(bf), _rand(n, W, seed=2).to(bf)
+    w_up, w_down = _rand(E, ff, W, seed=3, scale=1.0 / W**0.5).to(bf), _rand(E, W, ff, seed=4, scale=1.0 / ff**0.5).to(bf)
+    ids = torch.stack([torch.randperm(E + 2, generator=g)[:top] for _ in range(n)]).to(torch.int32)
+    weights, norm, h = torch.rand(n, top, generator=g), 1 + 0.2 * _rand(W, seed=6), _rand(n, W, seed=7)
+    want = torch.zeros(n, W)
+    ref.moe_experts(want, x.float(), ids, weights, w_up.float(), w_down.float(), "relu2", gated=False, shared=shared.float())
+    h_dev = h.cuda()
+    sums = ops.moe_products(x.cuda(), ids.cuda(), weights.cuda(), w_up.cuda(), w_down.cuda(), "relu2", gated=False, shared=shared.cuda())
+    ops.moe_combine_norm_add(h_dev, sums, norm.cuda(), 1e-5, 1.0)
+    _close(h_dev, h + want / torch.sqrt((want * want).mean(-1, keepdim=True) + 1e-5) * norm, 2e-2)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("score", ["sigmoid", "softmax", "softmax_chosen"])
+def test_routing_does_not_depend_on_how_many_tokens_there_are(dtype, score):
+    """The kernel for many tokens adds every sum up in the order of the one for few: the same choices and weights, bit for bit."""
+    W, E, top = 264, 21, 5
+    x, router, correction = _rand(603, W, seed=1).to(dtype).cuda(), _rand(E, W, seed=2, scale=0.1).cuda(), _rand(E, seed=3, scale=0.2).cuda()
+    ids, weights = torch.zeros(603, top, dtype=torch.int32, device="cuda"), torch.zeros(603, top, device="cuda")
+    ops.moe_route(ids, weights, x, router, correction, 3, 2, 1.5, score)
+    for first in range(0, 603, 201):
+        some_ids, some_weights = torch.zeros(201, top, dtype=torch.int32, device="cuda"), torch.zeros(201, top, device="cuda")
+        ops.moe_route(some_ids, some_weights, x[first : first + 201].contiguous(), router, correction, 3, 2, 1.5, score)
+        assert torch.equal(some_ids, ids[first : first + 201]) and torch.equal(some_weights, weights[first : first + 201])
