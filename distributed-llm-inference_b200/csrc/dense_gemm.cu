@@ -29,6 +29,10 @@
 //   acc_full[b]  (each CTA)   accumulator b is finished: the commit arrives in both CTAs
 //   acc_empty[b] (first CTA)  the epilogue threads of both CTAs (256) have read accumulator b
 //
+// The grouped form (one product per expert of a routed feed-forward, the rows of x sorted by expert and every expert's run padded to
+// whole tiles of 256) is the same kernel: how many tiles there are, and which expert's rows of W a tile reads, is looked up on the
+// device, so no launch depends on the data.
+//
 // Every wait on an mbarrier is bounded: after `wait_limit` polls the kernel records a code in *error_flag,
 // stops issuing work, frees its tensor memory and returns.  Neither CTA leaves before the other has reached the end.
 #include <cuda.h>
@@ -98,7 +102,8 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&v)[32]) {
 //                rotated by the token's position (rotate-half pairing over the first `rot` elements, rot 0, 64 or
 //                128; cosines and sines from the step's table [tokens, rot]: cos | sin); q goes to
 //                out[t, nh * d], k and v into the cache pages at the token's slot
-enum { EP_STORE = 0, EP_SWIGLU = 1, EP_ROTARY = 2 };
+//   EP_F32       out32[t, f] = sum, float32
+enum { EP_STORE = 0, EP_SWIGLU = 1, EP_ROTARY = 2, EP_F32 = 3 };
 struct DenseParams {
   __nv_bfloat16* out;
   int tokens, features, k_tiles, m_tiles, n_tiles;
@@ -113,6 +118,13 @@ struct DenseParams {
   int act;        // EP_STORE: an activation on the (bfloat16-rounded) sums before they are stored: 0 none, 1 relu^2, 2 gelu-tanh, 3 silu
                   // EP_SWIGLU: what is applied to the gate: 0 silu, 1 gelu-tanh, 2 g * sigmoid(1.702 g)
   float glu_limit, glu_shift;  // EP_SWIGLU: act(min(gate, limit)) * (clamp(up, -limit, limit) + shift); limit 0: no bounds
+  float* out32;   // EP_F32
+  // the grouped form: rows in use (a multiple of 256), the expert of every tile of 256 rows, the pair of every row (-1: padding, which is
+  // not written), and the rows of W an expert has
+  const int* used_rows;
+  const int* tile_expert;
+  const int* row_pair;
+  int expert_rows;
   int skip_tile;  // -1 in every launch of the engine: the k step whose copies a test leaves out (dli_dense_gemm_wait_test)
 };
 
@@ -150,8 +162,7 @@ __device__ __forceinline__ void load32(const float* src, float (&f)[32]) {
 // a warp touches one row per instruction; the extra passes cost more than the scattered sectors: q|k|v with rotary
 // 41 -> 74 us at 2,048 tokens.)  What an epilogue reads from global memory (cosines and sines) is asked for before
 // the accumulator's chunk is waited for, all loads of a chunk together.
-__device__ __forceinline__ void epilogue_row(const DenseParams& p, uint32_t acc, int row, int n) {
-  const bool live = row < p.tokens;
+__device__ __forceinline__ void epilogue_row(const DenseParams& p, uint32_t acc, int row, int n, bool live) {
   const int f0 = n * BN;  // first feature of the tile
   if (p.mode == EP_STORE) {
     __nv_bfloat16* dst = p.out + (size_t)row * p.features + f0;
@@ -173,6 +184,23 @@ __device__ __forceinline__ void epilogue_row(const DenseParams& p, uint32_t acc,
 #pragma unroll
         for (int j = 0; j < 32; j += 8)
           if (f0 + c + j < p.features) store8(dst + c + j, f + j);  // features are a multiple of 8
+      }
+    }
+    return;
+  }
+  if (p.mode == EP_F32) {
+    float* dst = p.out32 + (size_t)row * p.features + f0;
+#pragma unroll 1
+    for (int c = 0; c < BN && f0 + c < p.features; c += 32) {
+      float f[32];
+      load_chunk(acc + c, f);
+      if (live) {
+#pragma unroll
+        for (int j = 0; j < 32; j += 8)
+          if (f0 + c + j < p.features) {
+            *reinterpret_cast<float4*>(dst + c + j) = make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]);
+            *reinterpret_cast<float4*>(dst + c + j + 4) = make_float4(f[j + 4], f[j + 5], f[j + 6], f[j + 7]);
+          }
       }
     }
     return;
@@ -307,6 +335,7 @@ __device__ __forceinline__ void mbar_arrive_at(uint32_t bar, uint32_t cta) {
                ::"r"(bar), "r"(cta) : "memory");
 }
 
+template <bool GROUPED>
 __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x,
                                                                      const __grid_constant__ CUtensorMap map_w, const DenseParams p) {
   pdl_launch_dependents();
@@ -342,17 +371,21 @@ __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __gri
   cluster_sync_all();  // the other CTA's barriers are set up before anything is sent to them
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const uint32_t tmem = *tmem_slot;
-  const int m_pairs = (p.m_tiles + 1) / 2;  // tiles of 256 tokens
-  const int tiles = m_pairs * p.n_tiles;
+  // tiles of 256 tokens (the grouped form: the work of a kernel before this one, asked for behind pdl_wait)
+  auto m_pairs_of = [&]() -> int { return GROUPED ? *p.used_rows / (2 * BM) : (p.m_tiles + 1) / 2; };
   const int pair = blockIdx.x >> 1, pairs = gridDim.x >> 1;
 
   if (warp == 0) {
     // ---- copies: this CTA's 128 tokens and its half of the weight tile's rows
     if (lane == 0) {
       pdl_wait();  // the activations are the work of the kernel before this one
+      const int m_pairs = m_pairs_of(), tiles = m_pairs * p.n_tiles;
       int it = 0;
       for (int tile = pair; tile < tiles && !*failed; tile += pairs) {
         const int m = tile % m_pairs, n = tile / m_pairs;
+        // the grouped form fetches its half of the weight tile as two boxes of 64 rows: neighbours, or the gates and the ups of 64 features
+        const bool glu = GROUPED && p.mode == EP_SWIGLU;
+        const int w_row = GROUPED ? p.tile_expert[m] * p.expert_rows + n * (glu ? BN / 2 : BN) + (int)rank * (glu ? 64 : BN / 2) : n * BN + (int)rank * (BN / 2);
         for (int kt = 0; kt < p.k_tiles; ++kt, ++it) {
           const int s = it % PAIR_STAGES;
           if (it >= PAIR_STAGES && !mbar_wait(empty0 + 8 * s, ((it / PAIR_STAGES) - 1) & 1, p.wait_limit, failed)) {
@@ -363,7 +396,8 @@ __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __gri
           const uint32_t a = smem_u32(smem + (size_t)s * PAIR_STAGE_BYTES);
           if (rank == 0) mbar_expect_tx(full0 + 8 * s, 2 * PAIR_STAGE_BYTES);
           tma_load_2d_pair(a, &map_x, kt * BK, m * 2 * BM + (int)rank * BM, full0 + 8 * s);
-          tma_load_2d_pair(a + A_BYTES, &map_w, kt * BK, n * BN + (int)rank * (BN / 2), full0 + 8 * s);
+          tma_load_2d_pair(a + A_BYTES, &map_w, kt * BK, w_row, full0 + 8 * s);
+          if (GROUPED) tma_load_2d_pair(a + A_BYTES + PAIR_B_BYTES / 2, &map_w, kt * BK, w_row + (glu ? p.expert_rows / 2 : 64), full0 + 8 * s);
         }
       }
     }
@@ -372,6 +406,8 @@ __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __gri
     // ---- products: the first CTA's thread issues them for both
     if (lane == 0 && rank == 0) {
       const uint32_t idesc = instr_desc(2 * BM, BN);
+      if (GROUPED) pdl_wait();
+      const int tiles = m_pairs_of() * p.n_tiles;
       int it = 0, local = 0;
       for (int tile = pair; tile < tiles && !*failed; tile += pairs, ++local) {
         const int buf = local & 1;
@@ -405,6 +441,7 @@ __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __gri
     const int quad = warp & 3;
     const uint32_t lane_bits = (uint32_t)(quad * 32) << 16;
     pdl_wait();  // the output may alias memory that the kernel before this one still reads
+    const int m_pairs = m_pairs_of(), tiles = m_pairs * p.n_tiles;
     int local = 0;
     for (int tile = pair; tile < tiles; tile += pairs, ++local) {
       const int m = tile % m_pairs, n = tile / m_pairs;
@@ -414,7 +451,8 @@ __global__ void __launch_bounds__(THREADS, 1) dense_gemm_pair_kernel(const __gri
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      epilogue_row(p, tmem + buf * BN + lane_bits, m * 2 * BM + (int)rank * BM + quad * 32 + lane, n);
+      const int row = m * 2 * BM + (int)rank * BM + quad * 32 + lane;
+      epilogue_row(p, tmem + buf * BN + lane_bits, row, n, row < p.tokens && (!GROUPED || p.row_pair[row] >= 0));
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       mbar_arrive_at(acc_empty0 + 8 * buf, 0);
     }
@@ -482,16 +520,18 @@ static cudaError_t launch_pdl_x(void (*kernel)(KArgs...), dim3 grid, dim3 block,
   return cudaLaunchKernelEx(&cfg, kernel, args...);
 }
 
-static int launch_dense(DenseParams p, const void* x, const void* w, int tokens, int features, int K, cudaStream_t stream) {
+// grouped: w holds `experts` matrices [p.expert_rows, K] back to back, and p.used_rows, p.tile_expert and p.row_pair are set
+static int launch_dense(DenseParams p, const void* x, const void* w, int tokens, int features, int K, cudaStream_t stream, int experts = 0) {
   if (tokens < 1 || features < 8 || features % 8 || K < 8 || K % 8) return DLI_ERR_UNSUPPORTED;
-  if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)p.out) & 15) return DLI_ERR_UNSUPPORTED;
+  if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)p.out | (uintptr_t)p.out32) & 15) return DLI_ERR_UNSUPPORTED;
   if (!error_flag_host) {
     if (cudaHostAlloc((void**)&error_flag_host, sizeof(int), cudaHostAllocMapped) != cudaSuccess) return (int)cudaGetLastError();
     *error_flag_host = 0;
     if (cudaHostGetDevicePointer((void**)&error_flag_device, error_flag_host, 0) != cudaSuccess) return (int)cudaGetLastError();
   }
   CUtensorMap map_x, map_w;
-  if (!make_map(&map_x, x, tokens, K, BM) || !make_map(&map_w, w, features, K, BN / 2)) return DLI_ERR_UNSUPPORTED;  // W in boxes of half a tile's rows
+  // W in boxes of half a tile's rows (the grouped form: of a quarter)
+  if (!make_map(&map_x, x, tokens, K, BM) || !make_map(&map_w, w, experts ? (long long)experts * p.expert_rows : features, K, experts ? 64 : BN / 2)) return DLI_ERR_UNSUPPORTED;
   p.tokens = tokens; p.features = features;
   p.k_tiles = (K + BK - 1) / BK;
   p.m_tiles = (tokens + BM - 1) / BM;
@@ -503,15 +543,38 @@ static int launch_dense(DenseParams p, const void* x, const void* w, int tokens,
   }
   static OncePerDevice configured;
   if (!configured.here()) {
-    cudaError_t e = cudaFuncSetAttribute(dense_gemm_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES);
+    cudaError_t e = cudaFuncSetAttribute(dense_gemm_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(dense_gemm_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PAIR_SMEM_BYTES);
     if (e != cudaSuccess) return (int)e;
     configured.here() = true;
   }
   const long long tiles = (long long)((p.m_tiles + 1) / 2) * p.n_tiles;
   const long long pairs = sm_count() / 2;
   const int grid = 2 * (int)(tiles < pairs ? tiles : pairs);
-  cudaError_t e = launch_pdl_x(dense_gemm_pair_kernel, dim3(grid), dim3(THREADS), (size_t)PAIR_SMEM_BYTES, stream, 2, map_x, map_w, p);
+  cudaError_t e = launch_pdl_x(experts ? dense_gemm_pair_kernel<true> : dense_gemm_pair_kernel<false>, dim3(grid), dim3(THREADS), (size_t)PAIR_SMEM_BYTES, stream, 2,
+                               map_x, map_w, p);
   return (int)(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// One product per expert over rows sorted by expert.  x [rows, K]: the experts' runs, each padded to whole tiles of 256 rows; *used_rows of
+// them are in use (a multiple of 256 on the device, at most `rows`), tile_expert[i] is the expert of the rows 256 i .., row_pair[r] >= 0
+// says that row r holds something (other rows of the output are not written).  w [experts][features][K].
+//   epilogue 0: out [rows][features] bfloat16 = act(x w_e^T) (1 relu^2, 2 gelu-tanh, 3 silu)
+//   epilogue 1: out [rows][features / 2] bfloat16 = act(gate) * up, w_e the gates' rows, then the ups' (act 0 silu, 1 gelu-tanh, 2 g sigmoid(1.702 g))
+//   epilogue 2: out [rows][features] float32 = x w_e^T
+DLI_EXPORT int dli_dense_gemm_grouped(void* out, const void* x, const void* w, const int* used_rows, const int* tile_expert, const int* row_pair, int rows,
+                                      int features, int K, int experts, int epilogue, int act, cudaStream_t stream) {
+  if (experts < 1 || rows < 1 || rows % (2 * BM) || epilogue < 0 || epilogue > 2 || (epilogue == 0 && (act < 1 || act > 3)) ||
+      (epilogue == 1 && (features % 16 || act < 0 || act > 2)) || (long long)experts * features > 0x3fffffff || (uintptr_t)out & 15)
+    return DLI_ERR_UNSUPPORTED;
+  DenseParams p = {};
+  p.mode = epilogue == 0 ? EP_STORE : epilogue == 1 ? EP_SWIGLU : EP_F32;
+  if (epilogue == 2) p.out32 = (float*)out;
+  else p.out = (__nv_bfloat16*)out;
+  p.act = epilogue == 2 ? 0 : act;
+  p.used_rows = used_rows; p.tile_expert = tile_expert; p.row_pair = row_pair;
+  p.expert_rows = features;
+  return launch_dense(p, x, w, rows, features, K, stream, experts);
 }
 
 // out [tokens, features] = x [tokens, K] times w [features, K] transposed.  K and features multiples of 8.

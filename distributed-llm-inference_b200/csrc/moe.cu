@@ -1,6 +1,6 @@
-// A routed mixture of small feed-forwards: the router (float32 throughout), and the experts' products for steps of few
-// tokens, one (token, chosen expert) pair at a time on the CUDA cores.  (Steps of many tokens in bfloat16 take the
-// grouped tensor-core products of moe_grouped.cu.)
+// A routed mixture of small feed-forwards: the router (float32 throughout), and the experts' products one (token, chosen expert) pair at a
+// time on the CUDA cores, for float32 models and for sizes that the tensor-core products (moe_few.cu, the grouped form in dense_gemm.cu) do
+// not take.
 #include <math_constants.h>
 
 #include "common.cuh"

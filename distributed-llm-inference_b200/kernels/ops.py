@@ -1743,7 +1743,7 @@ def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, 
 # ------------------------------------------------------------------ routed mixture of small feed-forwards
 
 MOE_MAX_TOP = 32
-MOE_GROUPED_TILE_ROWS = 64  # BM of csrc/moe_grouped.cu
+MOE_TILE_ROWS = 256  # of a pair of SMs' tile in csrc/dense_gemm.cu
 MOE_FEW_MAX_TOKENS = 64  # up to here a step's experts are found without sorting the pairs (csrc/moe_few.cu)
 MOE_NORM_ADD_MAX_SIZE = 12288
 
@@ -1751,6 +1751,8 @@ MOE_NORM_ADD_MAX_SIZE = 12288
 def moe_products_supported(W: int, ff: int, dtype: torch.dtype) -> bool:
     """Whether the experts' products of a step go to the tensor-core kernels: bfloat16, rows of whole 16-byte chunks."""
     return dtype == torch.bfloat16 and W % 8 == 0 and ff % 8 == 0
+
+
 MOE_PAIR_CHUNK = 8192  # tokens a launch of the pair kernels takes (their grids count (token, expert) pairs along y)
 
 
@@ -1811,10 +1813,10 @@ def _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared):
 
 def moe_products(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, activation: str = "silu",
                  gated: bool = True, shared: torch.Tensor | None = None, extra: tuple[torch.Tensor, torch.Tensor, str] | None = None,
-                 stages: int = 0, few: bool | None = None) -> MoeSums:
+                 few: bool | None = None) -> MoeSums:
     """The experts' products of ``moe_experts`` in bfloat16, not yet added up.  Up to MOE_FEW_MAX_TOKENS tokens every chosen expert's matrix
-    is streamed once and nothing is sorted (csrc/moe_few.cu); more tokens are sorted by expert and take two grouped products
-    (csrc/moe_grouped.cu; ``few`` False: so do few).  ``extra`` (up [f, W], down [W, f], activation): a feed-forward without a gate that runs
+    is streamed once and nothing is sorted (csrc/moe_few.cu); more tokens are sorted by expert (csrc/moe_sort.cu) and take two
+    grouped tcgen05 products over tiles of 256 rows (csrc/dense_gemm.cu).  ``few`` True or False: the caller's choice.  ``extra`` (up [f, W], down [W, f], activation): a feed-forward without a gate that runs
     for every token and, with few tokens and beside experts without a gate, rides in the same launches."""
     n, W, top, E, ff, act = _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared)
     if not moe_products_supported(W, ff, x.dtype):
@@ -1838,16 +1840,22 @@ def moe_products(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up
         return MoeSums(partial, None, ids, weights, x, E, shared, pairs if extra is not None else None)
     if extra is not None:
         raise KernelError("moe_products: a feed-forward rides along with few tokens only")
-    tiles = min(pairs, E) + pairs // MOE_GROUPED_TILE_ROWS
-    rows = tiles * MOE_GROUPED_TILE_ROWS
+    tiles = min(pairs, E) + pairs // MOE_TILE_ROWS
+    rows = tiles * MOE_TILE_ROWS
+    # counts [E + 1] | offsets [E + 1] | rank [pairs] | pos [pairs] | tile_expert [tiles] | row_pair [rows]
     ints = torch.empty(2 * (E + 1) + 2 * pairs + tiles + rows, dtype=torch.int32, device=x.device)
+    used, pos, tile_expert, row_pair = (ints[at:] for at in (2 * E + 1, 2 * (E + 1) + pairs, 2 * (E + 1) + 2 * pairs, 2 * (E + 1) + 2 * pairs + tiles))
+    xs = torch.empty((rows, W), dtype=x.dtype, device=x.device)
     hidden = torch.empty((rows, ff), dtype=x.dtype, device=x.device)
     partial = torch.empty((rows, W), dtype=torch.float32, device=x.device)
-    g = _fn("moe_grouped.cu", "dli_moe_grouped", [c_void_p] * 7 + [c_int] * 8 + [c_void_p])
-    _check(g(_ptr(x), _ptr(ids), _ptr(w_up), _ptr(w_down), _ptr(ints), _ptr(hidden), _ptr(partial), n, W, ff, E, top, act, int(gated), int(stages), _stream()),
-           "moe_products")
-    launch_count += 2 if pairs <= 2048 else 5  # three kernels a call (one block sorts up to 2,048 pairs), else six
-    return MoeSums(partial, ints[2 * (E + 1) + pairs : 2 * (E + 1) + 2 * pairs], ids, weights, x, E, shared, None)
+    f = _fn("moe_sort.cu", "dli_moe_sort_gather", [c_void_p] * 4 + [c_int] * 5 + [c_void_p])
+    _check(f(_ptr(xs), _ptr(x), _ptr(ids), _ptr(ints), n, W, E, top, MOE_TILE_ROWS, _stream()), "moe_products")
+    launch_count += 1 if pairs <= 2048 else 4  # two kernels a call (one block sorts up to 2,048 pairs), else five
+    g = _fn("dense_gemm.cu", "dli_dense_gemm_grouped", [c_void_p] * 6 + [c_int] * 6 + [c_void_p])
+    maps = (_ptr(used), _ptr(tile_expert), _ptr(row_pair))
+    _check(g(_ptr(hidden), _ptr(xs), _ptr(w_up), *maps, rows, (2 if gated else 1) * ff, W, E, 1 if gated else 0, act if gated else act + 1, _stream()), "moe_products")
+    _check(g(_ptr(partial), _ptr(hidden), _ptr(w_down), *maps, rows, W, ff, E, 2, 0, _stream()), "moe_products")
+    return MoeSums(partial, pos, ids, weights, x, E, shared, None)
 
 
 def _moe_combine(sums: MoeSums, out, h, y, norm_weight, eps, mult) -> None:
@@ -1876,19 +1884,18 @@ def moe_combine_norm_add(h: torch.Tensor, sums: MoeSums, weight: torch.Tensor, e
 
 
 def moe_experts(out: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
-                activation: str = "silu", stages: int = 0, gated: bool = True, shared: torch.Tensor | None = None) -> None:
+                activation: str = "silu", gated: bool = True, shared: torch.Tensor | None = None) -> None:
     """out[t] = sum_k weights[t, k] * y_k (+ shared[t]), added in the order of k in float32.  With e = ids[t, k] below E = len(w_down):
     y_k = down_e(act(gate_e x[t]) * (up_e x[t])), or down_e(act(up_e x[t])) without ``gated``; from E on the expert is the identity,
     y_k = x[t].  w_up [E, 2 ff, W] (an expert's gate rows, then its up rows) or [E, ff, W], w_down [E, W, ff].  The inner sums are
     rounded to the activation dtype before the activation, and so is what goes down.  ``activation``: one of GLU_ACTIVATIONS, or of
-    ACTIVATIONS without a gate.  ``stages`` (2, 3; 0: chosen from the step's shape): the grouped products for many tokens, their
-    asynchronous copies that deep."""
+    ACTIVATIONS without a gate."""
     n, W, top, E, ff, act = _moe_sizes(x, ids, weights, w_up, w_down, activation, gated, shared)
     _need(out, "out", x.dtype)
     if tuple(out.shape) != (n, W):
         raise KernelError("moe_experts: out has the input's shape")
     if moe_products_supported(W, ff, x.dtype):
-        moe_combine(out, moe_products(x, ids, weights, w_up, w_down, activation, gated, shared, stages=stages, few=False if stages else None))
+        moe_combine(out, moe_products(x, ids, weights, w_up, w_down, activation, gated, shared))
         return
     global launch_count
     f = _fn("moe.cu", "dli_moe_pairs", [c_void_p] * 8 + [c_int] * 8 + [c_void_p])

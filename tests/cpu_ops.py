@@ -813,7 +813,7 @@ def _glu_act(g, activation):
 _plain_act = activation  # the stand-in of that name, which a parameter hides below
 
 
-def moe_experts(out, x, ids, weights, w_up, w_down, activation="silu", stages=0, gated=True, shared=None):
+def moe_experts(out, x, ids, weights, w_up, w_down, activation="silu", gated=True, shared=None):
     n, top = ids.shape
     E, _, ff = w_down.shape
     acc = torch.zeros((n, x.shape[1]))

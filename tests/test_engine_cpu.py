@@ -307,7 +307,7 @@ def test_bfloat16_logits_whole_in_portions_and_token_by_token(models, model_d64,
     assert ran.get("skinny_gemm_residual", 0) > 0 and ran.get("add_rmsnorm", 0) > 0 and ran.get("silu_mul", 0) > 0
     assert ran.get("skinny_gemm_rotary", 0) > 0 or cfg["head_dim"] == 48  # a head of 48 does not divide the product's tile
     assert (ran.get("skinny_gemm_swiglu", 0) > 0) == (cfg["intermediate_size"] % 64 == 0)
-    if name == "d64":
+    if cfg["head_dim"] > 32:  # heads that fill enough of a slab of 64 columns
         assert ran.get("paged_decode_tma", 0) > 0 and ran.get("paged_prefill_tc", 0) > 0 and "paged_attention_mma" not in ran
     else:
         assert ran.get("paged_attention_mma", 0) > 0 and "paged_decode_tma" not in ran

@@ -58,7 +58,7 @@ def detect():
 
 MUTANTS = {
     "llama3 scaling leaves the long wavelengths alone": (rotary_mod, "inverse_frequencies", "torch.where(wavelen > old / low, inv / factor, inv)", "torch.where(wavelen > old / low, inv, inv)"),
-    "linear scaling multiplies": (rotary_mod, "inverse_frequencies", "return inv / float(params[\"factor\"])", "return inv * float(params[\"factor\"])"),
+    "linear scaling multiplies": (rotary_mod, "inverse_frequencies", "(inv / float(params[\"factor\"]))", "(inv * float(params[\"factor\"]))"),
     "the feed-forward's output of the layer before is forgotten": (block_mod.PreNormBlock, "forward", "stream.take_pending(), self.mixer)", "None, self.mixer)"),
     "the mixer's output is not added": (block_mod.PreNormBlock, "forward", "normed_input(self.ffn_norm, stream.h, a, self.ffn)", "normed_input(self.ffn_norm, stream.h, None, self.ffn)"),
     "every layer writes into the first layer's cache": (model_mod.DecoderModel, "forward", "forward(stream, batch, caches[i])", "forward(stream, batch, caches[0])"),

@@ -31,7 +31,7 @@ def detect():
 SPEC = (config_mod, "novunex_model_spec")
 MUTANTS = {
     "the feed-forward reads the mixer's output": (OutNormBlock, "forward", "f = self.ffn.forward(stream.activation(dtype))", "f = self.ffn.forward(a)"),
-    "the feed-forward's norm is the mixer's": (OutNormBlock, "forward", "self.ffn_post_norm.add_scaled_into(h, f,", "self.mixer_post_norm.add_scaled_into(h, f,"),
+    "the feed-forward's norm is the mixer's": (OutNormBlock, "forward", "else self.ffn_post_norm.add_scaled_into", "else self.mixer_post_norm.add_scaled_into"),
     "the one in the denominator is left out": (SinkAttention, "forward", "sink=self.sink)", "sink=None)"),
     "every layer has the one in the denominator": (*SPEC, '"sink": 0.0 if first else None', '"sink": 0.0'),
     "the one is e": (*SPEC, '"sink": 0.0 if first else None', '"sink": 1.0 if first else None'),

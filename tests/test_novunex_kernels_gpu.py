@@ -165,7 +165,8 @@ def test_router_by_softmax_over_all_outputs(dtype, tol):
 
 @pytest.mark.parametrize("gated", [False, True])
 @pytest.mark.parametrize("dtype,tol", DTYPES)
-@pytest.mark.parametrize("sizes", [(48, 20, 5, 3, 3), (64, 64, 8, 0, 4), (40, 136, 3, 6, 5), (256, 72, 12, 4, 6), (200, 64, 1, 1, 2), (51, 11, 4, 2, 2), (320, 256, 4, 2, 3)])
+@pytest.mark.parametrize("sizes", [(48, 20, 5, 3, 3), (64, 64, 8, 0, 4), (40, 136, 3, 6, 5), (256, 72, 12, 4, 6), (200, 64, 1, 1, 2), (51, 11, 4, 2, 2), (320, 256, 4, 2, 3), (72, 328, 9, 1, 4),
+                                   (520, 384, 2, 0, 2)])
 def test_experts(sizes, dtype, tol, gated):
     """Experts with and without a gate beside identities, with and without a shared output, for one token, as many as one, two and four
     row tiles of the unsorted kernels hold and one more, and so many that the sort takes several launches; expert counts that leave
@@ -183,10 +184,15 @@ def test_experts(sizes, dtype, tol, gated):
         for sh in (shared, None):
             want, got = torch.zeros(n, W, dtype=dtype), torch.full((n, W), 7.0, dtype=dtype, device="cuda")
             ref.moe_experts(want, x, ids, weights, w_up, w_down, act, gated=gated, shared=sh)
-            for stages in (0, 2, 3):
-                ops.moe_experts(got, x.cuda(), ids.cuda(), weights.cuda(), w_up.cuda(), w_down.cuda(), act, stages=stages, gated=gated,
-                                shared=None if sh is None else sh.cuda())
-                _close(got, want, tol, f"{n} tokens, shared={sh is not None}, stages={stages}")
+            ops.moe_experts(got, x.cuda(), ids.cuda(), weights.cuda(), w_up.cuda(), w_down.cuda(), act, gated=gated, shared=None if sh is None else sh.cuda())
+            _close(got, want, tol, f"{n} tokens, shared={sh is not None}")
+            if ops.moe_products_supported(W, ff, dtype):  # every form of the products, whatever the step's shape would choose
+                for few in (False, True) if n <= ops.MOE_FEW_MAX_TOKENS else (False,):
+                    got.fill_(7.0)
+                    sums = ops.moe_products(x.cuda(), ids.cuda(), weights.cuda(), w_up.cuda(), w_down.cuda(), act, gated=gated,
+                                            shared=None if sh is None else sh.cuda(), few=few)
+                    ops.moe_combine(got, sums)
+                    _close(got, want, tol, f"{n} tokens, shared={sh is not None}, few={few}")
 
 
 def test_plain_activations_of_experts():
