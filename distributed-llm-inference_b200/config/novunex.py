@@ -164,7 +164,7 @@ def novunex_model_spec(cfg: NovunexConfig) -> ModelSpec:
         mixer = PartSpec("sink_attention", {
             "hidden_size": W, "num_heads": m.heads, "num_kv_heads": m.kv_heads, "head_dim": m.dim, "value_dim": m.vdim, "scale": m.scale,
             "position": _position(m), "sink": 0.0 if first else None, "qk_norm_eps": cfg.eps, "qk_norm": "head" if first else "projection",
-            "own_kv": m.kv_from is None, "tensors": names}, p + "mix.")
+            "own_kv": m.kv_from is None, "pad_rows": True, "tensors": names}, p + "mix.")
         parts = {"mixer": mixer, "mixer_post_norm": out_norm(p + "norm1")}
         f = layer.mlp
         if f is not None:

@@ -93,12 +93,13 @@ class SinkAttention(Part):
     * ``own_kv`` false: no key and value tensors; the layer's run step reads another step's cache (keys as that layer wrote them,
       normed and rotated) with its own queries, mask and everything else.
 
-    A cached token is one key row and one value row per KV head; in bfloat16 both are padded with zeros to a multiple of 16, for the
-    tensor-core kernels (and the output projection's matrix with zero columns to match, once, at load).
+    A cached token is one key row and one value row per KV head; with ``pad_rows`` both are padded with zeros to a multiple of 16 in
+    bfloat16, so that the tensor-core kernels serve every size (and the output projection's matrix with zero columns to match,
+    once, at load).
     One product yields q | k (| v) (| g); one kernel norms, rotates and writes the cache (the position part's
     ``norm_rotate_and_store``); the framework's attention kernels run with their sink argument.
     params: hidden_size, num_heads, num_kv_heads, head_dim, value_dim, scale, window, position (PartSpec), sink,
-    qk_norm_eps, qk_norm, values, gate, own_kv, tensors (names of q, k, v, g, o, q_norm, k_norm)."""
+    qk_norm_eps, qk_norm, values, gate, own_kv, pad_rows, tensors (names of q, k, v, g, o, q_norm, k_norm)."""
 
     graph_capturable = True
     takes_scaled_rows = False
@@ -110,7 +111,7 @@ class SinkAttention(Part):
         self.nh, self.nkv, self.d = int(p["num_heads"]), int(p["num_kv_heads"]), int(p["head_dim"])
         self.dv = int(p.get("value_dim") or self.d)
         self.row, self.vrow = self.d, self.dv  # what a page keeps per token and KV head: of keys, of values
-        if env.dtype == torch.bfloat16:
+        if p.get("pad_rows") and env.dtype == torch.bfloat16:
             self.row, self.vrow = -(-self.d // 16) * 16, -(-self.dv // 16) * 16
         self.scale = float(p["scale"])
         self.window = p.get("window")
