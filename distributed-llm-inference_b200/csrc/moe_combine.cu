@@ -95,7 +95,7 @@ DLI_EXPORT int dli_moe_combine(void* out, float* h, void* y, const float* norm_w
                                const float* weights, const void* x, const void* shared, const float* shared_rows, int n, int W, int E, int top,
                                cudaStream_t stream) {
   if (n == 0) return 0;
-  if (W < 8 || (W % 8) || top < 1 || E < 1 || (h ? !norm_w || W > 12288 : !out) ||
+  if (W < 8 || (W % 8) || top < 1 || E < 1 || (h ? !norm_w || W > 12160 : !out) ||
       ((((uintptr_t)out) | ((uintptr_t)h) | ((uintptr_t)y) | ((uintptr_t)norm_w) | ((uintptr_t)partial) | ((uintptr_t)x) | ((uintptr_t)shared) | ((uintptr_t)shared_rows)) & 15))
     return DLI_ERR_UNSUPPORTED;
   const Params p{partial, pos, ids, weights, (const bf16*)x, (const bf16*)shared, shared_rows, W, E, top};

@@ -1745,7 +1745,7 @@ def matrix_memory_scan(o: torch.Tensor, divisor: torch.Tensor, u: torch.Tensor, 
 MOE_MAX_TOP = 32
 MOE_TILE_ROWS = 256  # of a pair of SMs' tile in csrc/dense_gemm.cu
 MOE_FEW_MAX_TOKENS = 64  # up to here a step's experts are found without sorting the pairs (csrc/moe_few.cu)
-MOE_NORM_ADD_MAX_SIZE = 12288
+MOE_NORM_ADD_MAX_SIZE = 12160  # a row of float32 and the reduction's scratch in 48 KB
 
 
 def moe_products_supported(W: int, ff: int, dtype: torch.dtype) -> bool:
